@@ -18,6 +18,8 @@ from . import lilupel as _lilupel  # registers the architecture
 from .lilupel import LilupelConfig
 from . import darusun as _darusun  # registers the architecture
 from .darusun import DarusunConfig
+from . import dibedra as _dibedra  # registers the architecture
+from .dibedra import DibedraConfig
 
 
 def read_config_json(folder: str) -> dict:

@@ -63,7 +63,53 @@ struct DecodeQkv {
     float q_scale;
 };
 
+// What a mixer may do to a head besides: a root-mean-square norm per head of q and k before the rotation (32-bit, a weight
+// of the head size shared by the heads), neighbouring dims paired in the rotation (dim 2i with 2i + 1), values that are
+// the keys as projected, rows that go on behind the heads read here, and a gate per element on the result.  The query
+// heads of a key/value head may be shared out among ``chunks`` blocks (more than eight of them on one key head).  Comes with
+// an entry point of its own, for the same reason as the record above.
+struct DecodeHead {
+    const float* q_gamma;        // [hd]
+    const float* k_gamma;        // [hd]
+    float eps;
+    int ld;                      // columns of a row of DecodeQkv.qkv
+    int v_from_k;                // the values are the key columns as projected; rows hold no v
+    int gate_off;                // >= 0: the result of head h is multiplied by sigmoid(row[gate_off + h * hd + d])
+    int chunks;
+};
+
 #include "decode_common.cuh"
+
+// One 16-byte chunk (8 dims from dim 8 c on) of a head, normed (times inv and the weight), its pairs turned and scaled.
+__device__ __forceinline__ uint4 ad_head_chunk(const __nv_bfloat16* head, int c, float inv, const float* gamma, int half,
+                                               const float* cs, const float* sn, float sc) {
+    const uint4 raw = *(const uint4*)(head + c * 8);
+    const __nv_bfloat162* p2 = (const __nv_bfloat162*)&raw;
+    __nv_bfloat162 o2[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(p2[e]);
+        const float u = f.x * inv * gamma[c * 8 + 2 * e], w = f.y * inv * gamma[c * 8 + 2 * e + 1];
+        const int i = c * 4 + e;
+        float co = 1.f, si = 0.f;
+        if (cs && i < half) { co = cs[i]; si = sn[i]; }
+        o2[e] = __floats2bfloat162_rn((u * co - w * si) * sc, (w * co + u * si) * sc);
+    }
+    return *(const uint4*)o2;
+}
+__device__ __forceinline__ float ad_sum_sq(const __nv_bfloat16* head, int c) {
+    const uint4 raw = *(const uint4*)(head + c * 8);
+    const __nv_bfloat162* p2 = (const __nv_bfloat162*)&raw;
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(p2[e]); s = fmaf(f.x, f.x, s); s = fmaf(f.y, f.y, s); }
+    return s;
+}
+__device__ __forceinline__ float ad_gate(const DecodeQkv& x, const DecodeHead& hh, int b, int h, int d) {
+    if (hh.gate_off < 0) return 1.f;
+    const float g = __bfloat162float(x.qkv[(size_t)b * hh.ld + hh.gate_off + (size_t)h * AD_HD + d]);
+    return 1.0f / (1.0f + __expf(-g));
+}
 
 __device__ __forceinline__ void ad_cp16(unsigned dst, const void* src, int bytes) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes));
@@ -85,22 +131,24 @@ __device__ __forceinline__ void ad_load_page(unsigned dst, const __nv_bfloat16* 
     }
 }
 
-// CLUSTER: the splits of one (sequence, key/value head) are the blocks of a cluster
-template <bool CLUSTER>
+// CLUSTER: the splits of one (sequence, key/value head) are the blocks of a cluster.  HEAD: DecodeHead applies.
+template <bool CLUSTER, bool HEAD>
 __global__ void __launch_bounds__(AD_THREADS)
-attn_decode_kernel(DecodeArgs a, DecodeQkv x) {
+attn_decode_kernel(DecodeArgs a, DecodeQkv x, DecodeHead hh) {
     extern __shared__ __align__(16) unsigned char smem[];
     // stage s: keys at 2 s AD_TILE, values one tile further; then per-warp scratch
     const unsigned sbase = ad_smem(smem);
     __nv_bfloat16* pw = (__nv_bfloat16*)(smem + 2 * AD_STAGES * AD_TILE);      // [4 warps][8 heads][16 keys]
     float* mrg = (float*)(smem + 2 * AD_STAGES * AD_TILE + 4 * 8 * 16 * 2);    // [4][8][2] then [4][hd][G]
 
-    const int split = blockIdx.x, g = blockIdx.y, b = blockIdx.z;
+    const int chunks = HEAD ? hh.chunks : 1;              // blocks that share a key/value head's query heads
+    const int split = blockIdx.x, g = blockIdx.y / chunks, b = blockIdx.z;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int grp = lane >> 2, t = lane & 3;
     gl_grid_launch_dependents();
     gl_grid_wait();
-    const int G = a.nH / a.nKV;                          // query heads of this key/value head (<= 8)
+    const int G = a.nH / (a.nKV * chunks);               // query heads of this block (<= 8)
+    const int h0 = HEAD ? (int)blockIdx.y * G : g * G;   // the first of them
     const int pos = a.seq_ctx[b];                        // the query's position; keys lo..pos
     const int lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
     const int first_page = lo / GL_PAGE, n_pages = pos / GL_PAGE + 1 - first_page;
@@ -124,8 +172,41 @@ attn_decode_kernel(DecodeArgs a, DecodeQkv x) {
     }
     // the queries as the 8-column operand: column = head within the group, rows = head dims
     unsigned qb[AD_KS][2];
-    const size_t qkv_row = (size_t)(a.nH + 2 * a.nKV) * AD_HD;
-    if (x.qkv) {
+    const size_t qkv_row = HEAD ? (size_t)hh.ld : (size_t)(a.nH + 2 * a.nKV) * AD_HD;
+    float inv_k = 1.f;                                   // HEAD: the new key's norm
+    if constexpr (HEAD) {
+        // this block's query heads and the new key: sums of squares chunk by chunk, then norm, rotation and scale
+        __nv_bfloat16* qs = (__nv_bfloat16*)mrg;                       // [G][hd], free until the merge
+        float* ss = mrg + (size_t)G * AD_HD;                           // [G + 1][hd / 8]
+        const float* cs = x.cosv ? x.cosv + (size_t)b * x.half : nullptr;
+        const float* sn = x.sinv ? x.sinv + (size_t)b * x.half : nullptr;
+        const __nv_bfloat16* row = x.qkv + (size_t)b * qkv_row;
+        for (int i = tid; i < (G + 1) * AD_CHUNKS; i += AD_THREADS) {
+            const int hq = i / AD_CHUNKS, c = i - hq * AD_CHUNKS;
+            ss[i] = ad_sum_sq(row + (size_t)(hq < G ? h0 + hq : a.nH + g) * AD_HD, c);
+        }
+        __syncthreads();
+        {
+            float s = 0.f;
+            for (int c = 0; c < AD_CHUNKS; ++c) s += ss[G * AD_CHUNKS + c];
+            inv_k = 1.0f / sqrtf(s / (float)AD_HD + hh.eps);
+        }
+        for (int i = tid; i < G * AD_CHUNKS; i += AD_THREADS) {
+            const int hq = i / AD_CHUNKS, c = i - hq * AD_CHUNKS;
+            float s = 0.f;
+            for (int k = 0; k < AD_CHUNKS; ++k) s += ss[hq * AD_CHUNKS + k];
+            const float inv = 1.0f / sqrtf(s / (float)AD_HD + hh.eps);
+            *(uint4*)(qs + hq * AD_HD + c * 8) = ad_head_chunk(row + (size_t)(h0 + hq) * AD_HD, c, inv, hh.q_gamma, x.half, cs, sn, x.q_scale);
+        }
+        __syncthreads();
+        const __nv_bfloat16* qh = qs + grp * AD_HD;
+#pragma unroll
+        for (int kk = 0; kk < AD_KS; ++kk) {
+            qb[kk][0] = grp < G ? *(const unsigned*)(qh + kk * 16 + 2 * t) : 0u;
+            qb[kk][1] = grp < G ? *(const unsigned*)(qh + kk * 16 + 8 + 2 * t) : 0u;
+        }
+        __syncthreads();
+    } else if (x.qkv) {
         // rotated and scaled here: the group's query heads through this block's corner of shared memory
         __nv_bfloat16* qs = (__nv_bfloat16*)mrg;                       // [G][hd], free until the merge
         const float* cs = x.cosv ? x.cosv + (size_t)b * x.half : nullptr;
@@ -178,13 +259,22 @@ attn_decode_kernel(DecodeArgs a, DecodeQkv x) {
             // the row of this block's copy of the page that the copy from the cache brought stale
             if (tid < 2 * AD_CHUNKS) {
                 const int c = tid % AD_CHUNKS, is_v = tid / AD_CHUNKS, r = pos % GL_PAGE;
+                uint4 val;
+                if constexpr (HEAD) {
+                    const __nv_bfloat16* key = x.qkv + (size_t)b * qkv_row + ((size_t)a.nH + g) * AD_HD;
+                    if (is_v) val = *(const uint4*)(key + (hh.v_from_k ? 0 : (size_t)a.nKV * AD_HD) + c * 8);
+                    else val = ad_head_chunk(key, c, inv_k, hh.k_gamma, x.half, x.cosv ? x.cosv + (size_t)b * x.half : nullptr,
+                                             x.sinv ? x.sinv + (size_t)b * x.half : nullptr, 1.0f);
+                } else {
                 const __nv_bfloat16* head = x.qkv + (size_t)b * qkv_row + ((size_t)a.nH + (size_t)is_v * a.nKV + g) * AD_HD;
                 const float* cs = (!is_v && x.cosv) ? x.cosv + (size_t)b * x.half : nullptr;
                 const float* sn = (!is_v && x.sinv) ? x.sinv + (size_t)b * x.half : nullptr;
-                const uint4 val = ad_rotated_chunk(head, c, is_v ? 0 : x.half, cs, sn, 1.0f);
+                val = ad_rotated_chunk(head, c, is_v ? 0 : x.half, cs, sn, 1.0f);
+                }
                 *(uint4*)(smem + (2 * st + is_v) * AD_TILE + r * AD_ROW + c * 16) = val;
                 __nv_bfloat16* cache = (__nv_bfloat16*)(is_v ? a.v_cache : a.k_cache);
-                *(uint4*)(cache + (size_t)pg[p] * page_stride + head_off + (size_t)r * AD_HD + c * 8) = val;
+                if (!HEAD || blockIdx.y % chunks == 0)       // (one of the blocks that share the key head stores it)
+                    *(uint4*)(cache + (size_t)pg[p] * page_stride + head_off + (size_t)r * AD_HD + c * 8) = val;
             }
             __syncthreads();
         }
@@ -283,9 +373,11 @@ attn_decode_kernel(DecodeArgs a, DecodeQkv x) {
             ov = fmaf(f, o_w[((size_t)w * AD_HD + d) * G + hq], ov);
             l = fmaf(f, ml_w[(w * 8 + hq) * 2 + 1], l);
         }
-        const int h = g * G + hq;
+        const int h = h0 + hq;
         if (a.splits == 1) {
-            a.out[((size_t)b * a.nH + h) * AD_HD + d] = __float2bfloat16_rn(l > 0.f ? ov / l : 0.f);
+            float y = l > 0.f ? ov / l : 0.f;
+            if constexpr (HEAD) y *= ad_gate(x, hh, b, h, d);
+            a.out[((size_t)b * a.nH + h) * AD_HD + d] = __float2bfloat16_rn(y);
         } else if (CLUSTER) {
             fin_o[i] = ov;
             if (d == 0) { fin_ml[2 * hq] = m; fin_ml[2 * hq + 1] = l; }
@@ -316,7 +408,9 @@ attn_decode_kernel(DecodeArgs a, DecodeQkv x) {
                 ov = fmaf(f, cluster.map_shared_rank(fin_o, s)[i], ov);
                 l = fmaf(f, pml[2 * hq + 1], l);
             }
-            a.out[((size_t)b * a.nH + g * G + hq) * AD_HD + d] = __float2bfloat16_rn(l > 0.f ? ov / l : 0.f);
+            float y = l > 0.f ? ov / l : 0.f;
+            if constexpr (HEAD) y *= ad_gate(x, hh, b, h0 + hq, d);
+            a.out[((size_t)b * a.nH + h0 + hq) * AD_HD + d] = __float2bfloat16_rn(y);
         }
         cluster.sync();
     }
@@ -348,21 +442,22 @@ static size_t decode_smem(int G) {
     return 2 * AD_STAGES * (size_t)AD_TILE + 4 * 8 * 16 * 2 + sizeof(float) * (64 + 5 * (size_t)AD_HD * G + 2 * G);
 }
 
-static int launch_decode(const DecodeArgs& a, const DecodeQkv& x, cudaStream_t stream) {
+template <bool HEAD>
+static int launch_decode(const DecodeArgs& a, const DecodeQkv& x, const DecodeHead& hh, cudaStream_t stream) {
     static bool configured = false;
-    const size_t smem = decode_smem(a.nH / a.nKV);
+    const size_t smem = decode_smem(a.nH / (a.nKV * hh.chunks));
     if (!configured) {
-        if (cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(AD_MAXG)) != cudaSuccess ||
-            cudaFuncSetAttribute(attn_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(AD_MAXG)) != cudaSuccess) {
+        if (cudaFuncSetAttribute(attn_decode_kernel<false, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(AD_MAXG)) != cudaSuccess ||
+            cudaFuncSetAttribute(attn_decode_kernel<true, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(AD_MAXG)) != cudaSuccess) {
             cudaGetLastError();
             return GL_ERR_SMEM;
         }
         configured = true;
     }
-    const dim3 grid(a.splits, a.nKV, a.B);
+    const dim3 grid(a.splits, a.nKV * hh.chunks, a.B);
     if (a.splits > 1 && a.splits <= 8 && !a.part_o)
-        return gl_launch(attn_decode_kernel<true>, grid, dim3(AD_THREADS), smem, stream, a.splits, a, x);
-    return gl_launch(attn_decode_kernel<false>, grid, dim3(AD_THREADS), smem, stream, 1, a, x);
+        return gl_launch(attn_decode_kernel<true, HEAD>, grid, dim3(AD_THREADS), smem, stream, a.splits, a, x, hh);
+    return gl_launch(attn_decode_kernel<false, HEAD>, grid, dim3(AD_THREADS), smem, stream, 1, a, x, hh);
 }
 
 GL_API int gl_attention_decode_head_dim() { return AD_HD; }
@@ -387,13 +482,28 @@ GL_API int gl_attention_decode_qkv(const DecodeArgs* args, const DecodeQkv* extr
     return decode_checked(*args, x, stream);
 }
 
+// the same for a mixer with normed heads, values that are its keys, or a gate on the result (up to 8 splits)
+GL_API int gl_attention_decode_head(const DecodeArgs* args, const DecodeQkv* extra, const DecodeHead* head, cudaStream_t stream) {
+    const DecodeArgs& a = *args;
+    const DecodeQkv& x = *extra;
+    const DecodeHead& hh = *head;
+    if (a.B <= 0) return GL_OK;
+    if (!x.qkv || !hh.q_gamma || !hh.k_gamma || x.half < 0 || 2 * x.half > AD_HD || (x.half > 0 && (!x.cosv || !x.sinv))) return GL_ERR_SHAPE;
+    if (a.nH <= 0 || a.nKV <= 0 || hh.chunks <= 0 || a.nH % (a.nKV * hh.chunks) || a.nH / (a.nKV * hh.chunks) > AD_MAXG) return GL_ERR_SHAPE;
+    if (a.splits < 1 || a.splits > 8 || a.part_o || a.part_ml || a.B > 65535 || a.nKV * hh.chunks > 65535) return GL_ERR_SHAPE;
+    if (hh.ld % 8 || hh.ld < (a.nH + (hh.v_from_k ? 1 : 2) * a.nKV) * AD_HD || (hh.gate_off >= 0 && hh.gate_off + a.nH * AD_HD > hh.ld)) return GL_ERR_SHAPE;
+    if (((uintptr_t)x.qkv | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15) return GL_ERR_ALIGN;
+    return launch_decode<true>(a, x, hh, stream);
+}
+
 static int decode_checked(const DecodeArgs& a, const DecodeQkv& x, cudaStream_t stream) {
     if (a.B <= 0) return GL_OK;
     if (a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV || a.nH / a.nKV > AD_MAXG) return GL_ERR_SHAPE;
     if (a.splits < 1 || a.B > 65535 || a.nKV > 65535) return GL_ERR_SHAPE;
     if (a.splits > 8 && (!a.part_o || !a.part_ml)) return GL_ERR_SHAPE;     // more than a cluster holds: scratch
     if ((a.part_o == nullptr) != (a.part_ml == nullptr)) return GL_ERR_SHAPE;
-    const int rc = launch_decode(a, x, stream);
+    const DecodeHead none = {nullptr, nullptr, 0.f, 0, 0, -1, 1};
+    const int rc = launch_decode<false>(a, x, none, stream);
     if (rc != GL_OK) return rc;
     if (a.splits > 1 && a.part_o) {
         return gl_launch(attn_decode_merge_kernel, dim3(a.nH, a.B), dim3(AD_HD >= 128 ? 128 : 64), 0, stream, 1, a);

@@ -85,6 +85,13 @@ struct AttnArgs {
     float score_scale;
 };
 
+// A gate on the result, element by element: head h's output at token t is multiplied by sigmoid(gate[t, off + h*hd + d]).
+// A record of its own with an entry point of its own, so that AttnArgs stays what callers compiled against.
+struct AttnGate {
+    const __nv_bfloat16* gate;    // [T, ld] or null (no gate); ld and off multiples of 8
+    int ld, off;
+};
+
 struct AttnMaps { CUtensorMap q[4], k[4], v; };
 
 __device__ __forceinline__ float at_exp2(float x) {
@@ -94,7 +101,7 @@ __device__ __forceinline__ float at_exp2(float x) {
 }
 
 __global__ void __launch_bounds__(AT_THREADS, 1)
-attn_prefill_tc_kernel(AttnArgs a, const __grid_constant__ AttnMaps maps) {
+attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMaps maps) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ unsigned tmem_slot;
     __shared__ volatile int failed;
@@ -359,6 +366,17 @@ attn_prefill_tc_kernel(AttnArgs a, const __grid_constant__ AttnMaps maps) {
                 for (int c = 0; c < AT_HD; c += 16) {
                     unsigned t16[16];
                     tmem_ld16(tO + c, t16);
+                    if (gate.gate && r < rows) {
+                        const uint4* gp = (const uint4*)(gate.gate + (size_t)(qstart + q0 + t * AT_BM + r) * gate.ld + gate.off + h * AT_HD + c);
+                        const uint4 graw[2] = {gp[0], gp[1]};
+                        const __nv_bfloat162* g2 = (const __nv_bfloat162*)graw;
+#pragma unroll
+                        for (int i = 0; i < 16; i += 2) {
+                            const float2 f = __bfloat1622float2(g2[i / 2]);
+                            t16[i] = __float_as_uint(__uint_as_float(t16[i]) / (1.f + __expf(-f.x)));
+                            t16[i + 1] = __float_as_uint(__uint_as_float(t16[i + 1]) / (1.f + __expf(-f.y)));
+                        }
+                    }
                     if (r < rows) {
                         uint4 pk[2];
                         unsigned* pw = (unsigned*)pk;
@@ -399,9 +417,7 @@ GL_API int gl_attention_prefill_tc_wait_failed() {
     return v;
 }
 
-// n_tokens: rows of q; n_pages: pages of the cache entry
-GL_API int gl_attention_prefill_tc(const AttnArgs* args, int n_tokens, int n_pages, cudaStream_t stream) {
-    const AttnArgs& a = *args;
+static int prefill_tc(const AttnArgs& a, const AttnGate& gate, int n_tokens, int n_pages, cudaStream_t stream) {
     if (a.B <= 0 || a.max_qlen <= 0) return GL_OK;
     if (a.hd != AT_HD || a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV) return GL_ERR_SHAPE;
     if (a.score_scale != 1.0f) return GL_ERR_SHAPE;
@@ -430,6 +446,19 @@ GL_API int gl_attention_prefill_tc(const AttnArgs* args, int n_tokens, int n_pag
     }
     const long long blocks = (long long)((a.max_qlen + 2 * AT_BM - 1) / (2 * AT_BM)) * a.nH * a.B;
     if (blocks > 0x7fffffffLL) return GL_ERR_SHAPE;
-    if (gl_launch(attn_prefill_tc_kernel, dim3((unsigned)blocks), dim3(AT_THREADS), smem, stream, 1, a, maps) != 0) return GL_ERR_LAUNCH;
+    if (gl_launch(attn_prefill_tc_kernel, dim3((unsigned)blocks), dim3(AT_THREADS), smem, stream, 1, a, gate, maps) != 0) return GL_ERR_LAUNCH;
     return GL_OK;
+}
+
+// n_tokens: rows of q; n_pages: pages of the cache entry
+GL_API int gl_attention_prefill_tc(const AttnArgs* args, int n_tokens, int n_pages, cudaStream_t stream) {
+    const AttnGate none = {nullptr, 0, 0};
+    return prefill_tc(*args, none, n_tokens, n_pages, stream);
+}
+
+// the same with a gate on the result
+GL_API int gl_attention_prefill_tc_gated(const AttnArgs* args, const AttnGate* gate, int n_tokens, int n_pages, cudaStream_t stream) {
+    if (!gate->gate || gate->ld % 8 || gate->off < 0 || gate->off % 8 || gate->off + args->nH * AT_HD > gate->ld) return GL_ERR_SHAPE;
+    if ((uintptr_t)gate->gate & 15) return GL_ERR_ALIGN;
+    return prefill_tc(*args, *gate, n_tokens, n_pages, stream);
 }

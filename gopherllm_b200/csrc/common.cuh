@@ -202,6 +202,20 @@ __device__ __forceinline__ float gl_activate(float x, int act) {
     }
 }
 
+// A gated feed-forward's inner value from its gate and its up projection: act(gate) * up, or with GL_GATED_CLIPPED (a
+// sigmoid-weighted gate with both sides clipped: numbers limit, slope, shift)
+//   g = min(gate, limit), u = clamp(up, -limit, limit):   g * sigmoid(slope * g) * (u + shift).
+#define GL_GATED_CLIPPED 32
+struct GlGated { int act; float limit, slope, shift; };
+template <bool EXACT>
+__device__ __forceinline__ float gl_gated(float g, float u, const GlGated& p) {
+    if (p.act != GL_GATED_CLIPPED) return gl_activate<EXACT>(g, p.act) * u;
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+    const float e = EXACT ? expf(-p.slope * g) : __expf(-p.slope * g);
+    return g / (1.0f + e) * (u + p.shift);
+}
+
 // the same for callers that carry an activation's own numbers along
 template <bool EXACT>
 __device__ __forceinline__ float gl_activate(float x, int act, float p0, float p1) {

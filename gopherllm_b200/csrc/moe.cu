@@ -3,12 +3,16 @@
 //   route     scores s = sigmoid(z) of a token's router logits; with groups, the experts form equal groups of
 //             neighbours, a group's score is the sum of its two largest scores and only experts of the best
 //             ``keep`` groups may be chosen; the ``top`` largest scores are chosen (the lower index wins a
-//             tie); their weights are s / (sum of the chosen s + 1e-20) * scale.  All 32-bit.
+//             tie); their weights are s / (sum of the chosen s + 1e-20) * scale.  All 32-bit.  Other forms: the
+//             softmax over the chosen logits alone; the softmax over all, with a correction that decides the choice
+//             but not the weights, which stay as they are.  A group's score may be its largest score instead.
+//             The router may have more outputs than there are experts: the others are the identity, a choice of
+//             which adds the token's input itself; they take no part in the plan and the products.
 //   plan      the step's assignments (token, choice) sorted by expert, and the list of row tiles: every
 //             expert's rows cut into tiles of MOE_TM, so that a grid of fixed size (an upper bound of tiles)
 //             covers whatever the router chose without the host learning of it.
 //   gate_up   for every tile: rows gathered from the tokens' inputs, times the expert's gate and up weights,
-//             silu(gate) * up written in sorted order.
+//             silu(gate) * up (or another gated form) written in sorted order.
 //   down      for every tile: those rows times the expert's down weights, times the assignment's weight,
 //             written 32-bit at the assignment's own place [token, choice].
 //   combine   out[t] = sum over a token's choices (in the order of the choices) + what is to be added.
@@ -33,14 +37,31 @@ struct RouteArgs {
     int T, E, top, groups, keep;
     float scale;
     const float* bias;        // [E] or null: added to the logits
-    int softmax_chosen;       // 1: the largest LOGITS are chosen and weighted by the softmax over the chosen logits alone
-                              // (times scale; one group); 0: sigmoid scores as above
+    int mode;                 // ROUTE_SIGMOID: sigmoid scores as above; ROUTE_SOFTMAX_CHOSEN: the largest LOGITS are chosen and
+                              // weighted by the softmax over the chosen logits alone (times scale; one group);
+                              // ROUTE_SOFTMAX_ALL: scores are the softmax over all logits; the largest s + correction are
+                              // chosen and weighted by s itself (times scale), not renormalised
+    const float* correction;  // [E] or null (ROUTE_SOFTMAX_ALL): joins the choice, not the weights; may be negative
+    int group_largest;        // a group's score is its largest score, not the sum of its two largest
 };
+
+enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_CHOSEN = 1, ROUTE_SOFTMAX_ALL = 2 };
+
+// floats of shared memory a token's choice needs: scores, group scores, and for the softmax over all its weights
+__host__ __device__ __forceinline__ int moe_choice_floats(const RouteArgs& a) {
+    return a.E + a.groups + (a.mode == ROUTE_SOFTMAX_ALL ? a.E : 0);
+}
+
+static bool route_possible(const RouteArgs& a) {
+    if (a.E <= 0 || a.top <= 0 || a.top > a.E || a.groups <= 0 || a.E % a.groups || a.keep <= 0 || a.keep > a.groups) return false;
+    if (a.mode < ROUTE_SIGMOID || a.mode > ROUTE_SOFTMAX_ALL || (a.correction && a.mode != ROUTE_SOFTMAX_ALL)) return false;
+    return (long long)a.keep * (a.E / a.groups) >= a.top && !(a.mode == ROUTE_SOFTMAX_CHOSEN && a.groups != 1);
+}
 
 // a token's score for expert e from its logit
 __device__ __forceinline__ float moe_score(const RouteArgs& a, float z, int e) {
     if (a.bias) z += a.bias[e];
-    return a.softmax_chosen ? z : 1.0f / (1.0f + expf(-z));
+    return a.mode == ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-z)) : z;
 }
 
 // the largest value among sc[e], e = first + lane, first + lane + 32, ... < last, and its (lowest) index
@@ -57,16 +78,31 @@ __device__ __forceinline__ void moe_argmax(const float* sc, int first, int last,
         const int oa = __shfl_xor_sync(0xffffffffu, at, o);
         if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
     }
+    if (at == 0x7fffffff) at = first;        // (no number among them: an index inside the range all the same)
 }
 
 __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float* gsc, int t, int lane) {
+    float* prob = gsc + a.groups;                            // [E] (ROUTE_SOFTMAX_ALL)
+    if (a.mode == ROUTE_SOFTMAX_ALL) {
+        float top = -INFINITY, sum = 0.f;
+        for (int e = lane; e < a.E; e += 32) top = fmaxf(top, sc[e]);
+        top = gl_warp_max(top);
+        for (int e = lane; e < a.E; e += 32) { const float p = expf(sc[e] - top); prob[e] = p; sum += p; }
+        sum = gl_warp_sum(sum);
+        for (int e = lane; e < a.E; e += 32) {
+            const float s = prob[e] / sum;
+            prob[e] = s;
+            sc[e] = a.correction ? s + a.correction[e] : s;
+        }
+        __syncwarp();
+    }
     if (a.groups > 1 && a.keep < a.groups) {
         const int per = a.E / a.groups;
         for (int g = 0; g < a.groups; ++g) {
             float b1, b2 = 0.f;
             int i1, i2;
             moe_argmax(sc, g * per, (g + 1) * per, lane, b1, i1);
-            if (per > 1) {
+            if (per > 1 && !a.group_largest) {
                 const float keep1 = sc[i1];
                 __syncwarp();
                 if (lane == 0) sc[i1] = -INFINITY;
@@ -89,10 +125,25 @@ __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float*
             __syncwarp();
         }
         for (int e = lane; e < a.E; e += 32)
-            if (gsc[e / per] != -INFINITY) sc[e] = -1.0f;    // scores lie in (0, 1): -1 is never chosen before them
+            if (gsc[e / per] != -INFINITY) sc[e] = -INFINITY;
         __syncwarp();
     }
-    if (a.softmax_chosen) {
+    if (a.mode == ROUTE_SOFTMAX_ALL) {
+        for (int k = 0; k < a.top; ++k) {
+            float b;
+            int e;
+            moe_argmax(sc, 0, a.E, lane, b, e);
+            __syncwarp();
+            if (lane == 0) {
+                a.ids[(size_t)t * a.top + k] = e;
+                a.weights[(size_t)t * a.top + k] = prob[e] * a.scale;
+                sc[e] = -INFINITY;
+            }
+            __syncwarp();
+        }
+        return;
+    }
+    if (a.mode == ROUTE_SOFTMAX_CHOSEN) {
         float first = 0.f, sum = 0.f;
         for (int k = 0; k < a.top; ++k) {
             float b;
@@ -123,7 +174,7 @@ __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float*
         if (lane == 0) {
             a.ids[(size_t)t * a.top + k] = e;
             a.weights[(size_t)t * a.top + k] = b;
-            sc[e] = -2.0f;
+            sc[e] = -INFINITY;
         }
         __syncwarp();
     }
@@ -140,7 +191,7 @@ moe_route_kernel(RouteArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= a.T) return;
-    float* sc = smem + (size_t)warp * (a.E + a.groups);      // [E] scores, then [groups] group scores
+    float* sc = smem + (size_t)warp * moe_choice_floats(a);  // [E] scores, then [groups] group scores, then [E] weights
     float* gsc = sc + a.E;
     for (int e = lane; e < a.E; e += 32) sc[e] = moe_score(a, a.logits[(size_t)t * a.E + e], e);
     __syncwarp();
@@ -168,7 +219,7 @@ moe_route_from_kernel(RouteFromArgs f) {
     const int t = blockIdx.x;
     float* sc = smem;                        // [E] scores
     float* gsc = sc + a.E;                   // [groups] group scores
-    float* xs = gsc + a.groups;              // [K] the token's input
+    float* xs = smem + moe_choice_floats(a); // [K] the token's input
     const TA* x = (const TA*)f.x + (size_t)t * f.K;
     for (int k = threadIdx.x; k < f.K; k += 128) xs[k] = gl_load(x + k);
     __syncthreads();
@@ -187,9 +238,8 @@ GL_API int gl_moe_route_from(const RouteFromArgs* args, int x_dtype, cudaStream_
     const RouteFromArgs& f = *args;
     const RouteArgs& a = f.r;
     if (a.T <= 0) return GL_OK;
-    if (f.K <= 0 || a.E <= 0 || a.top <= 0 || a.top > a.E || a.groups <= 0 || a.E % a.groups || a.keep <= 0 || a.keep > a.groups) return GL_ERR_SHAPE;
-    if ((long long)a.keep * (a.E / a.groups) < a.top || (a.softmax_chosen && a.groups != 1)) return GL_ERR_SHAPE;
-    const size_t smem = (size_t)(a.E + a.groups + f.K) * sizeof(float);
+    if (f.K <= 0 || !route_possible(a)) return GL_ERR_SHAPE;
+    const size_t smem = (size_t)(moe_choice_floats(a) + f.K) * sizeof(float);
     if (smem > 48 * 1024) return GL_ERR_SMEM;
     int rc;
     if (x_dtype == GL_F32) rc = gl_launch(moe_route_from_kernel<float>, dim3(a.T), dim3(128), smem, stream, 1, f);
@@ -201,9 +251,8 @@ GL_API int gl_moe_route_from(const RouteFromArgs* args, int x_dtype, cudaStream_
 GL_API int gl_moe_route(const RouteArgs* args, cudaStream_t stream) {
     const RouteArgs& a = *args;
     if (a.T <= 0) return GL_OK;
-    if (a.E <= 0 || a.top <= 0 || a.top > a.E || a.groups <= 0 || a.E % a.groups || a.keep <= 0 || a.keep > a.groups) return GL_ERR_SHAPE;
-    if ((long long)a.keep * (a.E / a.groups) < a.top || (a.softmax_chosen && a.groups != 1)) return GL_ERR_SHAPE;
-    const size_t smem = 4 * (size_t)(a.E + a.groups) * sizeof(float);
+    if (!route_possible(a)) return GL_ERR_SHAPE;
+    const size_t smem = 4 * (size_t)moe_choice_floats(a) * sizeof(float);
     if (smem > 48 * 1024) return GL_ERR_SMEM;
     return gl_launch(moe_route_kernel, dim3((a.T + 3) / 4), dim3(128), smem, stream, 1, a) == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
@@ -212,7 +261,7 @@ GL_API int gl_moe_route(const RouteArgs* args, cudaStream_t stream) {
 // The plan: one block.
 // ---------------------------------------------------------------------------
 struct PlanArgs {
-    const int* ids;           // [A] expert of every assignment (A = tokens * top)
+    const int* ids;           // [A] expert of every assignment (A = tokens * top); E and above: the identity, left out
     int* order;               // [A] assignments sorted by expert
     int* tile_expert;         // [max_tiles]
     int* tile_start;          // [max_tiles] first place in ``order``
@@ -232,9 +281,8 @@ moe_plan_kernel(PlanArgs a) {
     for (int e = threadIdx.x; e < a.E; e += blockDim.x) count[e] = 0;
     __syncthreads();
     for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        int e = a.ids[i];
-        e = e < 0 ? 0 : (e >= a.E ? a.E - 1 : e);
-        atomicAdd(&count[e], 1);
+        const int e = a.ids[i];
+        if ((unsigned)e < (unsigned)a.E) atomicAdd(&count[e], 1);
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -260,9 +308,8 @@ moe_plan_kernel(PlanArgs a) {
     }
     __syncthreads();
     for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        int e = a.ids[i];
-        e = e < 0 ? 0 : (e >= a.E ? a.E - 1 : e);
-        a.order[atomicAdd(&start[e], 1)] = i;
+        const int e = a.ids[i];
+        if ((unsigned)e < (unsigned)a.E) a.order[atomicAdd(&start[e], 1)] = i;
     }
 }
 
@@ -284,7 +331,7 @@ GL_API int gl_moe_plan(const PlanArgs* args, cudaStream_t stream) {
 struct PadPlanArgs {
     const int* ids;           // [A]
     int* order;               // [max_tiles * tile_m]
-    int* place;               // [A]
+    int* place;               // [A]; -1: the identity
     int* tile_expert;         // [max_tiles]
     int A, E, max_tiles, tile_m;
 };
@@ -301,9 +348,8 @@ moe_plan_padded_kernel(PadPlanArgs a) {
     for (int i = threadIdx.x; i < a.max_tiles * a.tile_m; i += blockDim.x) a.order[i] = -1;
     __syncthreads();
     for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        int e = a.ids[i];
-        e = e < 0 ? 0 : (e >= a.E ? a.E - 1 : e);
-        atomicAdd(&count[e], 1);
+        const int e = a.ids[i];
+        if ((unsigned)e < (unsigned)a.E) atomicAdd(&count[e], 1);
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -317,8 +363,8 @@ moe_plan_padded_kernel(PadPlanArgs a) {
     }
     __syncthreads();
     for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        int e = a.ids[i];
-        e = e < 0 ? 0 : (e >= a.E ? a.E - 1 : e);
+        const int e = a.ids[i];
+        if ((unsigned)e >= (unsigned)a.E) { a.place[i] = -1; continue; }
         const int row = atomicAdd(&start[e], 1);
         if (row < a.max_tiles * a.tile_m) a.order[row] = i;
         a.place[i] = row;
@@ -357,28 +403,43 @@ GL_API int gl_moe_gather_rows(const void* x, const int* order, void* xs, int row
                      (__nv_bfloat16*)xs, K, top) == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
-// out[t, :] = sum_k weights[t, k] * y[place[t, k], :] (+ add[t, :]), in the order of the choices
+// out[t, :] = sum_k weights[t, k] * y[place[t, k], :] (+ add[t, :]), in the order of the choices; a place of -1 is the
+// identity: the token's input x[t, :] (bfloat16) takes y's part.  Four columns a thread.
 __global__ void __launch_bounds__(256)
-moe_combine_placed_kernel(const float* y, const int* place, const float* weights, const float* add, float* out,
-                          long long n, int N, int top) {
+moe_combine_placed_kernel(const float* y, const int* place, const float* weights, const __nv_bfloat16* x, const float* add,
+                          float* out, long long n4, int N4, int top) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= n) return;
-    const long long t = i / N;
-    const int c = (int)(i - t * N);
-    float s = 0.f;
-    for (int k = 0; k < top; ++k) s += weights[t * top + k] * y[(size_t)place[t * top + k] * N + c];
-    out[i] = add ? add[i] + s : s;
+    if (i >= n4) return;
+    const long long t = i / N4;
+    const int c = (int)(i - t * N4);
+    float4 s = add ? ((const float4*)add)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k = 0; k < top; ++k) {
+        const float w = weights[t * top + k];
+        const int row = place[t * top + k];
+        float4 v;
+        if (row >= 0) {
+            v = ((const float4*)y)[(size_t)row * N4 + c];
+        } else {
+            const uint2 raw = ((const uint2*)x)[(size_t)t * N4 + c];
+            const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
+            v = make_float4(a.x, a.y, b.x, b.y);
+        }
+        sum.x = fmaf(w, v.x, sum.x); sum.y = fmaf(w, v.y, sum.y); sum.z = fmaf(w, v.z, sum.z); sum.w = fmaf(w, v.w, sum.w);
+    }
+    ((float4*)out)[i] = make_float4(s.x + sum.x, s.y + sum.y, s.z + sum.z, s.w + sum.w);
 }
 
-GL_API int gl_moe_combine_placed(const float* y, const int* place, const float* weights, const float* add, float* out,
-                                 int T, int N, int top, cudaStream_t stream) {
+GL_API int gl_moe_combine_placed(const float* y, const int* place, const float* weights, const void* x, const float* add,
+                                 float* out, int T, int N, int top, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
-    if (N <= 0 || top <= 0) return GL_ERR_SHAPE;
-    const long long n = (long long)T * N;
-    return gl_launch(moe_combine_placed_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, y, place, weights,
-                     add, out, n, N, top) == 0 ? GL_OK : GL_ERR_LAUNCH;
+    if (N <= 0 || N % 4 || top <= 0 || !x) return GL_ERR_SHAPE;
+    if (((uintptr_t)y | (uintptr_t)add | (uintptr_t)out) & 15 || ((uintptr_t)x & 7)) return GL_ERR_ALIGN;
+    const long long n4 = (long long)T * (N / 4);
+    return gl_launch(moe_combine_placed_kernel, dim3((unsigned)((n4 + 255) / 256)), dim3(256), 0, stream, 1, y, place, weights,
+                     (const __nv_bfloat16*)x, add, out, n4, N / 4, top) == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 // ---------------------------------------------------------------------------
@@ -397,6 +458,7 @@ struct ExpertArgs {
     const float* weights;     // [A] by assignment (down)
     int A, N, K, top, max_tiles;
     int E;                    // experts (to choose a kernel by the rows an expert meets on average)
+    GlGated act;              // gate_up: the gated form
 };
 
 #define MOE_TN 64
@@ -477,7 +539,7 @@ moe_expert_simt_kernel(ExpertArgs a) {
             if (n >= a.N) continue;
             if (GATED) {
                 const float g = acc0[i][j];
-                gl_store((TA*)a.out + (size_t)(start + r) * a.N + n, g / (1.0f + expf(-g)) * acc1[i][j]);
+                gl_store((TA*)a.out + (size_t)(start + r) * a.N + n, gl_gated<true>(g, acc1[i][j], a.act));
             } else {
                 const int asg = a.order[start + r];
                 ((float*)a.out)[(size_t)asg * a.N + n] = acc0[i][j] * a.weights[asg];
@@ -601,7 +663,7 @@ moe_expert_tc_kernel(ExpertArgs a) {
                 if (r >= nrows || n >= a.N) continue;
                 if (GATED) {
                     const float g = acc0[i][j][f];
-                    ((__nv_bfloat16*)a.out)[(size_t)(start + r) * a.N + n] = __float2bfloat16_rn(g / (1.0f + __expf(-g)) * acc1[i][j][f]);
+                    ((__nv_bfloat16*)a.out)[(size_t)(start + r) * a.N + n] = __float2bfloat16_rn(gl_gated<false>(g, acc1[i][j][f], a.act));
                 } else {
                     const int asg = a.order[start + r];
                     ((float*)a.out)[(size_t)asg * a.N + n] = acc0[i][j][f] * a.weights[asg];
@@ -704,7 +766,7 @@ moe_expert_rows_kernel(ExpertArgs a) {
                 const float u = GATED ? gl_warp_sum(accu[c][r]) : 0.f;
                 if (lane != 0 || n >= a.N) continue;
                 if (GATED) {
-                    ((__nv_bfloat16*)a.out)[(size_t)(start + r0 + r) * a.N + n] = __float2bfloat16_rn(g / (1.0f + __expf(-g)) * u);
+                    ((__nv_bfloat16*)a.out)[(size_t)(start + r0 + r) * a.N + n] = __float2bfloat16_rn(gl_gated<false>(g, u, a.act));
                 } else {
                     const int asg = a.order[start + r0 + r];
                     ((float*)a.out)[(size_t)asg * a.N + n] = g * a.weights[asg];
@@ -754,10 +816,13 @@ GL_API int gl_moe_down_simt(const ExpertArgs* args, int x_dtype, int w_dtype, cu
 }
 
 // ---------------------------------------------------------------------------
-// out[t, :] = sum_k y[t, k, :] (+ add[t, :]); out may be add itself.
+// out[t, :] = sum_k y[t, k, :] (+ add[t, :]); out may be add itself.  A choice at or above E is the identity: its part
+// is weights[t, k] * x[t, :].
 // ---------------------------------------------------------------------------
+template <typename TA>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const float* y, const float* add, float* out, long long n, int N, int top) {
+moe_combine_kernel(const float* y, const int* ids, const float* weights, const TA* x, const float* add, float* out, long long n,
+                   int N, int top, int E) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -765,16 +830,22 @@ moe_combine_kernel(const float* y, const float* add, float* out, long long n, in
     const long long t = i / N;
     const int c = (int)(i - t * N);
     float s = 0.f;
-    for (int k = 0; k < top; ++k) s += y[((size_t)t * top + k) * N + c];
+    for (int k = 0; k < top; ++k)
+        s += ids[t * top + k] < E ? y[((size_t)t * top + k) * N + c] : weights[t * top + k] * gl_load(x + (size_t)t * N + c);
     out[i] = add ? add[i] + s : s;
 }
 
-GL_API int gl_moe_combine(const float* y, const float* add, float* out, int T, int N, int top, cudaStream_t stream) {
+GL_API int gl_moe_combine(const float* y, const int* ids, const float* weights, const void* x, int x_dtype, const float* add,
+                          float* out, int T, int N, int top, int E, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
-    if (N <= 0 || top <= 0) return GL_ERR_SHAPE;
+    if (N <= 0 || top <= 0 || E <= 0) return GL_ERR_SHAPE;
     const long long n = (long long)T * N;
-    return gl_launch(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, y, add, out, n, N, top) == 0
-               ? GL_OK : GL_ERR_LAUNCH;
+    const dim3 grid((unsigned)((n + 255) / 256));
+    int rc;
+    if (x_dtype == GL_F32) rc = gl_launch(moe_combine_kernel<float>, grid, dim3(256), 0, stream, 1, y, ids, weights, (const float*)x, add, out, n, N, top, E);
+    else if (x_dtype == GL_BF16) rc = gl_launch(moe_combine_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, 1, y, ids, weights, (const __nv_bfloat16*)x, add, out, n, N, top, E);
+    else return GL_ERR_DTYPE;
+    return rc == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 // ---------------------------------------------------------------------------

@@ -31,9 +31,10 @@ GL_API int gl_rope_table(const int* pos, const float* inv_freq, float* cosv, flo
 }
 
 // The same tables from 64-bit frequencies: the angle pos * freq is a 64-bit product, so a table entry is
-// the correctly rounded cosine of the exact angle whatever the position.
+// the correctly rounded cosine of the exact angle whatever the position.  ``gain`` multiplies both tables (frequencies
+// stretched for longer contexts come with one).
 __global__ void rope_table64_kernel(const int* pos, const double* __restrict__ freq,
-                                    float* __restrict__ cosv, float* __restrict__ sinv, int T, int half) {
+                                    float* __restrict__ cosv, float* __restrict__ sinv, int T, int half, double gain) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     gl_grid_launch_dependents();
     gl_grid_wait();
@@ -41,15 +42,15 @@ __global__ void rope_table64_kernel(const int* pos, const double* __restrict__ f
     const int t = i / half, p = i % half;
     double s, c;
     sincos((double)pos[t] * freq[p], &s, &c);
-    cosv[i] = (float)c;
-    sinv[i] = (float)s;
+    cosv[i] = (float)(c * gain);
+    sinv[i] = (float)(s * gain);
 }
 
 GL_API int gl_rope_table64(const int* pos, const double* freq, float* cosv, float* sinv,
-                           int T, int half, cudaStream_t stream) {
+                           int T, int half, double gain, cudaStream_t stream) {
     if (T <= 0 || half <= 0) return GL_OK;
     const int n = T * half;
-    return gl_launch(rope_table64_kernel, dim3((n + 127) / 128), dim3(128), 0, stream, 1, pos, freq, cosv, sinv, T, half);
+    return gl_launch(rope_table64_kernel, dim3((n + 127) / 128), dim3(128), 0, stream, 1, pos, freq, cosv, sinv, T, half, gain);
 }
 
 struct QkvCacheArgs {
@@ -70,6 +71,8 @@ struct QkvCacheArgs {
     int interleaved, norm_rms, write_kv;
     float eps, q_scale;
     int n_pages;              // pages of the cache entry (read by builds that check indices; 0: unknown)
+    int ld;                   // columns of a row of qkv (0: (nH + 2 nKV) * hd): rows may go on behind the heads read here
+    int v_from_k;             // the values are the key columns as projected, before norm and rotation: rows hold no v
 };
 
 template <typename TA, typename TC>
@@ -86,7 +89,8 @@ __global__ void qkv_cache_kernel(QkvCacheArgs a) {
     if (kind != 0 && !a.write_kv) return;
     const int hd = a.hd;
     float* v = smem + warp * hd;
-    const TA* src = (const TA*)a.qkv + (size_t)t * heads * hd + (size_t)j * hd;
+    // (values that are the keys as projected are read from the key's columns)
+    const TA* src = (const TA*)a.qkv + (size_t)t * (a.ld > 0 ? a.ld : heads * hd) + (size_t)(kind == 2 && a.v_from_k ? j - a.nKV : j) * hd;
     for (int d = lane; d < hd; d += 32) v[d] = gl_load(src + d);
     __syncwarp();
 
@@ -205,11 +209,89 @@ qkv_cache_bf16_kernel(QkvCacheArgs a) {
     }
 }
 
+// bfloat16 rows and cache with a root-mean-square norm per head and neighbouring dims paired (dim 2i with 2i + 1): a lane
+// owns 8 dims of a head, that is four whole pairs, so only the sum of squares crosses lanes (a butterfly among the
+// head's LPH lanes, the next power of two at or above hd / 8).  Values that are the keys as projected are stored by the
+// lane that holds the key's raw dims.  Needs the head size and the row length to be multiples of 8.
+template <int LPH>
+__global__ void __launch_bounds__(128)
+qkv_headnorm_bf16_kernel(QkvCacheArgs a) {
+    gl_grid_launch_dependents();
+    const int c = threadIdx.x % LPH, chunks = a.hd >> 3;
+    const int heads = a.write_kv ? (a.v_from_k ? a.nH + a.nKV : a.nH + 2 * a.nKV) : a.nH;
+    const long long item = ((long long)blockIdx.x * 128 + threadIdx.x) / LPH;
+    const bool live = item < (long long)a.T * heads && c < chunks;
+    const int t = live ? (int)(item / heads) : 0, j = live ? (int)(item - (long long)t * heads) : 0;
+    const int kind = j < a.nH ? 0 : (j < a.nH + a.nKV ? 1 : 2);           // q, k, v
+    float gm[8];                                                          // (a weight: asked for before the wait)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) gm[e] = (live && kind != 2) ? (kind == 0 ? a.q_gamma : a.k_gamma)[c * 8 + e] : 0.f;
+    gl_grid_wait();
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (live) raw = *(const uint4*)((const __nv_bfloat16*)a.qkv + (size_t)t * a.ld + (size_t)j * a.hd + c * 8);
+    float v[8], s = 0.f;
+    const __nv_bfloat162* p2 = (const __nv_bfloat162*)&raw;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(p2[e]); v[2 * e] = f.x; v[2 * e + 1] = f.y; }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (!live) return;
+    uint4 out = raw;
+    if (kind != 2) {
+        const float inv = 1.0f / sqrtf(s / (float)a.hd + a.eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * inv * gm[e];
+        const float sc = kind == 0 ? a.q_scale : 1.0f;
+        __nv_bfloat162 o2[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int i = c * 4 + e;                                      // the pair's index
+            float co = 1.f, si = 0.f;
+            if (i < a.half && a.cosv) { co = a.cosv[(size_t)t * a.half + i]; si = a.sinv[(size_t)t * a.half + i]; }
+            o2[e] = __floats2bfloat162_rn((v[2 * e] * co - v[2 * e + 1] * si) * sc, (v[2 * e + 1] * co + v[2 * e] * si) * sc);
+        }
+        out = *(const uint4*)o2;
+    }
+    if (kind == 0) {
+        *(uint4*)((__nv_bfloat16*)a.q_out + ((size_t)t * a.nH + j) * a.hd + c * 8) = out;
+        return;
+    }
+    const int head = kind == 1 ? j - a.nH : j - a.nH - a.nKV;
+    const int pos = a.tok_pos[t];
+    const int slot = gl_checked(pos / GL_PAGE, a.max_pages, GL_BAD_POSITION);
+    const int page = gl_checked(a.pages[(size_t)a.tok_seq[t] * a.max_pages + slot], a.n_pages > 0 ? a.n_pages : 0x7fffffff, GL_BAD_PAGE);
+    const size_t at = (((size_t)page * a.nKV + head) * GL_PAGE + (pos % GL_PAGE)) * a.hd + c * 8;
+    *(uint4*)((__nv_bfloat16*)(kind == 1 ? a.k_cache : a.v_cache) + at) = out;
+    if (kind == 1 && a.v_from_k) *(uint4*)((__nv_bfloat16*)a.v_cache + at) = raw;
+}
+
+template <int LPH>
+static int launch_headnorm(const QkvCacheArgs& a, cudaStream_t stream) {
+    const long long heads = a.write_kv ? (a.v_from_k ? a.nH + a.nKV : a.nH + 2 * a.nKV) : a.nH;
+    return gl_launch(qkv_headnorm_bf16_kernel<LPH>, dim3((unsigned)((a.T * heads * LPH + 127) / 128)), dim3(128), 0, stream, 1, a);
+}
+
 GL_API int gl_qkv_cache(const QkvCacheArgs* args, int act_dtype, int cache_dtype, cudaStream_t stream) {
     const QkvCacheArgs& a = *args;
     if (a.T <= 0) return GL_OK;
     if (a.hd <= 0 || a.nH <= 0 || a.nKV <= 0 || 2 * a.half > a.hd) return GL_ERR_SHAPE;
-    if (act_dtype == GL_BF16 && cache_dtype == GL_BF16 && !a.q_gamma && !a.k_gamma && !a.interleaved &&
+    if (a.ld < 0 || (a.ld > 0 && a.ld < (a.nH + (a.v_from_k ? 1 : 2) * a.nKV) * a.hd) || (a.v_from_k && a.ld == 0)) return GL_ERR_SHAPE;
+    const bool aligned = !(((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15);
+    if (act_dtype == GL_BF16 && cache_dtype == GL_BF16 && a.q_gamma && a.k_gamma && !a.q_beta && !a.k_beta && a.norm_rms &&
+        (a.interleaved || a.half == 0) && a.hd % 8 == 0 && a.hd <= 256 && aligned) {
+        QkvCacheArgs b = a;
+        if (b.ld == 0) b.ld = (a.nH + 2 * a.nKV) * a.hd;
+        const int chunks = a.hd / 8;
+        if (b.ld % 8 == 0) {
+            if (chunks <= 4) return launch_headnorm<4>(b, stream);
+            if (chunks <= 8) return launch_headnorm<8>(b, stream);
+            if (chunks <= 16) return launch_headnorm<16>(b, stream);
+            return launch_headnorm<32>(b, stream);
+        }
+    }
+    if (act_dtype == GL_BF16 && cache_dtype == GL_BF16 && !a.q_gamma && !a.k_gamma && !a.interleaved && a.ld == 0 &&
         a.hd % 8 == 0 && a.half % 8 == 0 &&
         !(((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15)) {
         return gl_launch(qkv_cache_bf16_kernel, dim3((unsigned)a.T), dim3(256), 0, stream, 1, a);

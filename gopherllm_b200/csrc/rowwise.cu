@@ -339,6 +339,104 @@ GL_API int gl_norm(const float* x, const int* rows, const float* gamma, const fl
 }
 
 // ---------------------------------------------------------------------------
+// A squashing in place of a norm: out[r, d] = tanh(alpha * x[r, d]) * gamma[d] + beta[d] with one learned alpha (read on
+// the device: a layer's number is a tensor like its vectors).  No statistics, so a row is no unit of work; 32-bit
+// arithmetic, one rounding.  rows picks rows of x as for the norms above.
+// ---------------------------------------------------------------------------
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(256)
+dynamic_tanh_kernel(const float* x, const int* __restrict__ rows, const float* __restrict__ gamma, const float* __restrict__ beta,
+                    const float* __restrict__ alpha, TO* __restrict__ out, long long n, int D) {
+    gl_grid_launch_dependents();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    const long long r = i / D;
+    const int d = (int)(i - r * D);
+    const bool live = i < n;
+    float g[VEC], b[VEC];
+    // (weights: asked for before the wait)
+    if constexpr (VEC == 4) {
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 g4 = live ? *(const float4*)(gamma + d) : zero, b4 = live ? *(const float4*)(beta + d) : zero;
+        g[0] = g4.x; g[1] = g4.y; g[2] = g4.z; g[3] = g4.w;
+        b[0] = b4.x; b[1] = b4.y; b[2] = b4.z; b[3] = b4.w;
+    } else {
+        g[0] = live ? gamma[d] : 0.f;
+        b[0] = live ? beta[d] : 0.f;
+    }
+    const float a = *alpha;
+    gl_grid_wait();
+    if (!live) return;
+    const float* src = x + (size_t)(rows ? rows[r] : r) * D + d;
+    float v[VEC];
+    if constexpr (VEC == 4) {
+        const float4 f = __ldcg((const float4*)src);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+        v[0] = __ldcg(src);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = fmaf(tanhf(a * v[e]), g[e], b[e]);
+    if constexpr (VEC == 4 && sizeof(TO) == 4) {
+        *(float4*)(out + i) = make_float4(v[0], v[1], v[2], v[3]);
+    } else if constexpr (VEC == 4) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(v[0], v[1]), p1 = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 pk;
+        pk.x = *(const unsigned*)&p0; pk.y = *(const unsigned*)&p1;
+        *(uint2*)(out + i) = pk;
+    } else {
+        gl_store(out + i, v[0]);
+    }
+}
+
+template <typename TO>
+static int launch_dynamic_tanh(const float* x, const int* rows, const float* gamma, const float* beta, const float* alpha, TO* out,
+                               int R, int D, cudaStream_t stream) {
+    const long long n = (long long)R * D;
+    if (D % 4 == 0 && !(((uintptr_t)x | (uintptr_t)out | (uintptr_t)gamma | (uintptr_t)beta) & 15))
+        return gl_launch(dynamic_tanh_kernel<TO, 4>, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, stream, 1, x, rows, gamma,
+                         beta, alpha, out, n, D);
+    return gl_launch(dynamic_tanh_kernel<TO, 1>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, x, rows, gamma, beta,
+                     alpha, out, n, D);
+}
+
+GL_API int gl_dynamic_tanh(const float* x, const int* rows, const float* gamma, const float* beta, const float* alpha, void* out,
+                           int out_dtype, int R, int D, cudaStream_t stream) {
+    if (R <= 0) return GL_OK;
+    if (D <= 0 || !gamma || !beta || !alpha) return GL_ERR_SHAPE;
+    if (out_dtype == GL_F32) return launch_dynamic_tanh<float>(x, rows, gamma, beta, alpha, (float*)out, R, D, stream);
+    if (out_dtype == GL_BF16) return launch_dynamic_tanh<__nv_bfloat16>(x, rows, gamma, beta, alpha, (__nv_bfloat16*)out, R, D, stream);
+    return GL_ERR_DTYPE;
+}
+
+// ---------------------------------------------------------------------------
+// out[t, c] *= sigmoid(gate[t, gate_off + c]): a mixer's result gated element by element (where the kernel that made
+// it does not gate it itself).
+// ---------------------------------------------------------------------------
+template <typename TA>
+__global__ void __launch_bounds__(256)
+sigmoid_gate_kernel(TA* x, const TA* gate, long long n, int C, int ld, int off) {
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / C;
+        const float g = gl_load(gate + (size_t)t * ld + off + (i - t * C));
+        gl_store(x + i, gl_load(x + i) / (1.0f + expf(-g)));
+    }
+}
+
+GL_API int gl_sigmoid_gate(void* x, const void* gate, int T, int C, int ld, int off, int act_dtype, cudaStream_t stream) {
+    if (T <= 0) return GL_OK;
+    if (C <= 0 || off < 0 || off + C > ld) return GL_ERR_SHAPE;
+    const long long n = (long long)T * C, want = (n + 255) / 256;
+    const dim3 grid((unsigned)(want > 16384 ? 16384 : want));
+    if (act_dtype == GL_F32) return gl_launch(sigmoid_gate_kernel<float>, grid, dim3(256), 0, stream, 1, (float*)x, (const float*)gate, n, C, ld, off);
+    if (act_dtype == GL_BF16)
+        return gl_launch(sigmoid_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, 1, (__nv_bfloat16*)x, (const __nv_bfloat16*)gate,
+                         n, C, ld, off);
+    return GL_ERR_DTYPE;
+}
+
+// ---------------------------------------------------------------------------
 // Feeding a decode step's choices back on the device: the sampled token becomes
 // the next input, positions and cached lengths move on by one, and the choice is
 // appended to a history so that several steps can run without the host.
@@ -369,12 +467,13 @@ GL_API int gl_advance_decode(int* tokens, int* tok_pos, int* seq_ctx, const int*
 }
 
 // ---------------------------------------------------------------------------
-// Gated feed-forward, between its products: out[t, j] = act(gu[t, j]) * gu[t, F + j], where a row
-// of gu holds the gate's F columns and then the up projection's.  32-bit arithmetic, one rounding.
+// Gated feed-forward, between its products: out[t, j] = act(gu[t, j]) * gu[t, F + j] (or the clipped form,
+// gl_gated), where a row of gu holds the gate's F columns and then the up projection's.  32-bit arithmetic, one
+// rounding.
 // ---------------------------------------------------------------------------
 template <typename TA>
 __global__ void __launch_bounds__(256)
-gated_act_kernel(const TA* gu, TA* __restrict__ out, long long n, int F, int act) {
+gated_act_kernel(const TA* gu, TA* __restrict__ out, long long n, int F, GlGated act) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
@@ -382,13 +481,13 @@ gated_act_kernel(const TA* gu, TA* __restrict__ out, long long n, int F, int act
         const int j = (int)(i - t * F);
         const TA* row = gu + (size_t)t * 2 * F;
         const float g = gl_load(row + j), u = gl_load(row + F + j);
-        gl_store(out + i, gl_activate<true>(g, act) * u);
+        gl_store(out + i, gl_gated<true>(g, u, act));
     }
 }
 
 // bfloat16 rows whose halves are whole 16-byte units: eight columns a thread, 16-byte loads and stores
 __global__ void __launch_bounds__(256)
-gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out, long long n8, int F8, int act) {
+gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out, long long n8, int F8, GlGated act) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n8; i += (long long)gridDim.x * blockDim.x) {
@@ -403,15 +502,17 @@ gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const float2 gf = __bfloat1622float2(g2[e]), uf = __bfloat1622float2(u2[e]);
-            o2[e] = __floats2bfloat162_rn(gl_activate<true>(gf.x, act) * uf.x, gl_activate<true>(gf.y, act) * uf.y);
+            o2[e] = __floats2bfloat162_rn(gl_gated<true>(gf.x, uf.x, act), gl_gated<true>(gf.y, uf.y, act));
         }
         ((uint4*)out)[i] = o;
     }
 }
 
-GL_API int gl_gated_act(const void* gu, void* out, int T, int F, int act, int act_dtype, cudaStream_t stream) {
+GL_API int gl_gated_act(const void* gu, void* out, int T, int F, int act_code, float limit, float slope, float shift,
+                        int act_dtype, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
     if (F <= 0) return GL_ERR_SHAPE;
+    const GlGated act = {act_code, limit, slope, shift};
     const long long n = (long long)T * F;
     if (act_dtype == GL_BF16 && F % 8 == 0 && !(((uintptr_t)gu | (uintptr_t)out) & 15)) {
         const long long n8 = n / 8, want8 = (n8 + 255) / 256;

@@ -340,6 +340,35 @@ def norm(x: torch.Tensor, gamma: torch.Tensor, beta: Optional[torch.Tensor], eps
     return out
 
 
+def dynamic_tanh(x: torch.Tensor, gamma: torch.Tensor, beta: torch.Tensor, alpha: torch.Tensor, out_dtype: torch.dtype,
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """tanh(alpha * x) * gamma + beta of float32 rows, alpha one number on the device ([1]); ``rows`` picks rows of x."""
+    _need(x, "x", torch.float32)
+    D = x.shape[-1]
+    _need(gamma, "gamma", torch.float32, (D,))
+    _need(beta, "beta", torch.float32, (D,))
+    _need(alpha, "alpha", torch.float32, (1,))
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    R = rows.numel() if rows is not None else x.numel() // D
+    out = empty((R, D), out_dtype, x.device)
+    _check(_launch(_lib("rowwise.cu").gl_dynamic_tanh, _ptr(x), _ptr(rows), _ptr(gamma), _ptr(beta), _ptr(alpha), _ptr(out),
+                   c_int(dtype_code(out_dtype)), c_int(R), c_int(D), _stream()), "dynamic_tanh")
+    return out
+
+
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, gate_off: int) -> torch.Tensor:
+    """In place: x[t, c] *= sigmoid(gate[t, gate_off + c])."""
+    _need(x, "x")
+    _need(gate, "gate", x.dtype)
+    T, C = x.shape
+    if gate.shape[0] != T or gate_off < 0 or gate_off + C > gate.shape[1]:
+        raise KernelError(f"sigmoid_gate: columns {gate_off}..{gate_off + C} of rows {tuple(gate.shape)} do not gate {tuple(x.shape)}")
+    _check(_launch(_lib("rowwise.cu").gl_sigmoid_gate, _ptr(x), _ptr(gate), c_int(T), c_int(C), c_int(gate.shape[1]), c_int(gate_off),
+                   c_int(dtype_code(x.dtype)), _stream()), "sigmoid_gate")
+    return x
+
+
 def advance_decode(tokens, tok_pos, seq_ctx, sampled, history, counter) -> None:
     """After a decode step on the device: tokens <- sampled, positions and cached lengths + 1,
     history[counter] <- sampled, counter + 1 (all int32; history is [max_steps, B])."""
@@ -356,9 +385,9 @@ def advance_decode(tokens, tok_pos, seq_ctx, sampled, history, counter) -> None:
               c_int(B), c_int(history.shape[0]), _stream()), "advance_decode")
 
 
-def rope_table(pos: torch.Tensor, inv_freq: torch.Tensor):
+def rope_table(pos: torch.Tensor, inv_freq: torch.Tensor, gain: float = 1.0):
     """cos and sin of float32(pos) * inv_freq, each [T, half] float32.  With float64 frequencies the
-    angle is the 64-bit product pos * inv_freq."""
+    angle is the 64-bit product pos * inv_freq, and both tables are multiplied by ``gain``."""
     _need(pos, "pos", torch.int32)
     T, half = pos.numel(), inv_freq.numel()
     cosv = empty((T, half), torch.float32, pos.device)
@@ -366,10 +395,12 @@ def rope_table(pos: torch.Tensor, inv_freq: torch.Tensor):
     if inv_freq.dtype == torch.float64:
         _need(inv_freq, "inv_freq", torch.float64)
         fn = _lib("qkv_cache.cu").gl_rope_table64
-        _check(_launch(fn, _ptr(pos), _ptr(inv_freq), _ptr(cosv), _ptr(sinv), c_int(T), c_int(half), _stream()),
+        _check(_launch(fn, _ptr(pos), _ptr(inv_freq), _ptr(cosv), _ptr(sinv), c_int(T), c_int(half), ctypes.c_double(gain), _stream()),
                "rope_table")
         return cosv, sinv
     _need(inv_freq, "inv_freq", torch.float32)
+    if gain != 1.0:
+        raise KernelError("rope_table: a factor on the tables comes with 64-bit frequencies")
     fn = _lib("qkv_cache.cu").gl_rope_table
     _check(_launch(fn, _ptr(pos), _ptr(inv_freq), _ptr(cosv), _ptr(sinv), c_int(T), c_int(half), _stream()),
            "rope_table")
@@ -383,7 +414,7 @@ class _QkvCacheArgs(Structure):
                 ("tok_seq", c_void_p), ("tok_pos", c_void_p), ("pages", c_void_p),
                 ("T", c_int), ("nH", c_int), ("nKV", c_int), ("hd", c_int), ("half", c_int),
                 ("max_pages", c_int), ("interleaved", c_int), ("norm_rms", c_int), ("write_kv", c_int),
-                ("eps", c_float), ("q_scale", c_float), ("n_pages", c_int)]
+                ("eps", c_float), ("q_scale", c_float), ("n_pages", c_int), ("ld", c_int), ("v_from_k", c_int)]
 
 
 def qkv_to_cache(qkv: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
@@ -392,16 +423,19 @@ def qkv_to_cache(qkv: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, 
                  cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
                  interleaved: bool = False,
                  q_norm=None, k_norm=None, norm_eps: float = 0.0, norm_rms: bool = False,
-                 write_kv: bool = True) -> None:
+                 write_kv: bool = True, v_from_k: bool = False) -> None:
     """Head norm, rotation and scale of projected rows; q to ``q_out``, k and v into cache pages.
 
-    qkv: [T, (nH + 2 nKV) * hd]; k_cache, v_cache: [pages, nKV, PAGE, hd];
+    qkv: [T, (nH + 2 nKV) * hd], or longer rows that begin so; with ``v_from_k`` the rows hold no v: the
+    values are the key columns as projected, before norm and rotation.  k_cache, v_cache: [pages, nKV, PAGE, hd];
     pages: [B, max_pages] int32; q_norm / k_norm: (gamma, beta or None) or None.
     """
     _need(qkv, "qkv")
     T = qkv.shape[0]
-    width = (num_heads + 2 * num_kv_heads) * head_dim
-    _need(qkv, "qkv", shape=(T, width))
+    width = (num_heads + (1 if v_from_k else 2) * num_kv_heads) * head_dim
+    ld = qkv.shape[1]
+    if ld < width:
+        raise KernelError(f"qkv_to_cache: rows of {ld} columns do not hold {width}")
     _need(q_out, "q_out", qkv.dtype, (T, num_heads * head_dim))
     _need(k_cache, "k_cache")
     _need(v_cache, "v_cache", k_cache.dtype, k_cache.shape)
@@ -431,7 +465,7 @@ def qkv_to_cache(qkv: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, 
                       tok_seq.data_ptr(), tok_pos.data_ptr(), pages.data_ptr(),
                       T, num_heads, num_kv_heads, head_dim, half, pages.shape[-1],
                       1 if interleaved else 0, 1 if norm_rms else 0, 1 if write_kv else 0,
-                      norm_eps, q_scale, k_cache.shape[0])
+                      norm_eps, q_scale, k_cache.shape[0], 0 if ld == width and not v_from_k else ld, 1 if v_from_k else 0)
     fn = _lib("qkv_cache.cu").gl_qkv_cache
     _check(_launch(fn, byref(a), c_int(dtype_code(qkv.dtype)), c_int(dtype_code(k_cache.dtype)), _stream()),
            "qkv_to_cache")
@@ -497,12 +531,17 @@ def attention_prefill(q, out, k_cache, v_cache, seq_qstart, seq_qlen, seq_ctx, p
     _check(_launch(lib.gl_attention_prefill, byref(a), _stream()), "attention_prefill")
 
 
+class _AttnGate(Structure):
+    _fields_ = [("gate", c_void_p), ("ld", c_int), ("off", c_int)]
+
+
 def attention_prefill_tc(q, out, k_cache, v_cache, seq_qstart, seq_qlen, seq_ctx, pages,
                          num_heads: int, num_kv_heads: int, head_dim: int, max_qlen: int,
-                         window: int = 0) -> None:
+                         window: int = 0, gate: Optional[torch.Tensor] = None, gate_off: int = 0) -> None:
     """Causal attention of runs of new tokens over the bfloat16 cache on the 5th-generation
     tensor cores (tcgen05.mma for both products, operands by TMA, scores and partial outputs
-    in tensor memory); head sizes 16..128 in steps of 16."""
+    in tensor memory); head sizes 16..128 in steps of 16.  ``gate`` [T, ld] (ld and gate_off multiples of 8):
+    the result's column c is multiplied by sigmoid(gate[t, gate_off + c]) in the epilogue."""
     if head_dim % 16 or not 16 <= head_dim <= 128:
         raise KernelError(f"tcgen05 prefill attention takes head sizes 16..128 in steps of 16, not {head_dim}")
     if q.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16:
@@ -510,6 +549,12 @@ def attention_prefill_tc(q, out, k_cache, v_cache, seq_qstart, seq_qlen, seq_ctx
     a = _attn_args(q, out, k_cache, v_cache, seq_qstart, seq_qlen, seq_ctx, pages,
                    num_heads, num_kv_heads, head_dim, window, max_qlen, 1.0)
     lib = _lib("attention_prefill_tc.cu", catalog.head_dim_defines(head_dim))
+    if gate is not None:
+        _need(gate, "gate", torch.bfloat16)
+        x = _AttnGate(gate.data_ptr(), gate.shape[1], gate_off)
+        _check(_launch(lib.gl_attention_prefill_tc_gated, byref(a), byref(x), c_int(q.shape[0]), c_int(k_cache.shape[0]), _stream()),
+               "attention_prefill_tc")
+        return
     _check(_launch(lib.gl_attention_prefill_tc, byref(a), c_int(q.shape[0]), c_int(k_cache.shape[0]), _stream()),
            "attention_prefill_tc")
 
@@ -524,6 +569,11 @@ class _DecodeArgs(Structure):
 class _DecodeQkv(Structure):
     _fields_ = [("qkv", c_void_p), ("cosv", c_void_p), ("sinv", c_void_p), ("half", c_int), ("write_kv", c_int),
                 ("q_scale", c_float)]
+
+
+class _DecodeHead(Structure):
+    _fields_ = [("q_gamma", c_void_p), ("k_gamma", c_void_p), ("eps", c_float), ("ld", c_int), ("v_from_k", c_int),
+                ("gate_off", c_int), ("chunks", c_int)]
 
 
 DECODE_MAX_GROUP = 8      # query heads per key/value head the decode kernel takes
@@ -628,11 +678,77 @@ def attention_decode(q, out, k_cache, v_cache, seq_ctx, pages, num_heads: int, n
         _check(_launch(lib.gl_attention_decode_qkv, byref(a), byref(x), _stream()), "attention_decode", launches)
 
 
+def decode_head_chunks(group: int) -> int:
+    """Blocks that share a key/value head's ``group`` query heads in decode attention (each takes up to eight of them)."""
+    return next(n for n in range(1, group + 1) if group % n == 0 and group // n <= DECODE_MAX_GROUP)
+
+
+def decode_takes_head(act_dtype, cache_dtype, head_dim: int, row: int, interleaved: bool) -> bool:
+    """Whether ``attention_decode_head`` takes these types and sizes (rows of ``row`` columns)."""
+    return (act_dtype == torch.bfloat16 and cache_dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
+            and row % 8 == 0 and interleaved)
+
+
+def attention_decode_head(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, seq_ctx, pages,
+                          num_heads: int, num_kv_heads: int, head_dim: int, splits: int, q_gamma: torch.Tensor,
+                          k_gamma: torch.Tensor, eps: float, window: int = 0, cos: Optional[torch.Tensor] = None,
+                          sin: Optional[torch.Tensor] = None, q_scale: float = 1.0, write_kv: bool = True,
+                          v_from_k: bool = False, gate_off: int = -1) -> None:
+    """One query per sequence over the bfloat16 cache, straight from the projection's rows ``qkv`` [B, ld] = [q | k | v |
+    ...] (``v_from_k``: [q | k | ...], the values are the key columns as projected): every head of q and of the new key
+    divided by its root mean square times q_gamma / k_gamma [head_dim], dims 2i and 2i + 1 turned by the tables'
+    angles, queries scaled; the new key and value go to the cache (write_kv).  ``gate_off`` >= 0: column c of the result
+    is multiplied by sigmoid(qkv[b, gate_off + c]).  Up to 8 splits."""
+    B = out.shape[0]
+    _need(qkv, "qkv", torch.bfloat16)
+    ld = qkv.shape[1]
+    group = num_heads // max(1, num_kv_heads)
+    if qkv.shape[0] != B or num_heads % num_kv_heads or ld < (num_heads + (1 if v_from_k else 2) * num_kv_heads) * head_dim:
+        raise KernelError(f"attention_decode_head: rows {tuple(qkv.shape)} do not hold {num_heads} + {num_kv_heads} heads of {head_dim}")
+    if not decode_takes_head(qkv.dtype, k_cache.dtype, head_dim, ld, True) or not 1 <= splits <= 8:
+        raise KernelError("attention_decode_head: head sizes 16..256 in steps of 16, rows of whole 16-byte units, up to 8 splits")
+    _need(out, "out", torch.bfloat16, (B, num_heads * head_dim))
+    _need(k_cache, "k_cache", torch.bfloat16)
+    _need(v_cache, "v_cache", torch.bfloat16, k_cache.shape)
+    if tuple(k_cache.shape[1:]) != (num_kv_heads, PAGE, head_dim):
+        raise KernelError(f"cache pages must be [*, {num_kv_heads}, {PAGE}, {head_dim}], are {tuple(k_cache.shape)}")
+    _need(seq_ctx, "seq_ctx", torch.int32, (B,))
+    _need(pages, "pages", torch.int32)
+    if pages.shape[0] != B:
+        raise KernelError(f"pages has {pages.shape[0]} rows for {B} sequences")
+    for n, g in (("q_gamma", q_gamma), ("k_gamma", k_gamma)):
+        _need(g, n, torch.float32, (head_dim,))
+    half = 0
+    if cos is not None:
+        half = cos.shape[1]
+        _need(cos, "cos", torch.float32, (B, half))
+        _need(sin, "sin", torch.float32, (B, half))
+        if 2 * half > head_dim:
+            raise KernelError(f"rotary dimension {2 * half} exceeds head size {head_dim}")
+    a = _DecodeArgs(None, out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), seq_ctx.data_ptr(), pages.data_ptr(), None, None,
+                    B, num_heads, num_kv_heads, pages.shape[-1], window, splits)
+    x = _DecodeQkv(qkv.data_ptr(), _addr(cos), _addr(sin), half, int(bool(write_kv)), float(q_scale))
+    h = _DecodeHead(q_gamma.data_ptr(), k_gamma.data_ptr(), eps, ld, 1 if v_from_k else 0, gate_off, decode_head_chunks(group))
+    lib = _lib("attention_decode.cu", catalog.head_dim_defines(head_dim))
+    _check(_launch(lib.gl_attention_decode_head, byref(a), byref(x), byref(h), _stream()), "attention_decode")
+
+
 def attention(q, out, k_cache, v_cache, ctx, pages, num_heads: int, num_kv_heads: int,
-              head_dim: int, window: int = 0) -> None:
+              head_dim: int, window: int = 0, gate: Optional[torch.Tensor] = None, gate_off: int = 0) -> None:
     """Attention of a step's queries over the cache with the fastest kernel for the step's
     shape and element type.  ``ctx`` is the step's context (per-sequence starts, lengths,
-    cached lengths on the device; the longest query run and sequence on the host)."""
+    cached lengths on the device; the longest query run and sequence on the host).
+    ``gate`` [T, ld]: column c of the result is multiplied by sigmoid(gate[t, gate_off + c]), in the tcgen05 kernel's
+    epilogue where that kernel runs, else by a pass of its own."""
+    if gate is not None:
+        if (not ctx.is_decode and USE_TCGEN05 and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16
+                and head_dim % 16 == 0 and head_dim <= TC_ATTENTION_MAX_HEAD_DIM and gate.shape[1] % 8 == 0 and gate_off % 8 == 0):
+            attention_prefill_tc(q, out, k_cache, v_cache, ctx.seq_qstart, ctx.seq_qlen, ctx.seq_ctx, pages,
+                                 num_heads, num_kv_heads, head_dim, ctx.max_qlen, window, gate, gate_off)
+            return
+        attention(q, out, k_cache, v_cache, ctx, pages, num_heads, num_kv_heads, head_dim, window)
+        sigmoid_gate(out, gate, gate_off)
+        return
     if (ctx.is_decode and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16
             and head_dim % 16 == 0 and num_heads // num_kv_heads <= DECODE_MAX_GROUP):
         splits = decode_splits(ctx.n_seqs, num_kv_heads, ctx.max_len, q.device, head_dim,
@@ -1490,8 +1606,24 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     return out
 
 
+GATED_CLIPPED = 32       # GL_GATED_CLIPPED
+
+
+def _gated_code(act):
+    """(code, limit, slope, shift) of a gated form: an activation's name (act(gate) * up), or ("clipped", limit, slope,
+    shift): with g = min(gate, limit) and u = clamp(up, -limit, limit), g * sigmoid(slope * g) * (u + shift)."""
+    if isinstance(act, tuple):
+        if len(act) != 4 or act[0] != "clipped":
+            raise KernelError(f"gated form {act!r} unknown")
+        return GATED_CLIPPED, float(act[1]), float(act[2]), float(act[3])
+    if act not in ACTIVATIONS:
+        raise KernelError(f"activation {act!r} unknown")
+    return ACTIVATIONS[act], 0.0, 0.0, 0.0
+
+
 def gated_act(gu: torch.Tensor, act, inner: Optional[int] = None, row_gate: Optional[int] = None) -> torch.Tensor:
-    """act(gate) * up for rows that hold the gate's columns and then the up projection's.  ``inner``: the rows
+    """act(gate) * up (or another gated form, see _gated_code) for rows that hold the gate's columns and then the up
+    projection's.  ``inner``: the rows
     are longer than that, the gate's ``inner`` columns first, the up projection's behind them; ``row_gate``: the
     column of such a row whose sigmoid multiplies the whole row's result."""
     _need(gu, "gu")
@@ -1504,11 +1636,12 @@ def gated_act(gu: torch.Tensor, act, inner: Optional[int] = None, row_gate: Opti
         _check(_launch(fn, _ptr(gu), _ptr(out), c_int(T), c_int(inner), c_int(F2), c_int(-1 if row_gate is None else row_gate),
                        c_int(ACTIVATIONS[act]), c_int(dtype_code(gu.dtype)), _stream()), "gated_act")
         return out
-    if F2 % 2 or act not in ACTIVATIONS:
-        raise KernelError("gated_act: rows of gate and up columns and a known activation expected")
+    if F2 % 2:
+        raise KernelError("gated_act: rows of gate and up columns expected")
+    code, limit, slope, shift = _gated_code(act)
     out = empty((T, F2 // 2), gu.dtype, gu.device)
     fn = _lib("rowwise.cu").gl_gated_act
-    _check(_launch(fn, _ptr(gu), _ptr(out), c_int(T), c_int(F2 // 2), c_int(ACTIVATIONS[act]),
+    _check(_launch(fn, _ptr(gu), _ptr(out), c_int(T), c_int(F2 // 2), c_int(code), c_float(limit), c_float(slope), c_float(shift),
                    c_int(dtype_code(gu.dtype)), _stream()), "gated_act")
     return out
 
@@ -1608,33 +1741,43 @@ MOE_TILE_ROWS = 32
 class _RouteArgs(Structure):
     _fields_ = [("logits", c_void_p), ("ids", c_void_p), ("weights", c_void_p),
                 ("T", c_int), ("E", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int), ("scale", c_float),
-                ("bias", c_void_p), ("softmax_chosen", c_int)]
+                ("bias", c_void_p), ("mode", c_int), ("correction", c_void_p), ("group_largest", c_int)]
 
 
-def _route_mode(E: int, groups: int, bias, softmax_chosen: bool) -> None:
+def _route_mode(E: int, top: int, groups: int, keep: int, bias, softmax_chosen: bool, softmax_all: bool, correction) -> int:
     if bias is not None:
         _need(bias, "bias", torch.float32, (E,))
     if softmax_chosen and groups != 1:
         raise KernelError("moe_route: the softmax over the chosen logits takes one group of experts")
+    if softmax_chosen and softmax_all:
+        raise KernelError("moe_route: one softmax, over the chosen logits or over all")
+    if correction is not None:
+        _need(correction, "correction", torch.float32, (E,))
+        if not softmax_all:
+            raise KernelError("moe_route: a correction of the choice comes with the softmax over all logits")
+    if not (0 < top <= E and groups >= 1 and E % groups == 0 and 1 <= keep <= groups and keep * (E // groups) >= top):
+        raise KernelError(f"moe_route: top {top} of {E} experts in {groups} groups of which {keep} stay is not possible")
+    return 1 if softmax_chosen else 2 if softmax_all else 0
 
 
 def moe_route(logits: torch.Tensor, top: int, groups: int = 1, keep: int = 1, scale: float = 1.0,
-              bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False):
+              bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False, softmax_all: bool = False,
+              correction: Optional[torch.Tensor] = None, group_largest: bool = False):
     """Each token's ``top`` experts by sigmoid(logits) and their weights score / (sum of the chosen scores +
     1e-20) * scale: (ids int32 [T, top], weights float32 [T, top]).  With ``groups`` > 1 the experts form that
     many equal groups of neighbours; a group's score is the sum of its two largest scores and only experts of
     the best ``keep`` groups are chosen from.  ``bias`` [E] float32 is added to the logits first.  With
     ``softmax_chosen`` the ``top`` largest logits are chosen instead and weighted by the softmax over those
-    alone (times scale)."""
+    alone (times scale).  With ``softmax_all`` the scores are the softmax over all logits, the largest score +
+    ``correction`` ([E], may be negative) are chosen, and the weights are the scores themselves (times scale), not
+    renormalised.  ``group_largest``: a group's score is its largest score (with the correction)."""
     _need(logits, "logits", torch.float32)
     T, E = logits.shape
-    _route_mode(E, groups, bias, softmax_chosen)
-    if not (0 < top <= E and groups >= 1 and E % groups == 0 and 1 <= keep <= groups and keep * (E // groups) >= top):
-        raise KernelError(f"moe_route: top {top} of {E} experts in {groups} groups of which {keep} stay is not possible")
+    mode = _route_mode(E, top, groups, keep, bias, softmax_chosen, softmax_all, correction)
     ids = empty((T, top), torch.int32, logits.device)
     weights = empty((T, top), torch.float32, logits.device)
     a = _RouteArgs(logits.data_ptr(), ids.data_ptr(), weights.data_ptr(), T, E, top, groups, keep, scale, _addr(bias),
-                   1 if softmax_chosen else 0)
+                   mode, _addr(correction), 1 if group_largest else 0)
     _check(_launch(_lib("moe.cu").gl_moe_route, byref(a), _stream()), "moe_route")
     return ids, weights
 
@@ -1645,11 +1788,12 @@ class _RouteFromArgs(Structure):
     _fields_ = [("x", c_void_p), ("w", c_void_p), ("K", c_int),
                 ("logits", c_void_p), ("ids", c_void_p), ("weights", c_void_p),
                 ("T", c_int), ("E", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int), ("scale", c_float),
-                ("bias", c_void_p), ("softmax_chosen", c_int)]
+                ("bias", c_void_p), ("mode", c_int), ("correction", c_void_p), ("group_largest", c_int)]
 
 
 def moe_route_from(x: torch.Tensor, w_router: torch.Tensor, top: int, groups: int = 1, keep: int = 1, scale: float = 1.0,
-                   bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False):
+                   bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False, softmax_all: bool = False,
+                   correction: Optional[torch.Tensor] = None, group_largest: bool = False):
     """``moe_route`` of the logits x . w_router^T ([T, K] in the activation type, [E, K] float32) in one kernel:
     a token's logits are sums over k in an order of their own, whatever else is in the step.  Inputs too wide
     for a block's shared memory take the plain product and ``moe_route``."""
@@ -1659,15 +1803,14 @@ def moe_route_from(x: torch.Tensor, w_router: torch.Tensor, top: int, groups: in
     E = w_router.shape[0]
     if w_router.shape[1] != K:
         raise KernelError(f"moe_route_from: router {tuple(w_router.shape)} does not fit x {tuple(x.shape)}")
-    _route_mode(E, groups, bias, softmax_chosen)
-    if (E + groups + K) * 4 > 48 * 1024:
-        return moe_route(gemm_simt(x, w_router, out_dtype=torch.float32), top, groups, keep, scale, bias, softmax_chosen)
-    if not (0 < top <= E and groups >= 1 and E % groups == 0 and 1 <= keep <= groups and keep * (E // groups) >= top):
-        raise KernelError(f"moe_route: top {top} of {E} experts in {groups} groups of which {keep} stay is not possible")
+    mode = _route_mode(E, top, groups, keep, bias, softmax_chosen, softmax_all, correction)
+    if (2 * E + groups + K) * 4 > 48 * 1024:
+        return moe_route(gemm_simt(x, w_router, out_dtype=torch.float32), top, groups, keep, scale, bias, softmax_chosen,
+                         softmax_all, correction, group_largest)
     ids = empty((T, top), torch.int32, x.device)
     weights = empty((T, top), torch.float32, x.device)
     a = _RouteFromArgs(x.data_ptr(), w_router.data_ptr(), K, None, ids.data_ptr(), weights.data_ptr(), T, E, top, groups,
-                       keep, scale, _addr(bias), 1 if softmax_chosen else 0)
+                       keep, scale, _addr(bias), mode, _addr(correction), 1 if group_largest else 0)
     _check(_launch(_lib("moe.cu").gl_moe_route_from, byref(a), c_int(dtype_code(x.dtype)), _stream()), "moe_route")
     return ids, weights
 
@@ -1680,7 +1823,8 @@ class _PlanArgs(Structure):
 class _ExpertArgs(Structure):
     _fields_ = [("x", c_void_p), ("w", c_void_p), ("out", c_void_p), ("order", c_void_p), ("tile_expert", c_void_p),
                 ("tile_start", c_void_p), ("tile_rows", c_void_p), ("n_tiles", c_void_p), ("weights", c_void_p),
-                ("A", c_int), ("N", c_int), ("K", c_int), ("top", c_int), ("max_tiles", c_int), ("E", c_int)]
+                ("A", c_int), ("N", c_int), ("K", c_int), ("top", c_int), ("max_tiles", c_int), ("E", c_int),
+                ("act", c_int), ("limit", c_float), ("slope", c_float), ("shift", c_float)]
 
 
 class _PadPlanArgs(Structure):
@@ -1695,9 +1839,10 @@ USE_MOE_TC = True        # bfloat16 experts on the tensor cores (False: the CUDA
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, add: Optional[torch.Tensor] = None,
-                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, act="silu") -> torch.Tensor:
     """out[t] = sum_k weights[t, k] * down_e(silu(gate_e(x[t])) * up_e(x[t])) + add[t], e = ids[t, k]; float32
-    [T, hidden].  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
+    [T, hidden].  ``act``: another gated form in silu's place (see gated_act).  A choice e >= E is the identity: its
+    part is weights[t, k] * x[t], and it takes no part in the products.  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
     The step's (token, choice) pairs are sorted by expert on the device and cut into tiles of rows; the grids
     cover the most tiles any choice can make, so nothing depends on the host knowing what the router chose.
     Which kernels run depends on the step's size alone: up to MOE_ROWS_KERNEL_PER_EXPERT pairs an expert on
@@ -1720,6 +1865,9 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     hidden = w_down.shape[1]
     if Kw != K or F2 % 2 or tuple(w_down.shape) != (E, hidden, F) or tuple(ids.shape) != (T, top):
         raise KernelError(f"moe_experts: weights {tuple(w_gate_up.shape)} / {tuple(w_down.shape)} do not fit x {tuple(x.shape)}")
+    if hidden != K:
+        raise KernelError("moe_experts: the experts' inputs and outputs have one width (a choice may be the input itself)")
+    code, limit, slope, shift = _gated_code(act)
     if add is not None:
         _need(add, "add", torch.float32, (T, hidden))
     if out is None:
@@ -1742,12 +1890,12 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         _check(_launch(lib.gl_moe_gather_rows, _ptr(x), _ptr(order), _ptr(xs), c_int(tiles * 128), c_int(K), c_int(top),
                        _stream()), "moe_gather_rows")
         gu = gemm_tcgen05_grouped(xs, w_gate_up, tile_expert, torch.bfloat16)
-        h = gated_act(gu, "silu")
+        h = gated_act(gu, act)
         y = gemm_tcgen05_grouped(h, w_down, tile_expert, torch.float32)
         if late_add is not None:
             add = late_add()
             _need(add, "add", torch.float32, (T, hidden))
-        _check(_launch(lib.gl_moe_combine_placed, _ptr(y), _ptr(place), _ptr(weights), _ptr(add), _ptr(out), c_int(T),
+        _check(_launch(lib.gl_moe_combine_placed, _ptr(y), _ptr(place), _ptr(weights), _ptr(x), _ptr(add), _ptr(out), c_int(T),
                        c_int(hidden), c_int(top), _stream()), "moe_combine")
         return out
     max_tiles = -(-A // MOE_TILE_ROWS) + min(E, A)
@@ -1762,16 +1910,17 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     y = empty((A, hidden), torch.float32, dev)
     xd, wd = c_int(dtype_code(x.dtype)), c_int(dtype_code(w_gate_up.dtype))
     g = _ExpertArgs(x.data_ptr(), w_gate_up.data_ptr(), h.data_ptr(), order.data_ptr(), tile_expert.data_ptr(),
-                    tile_start.data_ptr(), tile_rows.data_ptr(), n_tiles.data_ptr(), None, A, F, K, top, max_tiles, E)
+                    tile_start.data_ptr(), tile_rows.data_ptr(), n_tiles.data_ptr(), None, A, F, K, top, max_tiles, E, code, limit, slope, shift)
     _check(_launch(lib.gl_moe_gate_up if USE_MOE_TC else lib.gl_moe_gate_up_simt, byref(g), xd, wd, _stream()), "moe_gate_up")
     d = _ExpertArgs(h.data_ptr(), w_down.data_ptr(), y.data_ptr(), order.data_ptr(), tile_expert.data_ptr(),
                     tile_start.data_ptr(), tile_rows.data_ptr(), n_tiles.data_ptr(), weights.data_ptr(), A, hidden, F, top,
-                    max_tiles, E)
+                    max_tiles, E, 0, 0.0, 0.0, 0.0)
     _check(_launch(lib.gl_moe_down if USE_MOE_TC else lib.gl_moe_down_simt, byref(d), xd, wd, _stream()), "moe_down")
     if late_add is not None:
         add = late_add()
         _need(add, "add", torch.float32, (T, hidden))
-    _check(_launch(lib.gl_moe_combine, _ptr(y), _ptr(add), _ptr(out), c_int(T), c_int(hidden), c_int(top), _stream()),
+    _check(_launch(lib.gl_moe_combine, _ptr(y), _ptr(ids), _ptr(weights), _ptr(x), xd, _ptr(add), _ptr(out), c_int(T), c_int(hidden),
+                   c_int(top), c_int(E), _stream()),
            "moe_combine")
     return out
 

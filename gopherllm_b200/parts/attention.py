@@ -15,7 +15,11 @@ class Attention(Mixer):
     reference's fused matrix is, model.go:2222-2227), optional per-head norm of
     q and k, position encoding, query scale, cache write, attention over the
     cache, output projection.  Grouped-query attention when num_kv_heads <
-    num_heads (query head h reads group h / (nH/nKV), model.go:2828)."""
+    num_heads (query head h reads group h / (nH/nKV), model.go:2828).
+    Options, off by default.  ``values`` = "keys": the values are the keys as projected, before norm and position
+    encoding; there is no value projection.  ``gate``: the result is multiplied, element by element, by sigmoid(W_g x)
+    ("g.weight" [heads * head size, hidden]) before the output projection; the gate's rows ride in the fused product,
+    behind q, k and v."""
 
     deferred_add = True
     capturable = True
@@ -27,6 +31,13 @@ class Attention(Mixer):
         if spec.head_dim > 256:
             raise ValueError(f"head size {spec.head_dim} exceeds what the attention kernels take (256)")
         self.spec = spec
+        values = spec.option("values", "projected")
+        if values not in ("projected", "keys"):
+            raise ValueError(f"attention: values {values!r} are neither projected nor keys")
+        self.v_from_k = values == "keys"
+        self.gate = bool(spec.option("gate", False))
+        if spec.value_dim not in (0, spec.head_dim):
+            raise ValueError(f"attention: values of size {spec.value_dim} beside keys of size {spec.head_dim}")
         self.position = build_position(spec.position)
         self.q_norm = build_norm(spec.qk_norm) if spec.qk_norm else None
         self.k_norm = build_norm(spec.qk_norm) if spec.qk_norm else None
@@ -43,6 +54,12 @@ class Attention(Mixer):
                       "k.bias": ParamSpec((kv,), "vector", "bias"),
                       "v.bias": ParamSpec((kv,), "vector", "bias"),
                       "out.bias": ParamSpec((s.hidden,), "vector", "bias")})
+        if self.gate:
+            p["g.weight"] = ParamSpec((q, s.hidden))
+            if s.bias:
+                p["g.bias"] = ParamSpec((q,), "vector", "bias")
+        if self.v_from_k:
+            p = {k: v for k, v in p.items() if k not in ("v.weight", "v.bias")}
         if self.q_norm is not None:
             for name, n in (("q_norm", self.q_norm), ("k_norm", self.k_norm)):
                 for k, v in n.parameters().items():
@@ -50,13 +67,20 @@ class Attention(Mixer):
         return p
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
-        ws = [t["q.weight"], t["k.weight"], t["v.weight"]]
+        names = ["q", "k"] + ([] if self.v_from_k else ["v"]) + (["g"] if self.gate else [])
+        ws = [t[n + ".weight"] for n in names]
         if len({w.dtype for w in ws}) > 1:           # mixed storage: widen to the widest
             ws = [w.float() for w in ws]
+        pad = -sum(w.shape[0] for w in ws) % 8 if self.v_from_k or self.gate else 0      # rows of whole 16-byte units
+        if pad:
+            ws.append(torch.zeros((pad, ws[0].shape[1]), dtype=ws[0].dtype, device=ws[0].device))
         self.w_qkv = torch.cat(ws, dim=0).contiguous()
         self.w_out = t["out.weight"]
         if self.spec.bias:
-            self.b_qkv = torch.cat([t["q.bias"], t["k.bias"], t["v.bias"]]).contiguous()
+            bs = [t[n + ".bias"] for n in names]
+            if pad:
+                bs.append(torch.zeros(pad, dtype=bs[0].dtype, device=bs[0].device))
+            self.b_qkv = torch.cat(bs).contiguous()
             self.b_out = t["out.bias"]
         if self.q_norm is not None:
             self.q_norm.load({k[len("q_norm."):]: v for k, v in t.items() if k.startswith("q_norm.")})
@@ -83,7 +107,7 @@ class Attention(Mixer):
         return [("qkv", self.w_qkv, self.b_qkv, None), ("out", self.w_out, self.b_out, None)]
 
     def decode_fusable(self, ctx, cache):
-        if not ctx.is_decode or cache is None:
+        if not ctx.is_decode or cache is None or self.v_from_k or self.gate:
             return None
         s = self.spec
         tables = self.position.tables(ctx)
@@ -104,13 +128,26 @@ class Attention(Mixer):
         cos, sin = tables if tables is not None else (None, None)
         pages = ctx.pages[cache.group]
         group = s.num_heads // s.num_kv_heads
-        if (ctx.is_decode and group <= ops.DECODE_MAX_GROUP
+        gate_off = (s.num_heads + (1 if self.v_from_k else 2) * s.num_kv_heads) * s.head_dim if self.gate else -1
+        span = ctx.max_len if s.window <= 0 else min(ctx.max_len, s.window + ops.PAGE)      # positions a token's keys can lie on
+        if (ctx.is_decode and self.q_norm is not None and self.q_norm.rms and not s.qk_norm.bias
+                and ops.decode_takes_head(qkv.dtype, cache.k.dtype, s.head_dim, qkv.shape[1],
+                                          s.position.interleaved or cos is None)):
+            # one token a sequence: head norm, rotation, cache write, attention and gate in one kernel
+            o = ops.empty((T, s.num_heads * s.head_dim), ctx.act_dtype, xn.device)
+            chunks = ops.decode_head_chunks(group)
+            splits = ops.decode_splits(ctx.n_seqs, s.num_kv_heads * chunks, span, xn.device, s.head_dim, group // chunks)
+            ops.attention_decode_head(qkv, o, cache.k, cache.v, ctx.seq_ctx, pages, s.num_heads, s.num_kv_heads, s.head_dim,
+                                      splits, self.q_norm.weight, self.k_norm.weight, s.qk_norm.eps, s.window, cos, sin,
+                                      s.q_scale, cache.writes, self.v_from_k, gate_off)
+            return o, self.w_out, self.b_out
+        if (ctx.is_decode and not self.v_from_k and not self.gate and group <= ops.DECODE_MAX_GROUP
                 and ops.decode_takes_qkv(qkv.dtype, cache.k.dtype, s.head_dim, 0 if cos is None else cos.shape[1],
                                          s.position.interleaved, self.q_norm is not None)):
             # one token a sequence: attention reads the projection's output itself (rotation, query scale
             # and the cache write happen inside it), one kernel less between two products
             o = ops.empty((T, s.num_heads * s.head_dim), ctx.act_dtype, xn.device)
-            splits = ops.decode_splits(ctx.n_seqs, s.num_kv_heads, ctx.max_len, xn.device, s.head_dim, group)
+            splits = ops.decode_splits(ctx.n_seqs, s.num_kv_heads, span, xn.device, s.head_dim, group)
             ops.attention_decode(None, o, cache.k, cache.v, ctx.seq_ctx, pages, s.num_heads, s.num_kv_heads,
                                  s.head_dim, splits, s.window, qkv=qkv, cos=cos, sin=sin, q_scale=s.q_scale,
                                  write_kv=cache.writes)
@@ -124,12 +161,11 @@ class Attention(Mixer):
         ops.qkv_to_cache(qkv, q, cache.k, cache.v, ctx.tok_seq, ctx.tok_pos, pages,
                          s.num_heads, s.num_kv_heads, s.head_dim, s.q_scale, cos, sin,
                          interleaved=s.position.interleaved, q_norm=qn, k_norm=kn,
-                         norm_eps=eps, norm_rms=rms, write_kv=cache.writes)
+                         norm_eps=eps, norm_rms=rms, write_kv=cache.writes, v_from_k=self.v_from_k)
         o = ops.empty(q.shape, q.dtype, q.device)
         ops.attention(q, o, cache.k, cache.v, ctx, pages, s.num_heads, s.num_kv_heads,
-                      s.head_dim, window=s.window)
+                      s.head_dim, window=s.window, gate=qkv if self.gate else None, gate_off=gate_off)
         return o, self.w_out, self.b_out
-
 
 
 class MixedHeadAttention(Mixer):

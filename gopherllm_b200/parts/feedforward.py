@@ -138,8 +138,15 @@ class MixtureOfExperts(FeedForward):
     alone (one group); ``router_bias``: a learned vector is added to the logits.  ``shared_gate``: the shared expert's
     output is multiplied, token by token, by sigmoid(w_sg . x) ("shared.sg.weight" [1, hidden]); the row rides in the
     shared expert's first product and the share is applied before its last product, which is linear.
+    With ``weights`` = "softmax_all" the scores are the softmax over all logits and the chosen experts count by their
+    scores as they are (times router_scale); ``correction``: a learned vector that joins the scores for the choice
+    (groups included) but not the weights.  ``group_by`` = "largest": a group's score is its largest.
+    ``identity`` n: the router has n outputs behind the experts' that stand for the input itself: such a choice adds
+    its weight times the token's input and has no tensors.  Activation "clipped" (options ``limit``, ``slope``, ``shift``): an
+    expert is down(g sigmoid(slope g) (u + shift)) with g = min(gate(x), limit), u = clamp(up(x), -limit, limit).
     Options: ``experts``, ``top``, ``groups``, ``keep``, ``router_scale``, ``shared``, ``router``, ``vocab``,
-    ``weights``, ``router_bias``, ``shared_gate``; ``intermediate`` is an expert's inner size."""
+    ``weights``, ``router_bias``, ``shared_gate``, ``correction``, ``group_by``, ``identity``, ``limit``, ``slope``,
+    ``shift``; ``intermediate`` is an expert's inner size."""
     capturable = True
     launches_only = True
 
@@ -156,8 +163,19 @@ class MixtureOfExperts(FeedForward):
         self.weights_by = str(spec.option("weights", "scores"))
         self.router_bias = bool(spec.option("router_bias", False))
         self.shared_gate = bool(spec.option("shared_gate", False))
-        if self.weights_by not in ("scores", "softmax_chosen"):
-            raise ValueError(f"moe: weights {self.weights_by!r} are neither scores nor softmax_chosen")
+        if self.weights_by not in ("scores", "softmax_chosen", "softmax_all"):
+            raise ValueError(f"moe: weights {self.weights_by!r} are none of scores, softmax_chosen, softmax_all")
+        self.identity = int(spec.option("identity", 0))
+        self.outputs = self.E + self.identity            # of the router
+        self.has_correction = bool(spec.option("correction", False))
+        group_by = str(spec.option("group_by", "two_largest"))
+        if group_by not in ("two_largest", "largest"):
+            raise ValueError(f"moe: groups are scored by their two_largest or their largest score, not {group_by!r}")
+        self.group_largest = group_by == "largest"
+        if self.has_correction and self.weights_by != "softmax_all":
+            raise ValueError("moe: a correction of the choice comes with weights softmax_all")
+        if self.identity < 0 or (self.identity and self.router == "table"):
+            raise ValueError("moe: identity experts are outputs of a router")
         if self.router == "table" and (self.weights_by != "scores" or self.router_bias):
             raise ValueError("moe: a table of experts has neither logits nor a bias")
         if self.weights_by == "softmax_chosen" and self.groups != 1:
@@ -166,23 +184,30 @@ class MixtureOfExperts(FeedForward):
             raise ValueError("moe: a gate on the shared expert needs a shared expert")
         if self.router == "table" and self.vocab < 1:
             raise ValueError("moe: a table of experts by token id needs the vocabulary's size")
-        if spec.activation != "silu":
-            raise ValueError("the experts' activation is silu")
-        if not (0 < self.top <= self.E and self.groups >= 1 and self.E % self.groups == 0
-                and 1 <= self.keep <= self.groups and self.keep * (self.E // self.groups) >= self.top):
-            raise ValueError(f"moe: top {self.top} of {self.E} experts in {self.groups} groups of which "
+        if spec.activation not in ("silu", "clipped"):
+            raise ValueError("the experts' activation is silu or clipped")
+        self.act = "silu"
+        if spec.activation == "clipped":
+            if self.shared:
+                raise ValueError("moe: a shared expert has the activation silu")
+            self.act = ("clipped", float(spec.option("limit")), float(spec.option("slope", 1.0)), float(spec.option("shift", 0.0)))
+        if not (0 < self.top <= self.outputs and self.groups >= 1 and self.outputs % self.groups == 0
+                and 1 <= self.keep <= self.groups and self.keep * (self.outputs // self.groups) >= self.top):
+            raise ValueError(f"moe: top {self.top} of {self.outputs} experts in {self.groups} groups of which "
                              f"{self.keep} stay is not possible")
         self.w_router = self.w_router_16 = self.w_gu = self.w_down = self.ws_gu = self.ws_down = self.table = None
-        self.b_router = None
+        self.b_router = self.correction = None
 
     def parameters(self) -> Dict[str, ParamSpec]:
         s, F = self.spec, self.spec.intermediate
         if self.router == "table":
             p = {"table": ParamSpec((self.vocab, self.top), "table_int", f"distinct:{self.E}")}
         else:
-            p = {"router.weight": ParamSpec((self.E, s.hidden), "vector", "wide")}
+            p = {"router.weight": ParamSpec((self.outputs, s.hidden), "vector", "wide")}
             if self.router_bias:
-                p["router.bias"] = ParamSpec((self.E,), "vector", "bias")
+                p["router.bias"] = ParamSpec((self.outputs,), "vector", "bias")
+            if self.has_correction:
+                p["correction"] = ParamSpec((self.outputs,), "vector", "bias")
         for e in range(self.E):
             p[f"e{e}.gate.weight"] = ParamSpec((F, s.hidden))
             p[f"e{e}.up.weight"] = ParamSpec((F, s.hidden))
@@ -202,7 +227,7 @@ class MixtureOfExperts(FeedForward):
                 raise ValueError(f"moe: the table names experts outside 0..{self.E - 1}")
         else:
             self.w_router = t["router.weight"]
-            self.b_router = t.get("router.bias")
+            self.b_router, self.correction = t.get("router.bias"), t.get("correction")
             # Router weights whose values bfloat16 holds exactly (a 16-bit checkpoint's are) may go through the
             # tensor cores: the products are then exact and the sums 32-bit, which is what "32-bit logits" asks for.
             as16 = self.w_router.to(torch.bfloat16)
@@ -211,7 +236,7 @@ class MixtureOfExperts(FeedForward):
         if len({m.dtype for m in mats}) > 1:
             t = dict(t)
             for k in list(t):
-                if k not in ("router.weight", "router.bias", "table"):
+                if k not in ("router.weight", "router.bias", "correction", "table"):
                     t[k] = t[k].float()
         # every expert's gate rows, then its up rows: [E, 2F, hidden]; the down weights [E, hidden, F]
         self.w_gu = torch.stack([torch.cat([t[f"e{e}.gate.weight"], t[f"e{e}.up.weight"]], 0)
@@ -238,12 +263,13 @@ class MixtureOfExperts(FeedForward):
         """(experts int32 [T, top], weights float32 [T, top]) of the step's tokens."""
         if self.router == "table":
             return ops.moe_route_table(ctx.tokens, self.table, self.E)
+        how = dict(groups=self.groups, keep=self.keep, scale=self.scale, bias=self.b_router,
+                   softmax_chosen=self.weights_by == "softmax_chosen", softmax_all=self.weights_by == "softmax_all",
+                   correction=self.correction, group_largest=self.group_largest)
         if xn.dtype == torch.bfloat16 and self.w_router_16 is not None and xn.shape[1] % 8 == 0:
             logits = ops.linear(xn, self.w_router_16, None, out_dtype=torch.float32)
-            return ops.moe_route(logits, self.top, self.groups, self.keep, self.scale, self.b_router,
-                                 self.weights_by == "softmax_chosen")
-        return ops.moe_route_from(xn, self.w_router, self.top, self.groups, self.keep, self.scale, self.b_router,
-                                  self.weights_by == "softmax_chosen")
+            return ops.moe_route(logits, self.top, **how)
+        return ops.moe_route_from(xn, self.w_router, self.top, **how)
 
     def forward(self, xn, ctx, add: Sequence[torch.Tensor], out=None) -> torch.Tensor:
         if len(add) > (2 if self.shared else 1):
@@ -270,9 +296,9 @@ class MixtureOfExperts(FeedForward):
                 return ys
 
             ids, weights = self.route(xn, ctx)
-            return ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=shared, out=out)
+            return ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=shared, out=out, act=self.act)
         ids, weights = self.route(xn, ctx)
-        out = ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=add[0] if len(add) > 0 else None, out=out)
+        out = ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=add[0] if len(add) > 0 else None, out=out, act=self.act)
         if self.shared:
             gu = ops.linear(xn, self.ws_gu, None, out_dtype=ctx.act_dtype)
             hs = (ops.gated_act(gu, "silu", inner=self.shared, row_gate=2 * self.shared) if self.shared_gate

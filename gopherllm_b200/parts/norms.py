@@ -1,4 +1,4 @@
-"""Normalisation parts: LayerNorm and RMSNorm over the last axis."""
+"""Normalisation parts: LayerNorm and RMSNorm over the last axis, and a squashing that stands in a norm's place."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -50,5 +50,27 @@ class RMSNorm(LayerNorm):
     rms = True
 
 
+class DynamicTanh(Norm):
+    """y = tanh(alpha * x) * weight + bias with one learned alpha: no statistics over the row (``eps`` is not used)."""
+    capturable = True
+    launches_only = True
+
+    def __init__(self, spec: NormSpec):
+        self.spec = spec
+        self.weight = self.bias = self.alpha = None
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.spec.dim,), "vector", "gamma"), "bias": ParamSpec((self.spec.dim,), "vector", "beta"),
+                "alpha": ParamSpec((), "vector", "gamma")}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight, self.bias = tensors["weight"], tensors["bias"]
+        self.alpha = tensors["alpha"].reshape(1).contiguous()
+
+    def forward(self, x, out_dtype, rows=None):
+        return ops.dynamic_tanh(x, self.weight, self.bias, self.alpha, out_dtype, rows=rows)
+
+
 register_norm("layernorm", LayerNorm)
 register_norm("rmsnorm", RMSNorm)
+register_norm("dynamic_tanh", DynamicTanh)

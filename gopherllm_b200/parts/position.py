@@ -1,6 +1,8 @@
 """Position encodings a mixer can be given."""
 from __future__ import annotations
 
+import math
+
 import numpy as np
 import torch
 
@@ -20,11 +22,28 @@ def rope_inverse_frequencies(rotary_dim: int, theta: float) -> np.ndarray:
     return (np.float32(1.0) / base).astype(np.float32)
 
 
+def stretched_frequencies(rotary_dim: int, theta: float, factor: float, original: float, fast: float, slow: float):
+    """(64-bit frequencies [rotary_dim / 2], factor on the tables) of a rotation stretched to longer contexts the YaRN way:
+    pairs that turn more than ``fast`` times over ``original`` positions keep theta^(-2i/d), pairs that turn less than
+    ``slow`` times turn ``factor`` times slower, a linear ramp over the pairs between; cosine and sine are multiplied by
+    0.1 ln(factor) + 1."""
+    half = rotary_dim // 2
+    inv = np.float64(theta) ** (-2.0 * np.arange(half, dtype=np.float64) / rotary_dim)
+
+    def pair_of(turns):          # the pair (a real number) that turns so often over the original length
+        return rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo = max(math.floor(pair_of(fast)), 0)
+    hi = min(math.ceil(pair_of(slow)), rotary_dim - 1)
+    ramp = np.clip((np.arange(half, dtype=np.float64) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return inv / factor * ramp + inv * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class Rope(PositionEncoding):
     """Rotary embedding over the first ``rotary_dim`` dims of a head.  The
     angle float32(pos) * inv[i] is a 32-bit product; sine and cosine are taken
     in 64-bit (prepareRopeScratch, model.go:3041-3046).  The tables depend on
-    the step's positions only, so every layer of a step shares them."""
+    the step's positions only, so every layer of a step shares them.  Option ``exact_angles``: frequencies and angles
+    in 64-bit; with it option ``yarn`` = (factor, original, fast, slow): see stretched_frequencies."""
     capturable = True
     launches_only = True
 
@@ -33,14 +52,20 @@ class Rope(PositionEncoding):
             raise ValueError(f"rotary dimension {spec.rotary_dim} must be even")
         self.spec = spec
         self._inv = None
+        self._gain = 1.0
+        if spec.option("yarn") is not None and not spec.option("exact_angles", False):
+            raise ValueError("stretched frequencies come with exact angles")
 
     def tables(self, ctx):
         exact = bool(self.spec.option("exact_angles", False))
-        key = ("rope", self.spec.rotary_dim, float(self.spec.theta), exact)
+        yarn = self.spec.option("yarn")
+        key = ("rope", self.spec.rotary_dim, float(self.spec.theta), exact, yarn)
         hit = ctx.scratch.get(key)
         if hit is None:
             if self._inv is None or self._inv.device != ctx.device:
-                if exact:
+                if yarn is not None:
+                    inv, self._gain = stretched_frequencies(self.spec.rotary_dim, float(self.spec.theta), *yarn)
+                elif exact:
                     # frequencies theta^(-2i/d) and the angles pos * frequency in 64-bit: a table entry is then
                     # the rounded cosine of the true angle at any position (a 32-bit angle is off by up to
                     # position * 2^-24 radians, which a sharp head sees a thousand positions on)
@@ -49,7 +74,7 @@ class Rope(PositionEncoding):
                 else:
                     inv = rope_inverse_frequencies(self.spec.rotary_dim, self.spec.theta)
                 self._inv = torch.from_numpy(inv).to(ctx.device)
-            hit = ops.rope_table(ctx.tok_pos, self._inv)
+            hit = ops.rope_table(ctx.tok_pos, self._inv, self._gain)
             ctx.scratch[key] = hit
         return hit
 
