@@ -7,6 +7,7 @@
     python bench.py --design gozolix         the same for a Gozolix model, beside a Vopedra model of equal width and depth
     python bench.py --design lilupel         the same for a Lilupel model, beside a Vopedra model of equal width and depth
     python bench.py --design darusun         the same for a Darusun model, beside a Gozolix model of equal width and depth
+    python bench.py --design dibedra         the same for a Dibedra model, beside a Gozolix and a Phi model of equal width and depth
     python bench.py --design vopedra         prefill and decode of a Vopedra model at a few layer sizes beside a
                                              Phi model of equal width, depth and feed-forward weights
 
@@ -120,7 +121,7 @@ def main():
     ap.add_argument("--sections", default="decode,e2e,prefill,points",
                     help="which measurements to run (for profiling a part): decode,e2e,prefill,points")
     ap.add_argument("--model", default="phi-2", choices=sorted(MODELS), help="whose layer sizes to run")
-    ap.add_argument("--design", default=None, choices=["vopedra", "gozolix", "lilupel", "darusun"],
+    ap.add_argument("--design", default=None, choices=["vopedra", "gozolix", "lilupel", "darusun", "dibedra"],
                     help="instead: prefill and decode rates of another design at a few layer sizes, beside the Phi "
                          "model of equal width and depth")
     ap.add_argument("--ragged", action="store_true",
@@ -150,7 +151,7 @@ def main():
 
     if args.design == "vopedra":
         return design_vopedra(args)
-    if args.design in ("gozolix", "lilupel", "darusun"):
+    if args.design in ("gozolix", "lilupel", "darusun", "dibedra"):
         return design_vopedra(args, design=args.design)
     pk, pk_src = peaks()
     label, sizes, weight_seed = MODELS[args.model]
@@ -406,12 +407,33 @@ def darusun_sizes(width, heads, ff):
             "initializer_range": 0.02, "layers": five + second}
 
 
+def dibedra_sizes(width, heads, ff):
+    """A Dibedra model whose layers resemble a real model's at this width, ten layer runs: a windowed attention (512
+    positions, a quarter as many key/value heads as query heads) beside a dense feed-forward, beside a mixture of 32
+    experts and 8 identities (4 a token, out of 4 of 8 groups), beside another mixture, that layer's weights once more, and
+    beside a dense feed-forward; twice.  A token meets about as many feed-forward weights in every layer as in the
+    other designs."""
+    hd = width // heads
+    attn = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": 512},
+            "rot": {"dims": hd, "base": 100000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 30.0, "slow": 2.0}}}
+    dense = {"kind": "dense", "ff": (3 * ff // 2) // 64 * 64}
+    moe = {"kind": "moe", "expert": {"ff": max(64, ff // 4 // 64 * 64), "limit": 7.0},
+           "router": {"experts": 32, "top": 4, "identity": 8, "groups": {"count": 8, "keep": 4}}}
+    five = [{"type": "attention", "mixer": attn, "mlp": f} for f in (dense, moe, moe, moe, dense)]
+    five[3]["weights_of"] = 2
+    second = json.loads(json.dumps(five))
+    second[3]["weights_of"] = 7
+    return {"architecture": "Dibedra", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.25,
+            "initializer_range": 0.02, "layers": five + second}
+
+
 def design_vopedra(args, design="vopedra"):
     """Prefill and decode rates of Vopedra models (random weights) beside Phi models of the same width, the
     same number of layer runs and feed-forwards of the same number of weights; with ``design`` "gozolix" or
     "lilupel", of models of that design beside Vopedra models of the same width and number of layer runs; with
     "darusun", beside Gozolix models (the nearest relative: softmax attention, layers on another layer's keys, dense
-    feed-forwards and routed mixtures with a shared expert).  One JSON line."""
+    feed-forwards and routed mixtures with a shared expert); with "dibedra", beside Gozolix models (grouped attention,
+    dense feed-forwards, grouped routing) and Phi models (the same block).  One JSON line."""
     import numpy as np
     import torch
     import gopherllm_b200 as gl
@@ -472,6 +494,13 @@ def design_vopedra(args, design="vopedra"):
     clocks.start()
     rows = []
     for width, heads, ff_gated, ff_plain in ((1024, 16, 2752, 4096), (2048, 32, 5504, 8192)):
+        if design == "dibedra":
+            d = measure(dibedra_sizes(width, heads, ff_gated))
+            phi = dict(PHI15, hidden_size=width, num_attention_heads=heads, num_key_value_heads=heads,
+                       intermediate_size=(3 * ff_gated // 2) // 64 * 64, vocab_size=32000, num_hidden_layers=d["layer_runs"])
+            rows.append({"width": width, "heads": heads, design: d, "gozolix": measure(gozolix_sizes(width, heads, ff_gated)),
+                         "phi": measure(phi)})
+            continue
         if design == "darusun":
             rows.append({"width": width, "heads": heads, design: measure(darusun_sizes(width, heads, ff_gated)),
                          "gozolix": measure(gozolix_sizes(width, heads, ff_gated))})
@@ -485,8 +514,8 @@ def design_vopedra(args, design="vopedra"):
         phi = dict(PHI15, hidden_size=width, num_attention_heads=heads, num_key_value_heads=heads,
                    intermediate_size=ff_plain, vocab_size=32000, num_hidden_layers=v["layer_runs"])
         rows.append({"width": width, "heads": heads, "vopedra": v, "phi": measure(phi)})
-    if design in ("gozolix", "lilupel", "darusun"):
-        beside = "Gozolix" if design == "darusun" else "Vopedra"
+    if design in ("gozolix", "lilupel", "darusun", "dibedra"):
+        beside = {"darusun": "Gozolix", "dibedra": "Gozolix and Phi"}.get(design, "Vopedra")
         print(json.dumps({"metric": f"prefill and decode rates of {design.capitalize()} layer sizes beside {beside} of equal width and depth (bf16)",
                           "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic: random weights seed 7, uniform token ids",
                           "decode_steps_timed": K, "decode_context": 1024, "peaks": pk_src, "clocks": clocks.stop(), "sizes": rows}))

@@ -404,7 +404,7 @@ GL_API int gl_moe_gather_rows(const void* x, const int* order, void* xs, int row
 }
 
 // out[t, :] = sum_k weights[t, k] * y[place[t, k], :] (+ add[t, :]), in the order of the choices; a place of -1 is the
-// identity: the token's input x[t, :] (bfloat16) takes y's part.  Four columns a thread.
+// identity: the token's input x[t, :] (bfloat16, where given) takes y's part.  Four columns a thread.
 __global__ void __launch_bounds__(256)
 moe_combine_placed_kernel(const float* y, const int* place, const float* weights, const __nv_bfloat16* x, const float* add,
                           float* out, long long n4, int N4, int top) {
@@ -422,6 +422,8 @@ moe_combine_placed_kernel(const float* y, const int* place, const float* weights
         float4 v;
         if (row >= 0) {
             v = ((const float4*)y)[(size_t)row * N4 + c];
+        } else if (!x) {
+            continue;
         } else {
             const uint2 raw = ((const uint2*)x)[(size_t)t * N4 + c];
             const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
@@ -435,7 +437,7 @@ moe_combine_placed_kernel(const float* y, const int* place, const float* weights
 GL_API int gl_moe_combine_placed(const float* y, const int* place, const float* weights, const void* x, const float* add,
                                  float* out, int T, int N, int top, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
-    if (N <= 0 || N % 4 || top <= 0 || !x) return GL_ERR_SHAPE;
+    if (N <= 0 || N % 4 || top <= 0) return GL_ERR_SHAPE;
     if (((uintptr_t)y | (uintptr_t)add | (uintptr_t)out) & 15 || ((uintptr_t)x & 7)) return GL_ERR_ALIGN;
     const long long n4 = (long long)T * (N / 4);
     return gl_launch(moe_combine_placed_kernel, dim3((unsigned)((n4 + 255) / 256)), dim3(256), 0, stream, 1, y, place, weights,
@@ -817,7 +819,7 @@ GL_API int gl_moe_down_simt(const ExpertArgs* args, int x_dtype, int w_dtype, cu
 
 // ---------------------------------------------------------------------------
 // out[t, :] = sum_k y[t, k, :] (+ add[t, :]); out may be add itself.  A choice at or above E is the identity: its part
-// is weights[t, k] * x[t, :].
+// is weights[t, k] * x[t, :] (none where x is absent).
 // ---------------------------------------------------------------------------
 template <typename TA>
 __global__ void __launch_bounds__(256)
@@ -831,7 +833,8 @@ moe_combine_kernel(const float* y, const int* ids, const float* weights, const T
     const int c = (int)(i - t * N);
     float s = 0.f;
     for (int k = 0; k < top; ++k)
-        s += ids[t * top + k] < E ? y[((size_t)t * top + k) * N + c] : weights[t * top + k] * gl_load(x + (size_t)t * N + c);
+        if (ids[t * top + k] < E) s += y[((size_t)t * top + k) * N + c];
+        else if (x) s += weights[t * top + k] * gl_load(x + (size_t)t * N + c);
     out[i] = add ? add[i] + s : s;
 }
 

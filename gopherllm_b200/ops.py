@@ -1839,10 +1839,10 @@ USE_MOE_TC = True        # bfloat16 experts on the tensor cores (False: the CUDA
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, add: Optional[torch.Tensor] = None,
-                out: Optional[torch.Tensor] = None, act="silu") -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, act="silu", identity: bool = False) -> torch.Tensor:
     """out[t] = sum_k weights[t, k] * down_e(silu(gate_e(x[t])) * up_e(x[t])) + add[t], e = ids[t, k]; float32
-    [T, hidden].  ``act``: another gated form in silu's place (see gated_act).  A choice e >= E is the identity: its
-    part is weights[t, k] * x[t], and it takes no part in the products.  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
+    [T, hidden].  ``act``: another gated form in silu's place (see gated_act).  ``identity``: a choice e >= E is the
+    identity: its part is weights[t, k] * x[t], and it takes no part in the products.  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
     The step's (token, choice) pairs are sorted by expert on the device and cut into tiles of rows; the grids
     cover the most tiles any choice can make, so nothing depends on the host knowing what the router chose.
     Which kernels run depends on the step's size alone: up to MOE_ROWS_KERNEL_PER_EXPERT pairs an expert on
@@ -1865,8 +1865,9 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     hidden = w_down.shape[1]
     if Kw != K or F2 % 2 or tuple(w_down.shape) != (E, hidden, F) or tuple(ids.shape) != (T, top):
         raise KernelError(f"moe_experts: weights {tuple(w_gate_up.shape)} / {tuple(w_down.shape)} do not fit x {tuple(x.shape)}")
-    if hidden != K:
-        raise KernelError("moe_experts: the experts' inputs and outputs have one width (a choice may be the input itself)")
+    if identity and hidden != K:
+        raise KernelError("moe_experts: where a choice may be the input itself, inputs and outputs have one width")
+    x_id = x if identity else None
     code, limit, slope, shift = _gated_code(act)
     if add is not None:
         _need(add, "add", torch.float32, (T, hidden))
@@ -1895,7 +1896,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         if late_add is not None:
             add = late_add()
             _need(add, "add", torch.float32, (T, hidden))
-        _check(_launch(lib.gl_moe_combine_placed, _ptr(y), _ptr(place), _ptr(weights), _ptr(x), _ptr(add), _ptr(out), c_int(T),
+        _check(_launch(lib.gl_moe_combine_placed, _ptr(y), _ptr(place), _ptr(weights), _ptr(x_id), _ptr(add), _ptr(out), c_int(T),
                        c_int(hidden), c_int(top), _stream()), "moe_combine")
         return out
     max_tiles = -(-A // MOE_TILE_ROWS) + min(E, A)
@@ -1919,7 +1920,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     if late_add is not None:
         add = late_add()
         _need(add, "add", torch.float32, (T, hidden))
-    _check(_launch(lib.gl_moe_combine, _ptr(y), _ptr(ids), _ptr(weights), _ptr(x), xd, _ptr(add), _ptr(out), c_int(T), c_int(hidden),
+    _check(_launch(lib.gl_moe_combine, _ptr(y), _ptr(ids), _ptr(weights), _ptr(x_id), xd, _ptr(add), _ptr(out), c_int(T), c_int(hidden),
                    c_int(top), c_int(E), _stream()),
            "moe_combine")
     return out

@@ -296,9 +296,11 @@ class MixtureOfExperts(FeedForward):
                 return ys
 
             ids, weights = self.route(xn, ctx)
-            return ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=shared, out=out, act=self.act)
+            return ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=shared, out=out, act=self.act,
+                                   identity=self.identity > 0)
         ids, weights = self.route(xn, ctx)
-        out = ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=add[0] if len(add) > 0 else None, out=out, act=self.act)
+        out = ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=add[0] if len(add) > 0 else None, out=out,
+                              act=self.act, identity=self.identity > 0)
         if self.shared:
             gu = ops.linear(xn, self.ws_gu, None, out_dtype=ctx.act_dtype)
             hs = (ops.gated_act(gu, "silu", inner=self.shared, row_gate=2 * self.shared) if self.shared_gate
