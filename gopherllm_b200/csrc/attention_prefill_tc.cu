@@ -1,8 +1,9 @@
 // Prefill attention on the 5th-generation tensor cores: runs of new tokens against the
 // paged bfloat16 cache (their own keys included), causal, with an optional window.
 //
-// A block takes 256 consecutive query rows of one (sequence, head) as two tiles of 128 and
-// walks the keys a page (64) at a time.  One warp feeds shared memory by TMA: the query tiles
+// A block takes 256 consecutive query rows of one (sequence, head) as two tiles of 128 (or, where two
+// blocks of one tile fit an SM and suit the step better, 128 rows as one tile) and walks the keys a page
+// (64) at a time.  One warp feeds shared memory by TMA: the query tiles
 // once, then key pages and value pages, each in a ring of its own, several pages ahead.  Each
 // tile has a thread of its own that issues tcgen05.mma: scores S = Q K^T (M 128, N 64) into
 // one of the tile's two score buffers in tensor memory, two pages ahead of the rows, and
@@ -39,8 +40,9 @@ static_assert(GL_PAGE == 64, "a step is one page of 64 keys");
 
 #define AT_HD GL_HEAD_DIM
 #define AT_BM 128                 // query rows of a tile
-#define AT_THREADS 352
-#define AT_TMEM_COLS 512
+// A block of NT tiles: four row warps a tile, one warp that feeds shared memory, one issuing warp a tile
+#define AT_THREADS(NT) ((NT) * 160 + 32)
+#define AT_TMEM_COLS(NT) (256 * (NT))
 
 // pieces of the head size for queries and keys: widths 64, 64, 32, 16 as far as they fit
 struct AtSeg { int off, width; };
@@ -64,13 +66,13 @@ __host__ __device__ constexpr int at_seg_base(int i, int rows) {
 #define AT_VATOMS ((AT_HD + 63) / 64)
 #define AT_VATOM_BYTES (GL_PAGE * 128)                   // 64 keys x 64 dims
 #define AT_V_BYTES (AT_VATOMS * AT_VATOM_BYTES)          // a page of values
-// Pages in flight in each ring: as many as fit beside the two query tiles.
-__host__ __device__ constexpr int at_stages() {
-    int n = (227 * 1024 - 2048 - 2 * AT_Q_BYTES) / (AT_K_BYTES + AT_V_BYTES);
+// Pages in flight in each ring: as many as fit beside the query tiles, in one block an SM of two tiles or in two of one.
+__host__ __device__ constexpr int at_stages(int nt) {
+    int n = ((nt == 2 ? 227 * 1024 : 113 * 1024) - 2048 - nt * AT_Q_BYTES) / (AT_K_BYTES + AT_V_BYTES);
     return n > 8 ? 8 : n;
 }
-#define AT_STAGES at_stages()
-static_assert(AT_STAGES >= 4, "shared memory holds too few key/value pages");
+static_assert(at_stages(2) >= 4, "shared memory holds too few key/value pages");
+#define AT_ONE_TILE (at_stages(1) >= 3)      // whether blocks of one tile exist for this head size
 
 struct AttnArgs {
     const void* q;            // [T, nH*hd] bf16, already scaled
@@ -100,7 +102,8 @@ __device__ __forceinline__ float at_exp2(float x) {
     return y;
 }
 
-__global__ void __launch_bounds__(AT_THREADS, 1)
+template <int NT>
+__global__ void __launch_bounds__(AT_THREADS(NT), 3 - NT)
 attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMaps maps) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ unsigned tmem_slot;
@@ -108,7 +111,9 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
     unsigned char* smem = smem_raw + ((1024u - (gl_smem_u32(smem_raw) & 1023u)) & 1023u);
     const unsigned base = gl_smem_u32(smem);
     const unsigned sQ = base;                                          // [2] query tiles
-    const unsigned sK = sQ + 2 * AT_Q_BYTES;                           // [AT_STAGES] key pages
+    constexpr int AT_STAGES = at_stages(NT);
+    constexpr int PRODUCER = 4 * NT;                                   // the warp that feeds shared memory; issuers follow
+    const unsigned sK = sQ + NT * AT_Q_BYTES;                          // [AT_STAGES] key pages
     const unsigned sV = sK + AT_STAGES * AT_K_BYTES;                   // [AT_STAGES] value pages
     const unsigned bars = sV + AT_STAGES * AT_V_BYTES;
     const unsigned bar_q = bars;
@@ -124,12 +129,12 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
     // the far end: the blocks with the most keys to walk start first, whatever their sequence and head.
     const int h = blockIdx.x % a.nH, b = (blockIdx.x / a.nH) % a.B;
     const int qlen = a.seq_qlen[b];
-    const int qt = (a.max_qlen + 2 * AT_BM - 1) / (2 * AT_BM) - 1 - (int)(blockIdx.x / (a.nH * a.B));
-    if (qt * 2 * AT_BM >= qlen) return;
+    const int qt = (a.max_qlen + NT * AT_BM - 1) / (NT * AT_BM) - 1 - (int)(blockIdx.x / (a.nH * a.B));
+    if (qt * NT * AT_BM >= qlen) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int ctx = a.seq_ctx[b], qstart = a.seq_qstart[b];
-    const int q0 = qt * 2 * AT_BM;
-    const int rows_all = min(2 * AT_BM, qlen - q0);
+    const int q0 = qt * NT * AT_BM;
+    const int rows_all = min(NT * AT_BM, qlen - q0);
     const int g = h / (a.nH / a.nKV);
     const int total = ctx + qlen;
     const int p_first = ctx + q0;
@@ -145,16 +150,16 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
         failed = 0;
         mbar_init(bar_q, 1);
         for (int s = 0; s < AT_STAGES; ++s) {
-            mbar_init(bar_kf + 8 * s, 1); mbar_init(bar_ke + 8 * s, 2);     // both issuers release a page
-            mbar_init(bar_vf + 8 * s, 1); mbar_init(bar_ve + 8 * s, 2);
+            mbar_init(bar_kf + 8 * s, 1); mbar_init(bar_ke + 8 * s, NT);    // every issuer releases a page
+            mbar_init(bar_vf + 8 * s, 1); mbar_init(bar_ve + 8 * s, NT);
         }
-        for (int t = 0; t < 2; ++t) {
+        for (int t = 0; t < NT; ++t) {
             for (int i = 0; i < 2; ++i) { mbar_init(BAR_SF(t, i), 1); mbar_init(BAR_PF(t, i), 4); }
             mbar_init(BAR_PD(t), 1); mbar_init(BAR_OF(t), 1);
         }
         mbar_fence_init();
     }
-    if (warp == 8) tmem_alloc(gl_smem_u32(&tmem_slot), AT_TMEM_COLS);
+    if (warp == PRODUCER) tmem_alloc(gl_smem_u32(&tmem_slot), AT_TMEM_COLS(NT));
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -164,12 +169,12 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
     // tile t: score buffers at columns 256 t and 256 t + 64 (the weights of a page overwrite the first
     // 32 columns of its scores, two a column), output at 256 t + 128
 
-    if (warp == 8) {
+    if (warp == PRODUCER) {
         // ---- TMA producer ------------------------------------------------------
         if (lane == 0) {
-            mbar_expect_tx(bar_q, 2 * AT_BM * AT_HD * 2);
+            mbar_expect_tx(bar_q, NT * AT_BM * AT_HD * 2);
 #pragma unroll
-            for (int t = 0; t < 2; ++t)
+            for (int t = 0; t < NT; ++t)
 #pragma unroll
                 for (int s = 0; s < AT_NSEG; ++s)
                     tma_load_2d(sQ + t * AT_Q_BYTES + at_seg_base(s, AT_BM), &maps.q[s], h * AT_HD + at_seg(s).off,
@@ -190,12 +195,12 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
                     tma_load_2d(sV + st * AT_V_BYTES + c * AT_VATOM_BYTES, &maps.v, 64 * c, row, bar_vf + 8 * st);
             }
         }
-    } else if (warp == 9 || warp == 10) {
+    } else if (warp > PRODUCER) {
         // ---- MMA issuers: one thread a tile ----------------------------------------------
         if (lane == 0) {
             constexpr uint32_t idesc_s = umma_idesc_bf16(GL_PAGE, 0);
             constexpr uint32_t idesc_o = umma_idesc_bf16(AT_HD, 1);
-            const int t = warp - 9;
+            const int t = warp - PRODUCER - 1;
             const int nt = t ? n1 : n0;
             auto issue_scores = [&](int j) {                  // S_j = Q K_j^T into score buffer j & 1
                 const int st = j % AT_STAGES;
@@ -253,8 +258,8 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
             }
             if (!ok) failed = 1;
         }
-    } else if (warp < 8) {
-        // ---- softmax and output: warps 0..7, one query row per thread -------------------
+    } else {
+        // ---- softmax and output: the first four warps a tile, one query row per thread -------------------
         const int t = warp >> 2, quarter = warp & 3;
         const int r = quarter * 32 + lane;                                  // row inside the tile
         const int rows = min(AT_BM, rows_all - t * AT_BM);                  // valid rows of this tile (may be <= 0)
@@ -396,16 +401,20 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
     }
     tc_fence_before();
     __syncthreads();
-    if (warp == 8) {
+    if (warp == PRODUCER) {
         tc_fence_after();
-        tmem_dealloc(tmem, AT_TMEM_COLS);
+        tmem_dealloc(tmem, AT_TMEM_COLS(NT));
     }
     if (threadIdx.x == 0 && failed) atomicExch(&gl_wait_failed, 1);
 }
 
-static size_t at_smem() {
-    return 2 * (size_t)AT_Q_BYTES + AT_STAGES * ((size_t)AT_K_BYTES + AT_V_BYTES) + 512 + 1024;
+static size_t at_smem(int nt) {
+    return nt * (size_t)AT_Q_BYTES + at_stages(nt) * ((size_t)AT_K_BYTES + AT_V_BYTES) + 512 + 1024;
 }
+
+// 0: chosen by the step (default), 1 or 2: tiles a block (for measurements)
+static int at_tiles = 0;
+GL_API void gl_attention_prefill_tc_tiles(int n) { at_tiles = n; }
 
 GL_API int gl_attention_prefill_tc_head_dim() { return AT_HD; }
 
@@ -417,20 +426,44 @@ GL_API int gl_attention_prefill_tc_wait_failed() {
     return v;
 }
 
+template <int NT>
+static bool at_allow() {
+    return cudaFuncSetAttribute(attn_prefill_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)at_smem(NT)) == cudaSuccess;
+}
+template <int NT>
+static int at_launch(long long blocks, cudaStream_t stream, const AttnArgs& a, const AttnGate& gate, const AttnMaps& maps) {
+    return gl_launch(attn_prefill_tc_kernel<NT>, dim3((unsigned)blocks), dim3(AT_THREADS(NT)), at_smem(NT), stream, 1, a, gate, maps);
+}
+
+// Tiles a block.  Blocks of one tile, two an SM, overlap one's start and end with the other's pages and share the work
+// out in smaller pieces, at the price of every tile fetching its own pages: measured ahead with a window (32 heads of 64,
+// 2,048 tokens, 512 positions: 36.9 against 44.1 us; 8 x 1,024 tokens, 256 positions: 82 against 100) and where blocks
+// of two tiles do not fill the SMs (512 tokens: 17 against 18), behind without (2,048 tokens: 56 against 48).
+static int at_choose(const AttnArgs& a, int sms) {
+    if (!AT_ONE_TILE) return 2;
+    if (at_tiles) return at_tiles;
+    const long long pairs = (long long)((a.max_qlen + 2 * AT_BM - 1) / (2 * AT_BM)) * a.nH * a.B;
+    return a.window > 0 || pairs < sms ? 1 : 2;
+}
+
 static int prefill_tc(const AttnArgs& a, const AttnGate& gate, int n_tokens, int n_pages, cudaStream_t stream) {
     if (a.B <= 0 || a.max_qlen <= 0) return GL_OK;
     if (a.hd != AT_HD || a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV) return GL_ERR_SHAPE;
     if (a.score_scale != 1.0f) return GL_ERR_SHAPE;
     if (((uintptr_t)a.q | (uintptr_t)a.out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15) return GL_ERR_ALIGN;
-    const size_t smem = at_smem();
-    static bool configured = false;
-    if (!configured) {
-        if (cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    static int sms = 0;
+    if (!sms) {
+        int dev = 0;
+        cudaGetDevice(&dev);
+        cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+        if (sms <= 0) sms = 148;
+        if (!at_allow<2>() || !at_allow<(AT_ONE_TILE ? 1 : 2)>()) {
             cudaGetLastError();
+            sms = 0;
             return GL_ERR_SMEM;
         }
-        configured = true;
     }
+    const int nt = at_choose(a, sms);
     AttnMaps maps;
     const uint64_t kv_rows = (uint64_t)n_pages * a.nKV * GL_PAGE;
     for (int s = 0; s < AT_NSEG; ++s) {
@@ -444,10 +477,10 @@ static int prefill_tc(const AttnArgs& a, const AttnGate& gate, int n_tokens, int
         int rc = gl_cached_map(&maps.v, a.v_cache, kv_rows, AT_HD, GL_PAGE, 64, 2);
         if (rc != GL_OK) return rc;
     }
-    const long long blocks = (long long)((a.max_qlen + 2 * AT_BM - 1) / (2 * AT_BM)) * a.nH * a.B;
+    const long long blocks = (long long)((a.max_qlen + nt * AT_BM - 1) / (nt * AT_BM)) * a.nH * a.B;
     if (blocks > 0x7fffffffLL) return GL_ERR_SHAPE;
-    if (gl_launch(attn_prefill_tc_kernel, dim3((unsigned)blocks), dim3(AT_THREADS), smem, stream, 1, a, gate, maps) != 0) return GL_ERR_LAUNCH;
-    return GL_OK;
+    const int rc = nt == 1 ? at_launch<(AT_ONE_TILE ? 1 : 2)>(blocks, stream, a, gate, maps) : at_launch<2>(blocks, stream, a, gate, maps);
+    return rc == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 // n_tokens: rows of q; n_pages: pages of the cache entry

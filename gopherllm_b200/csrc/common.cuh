@@ -212,8 +212,8 @@ __device__ __forceinline__ float gl_gated(float g, float u, const GlGated& p) {
     if (p.act != GL_GATED_CLIPPED) return gl_activate<EXACT>(g, p.act) * u;
     g = fminf(g, p.limit);
     u = fminf(fmaxf(u, -p.limit), p.limit);
-    const float e = EXACT ? expf(-p.slope * g) : __expf(-p.slope * g);
-    return g / (1.0f + e) * (u + p.shift);
+    if (EXACT) return g / (1.0f + expf(-p.slope * g)) * (u + p.shift);
+    return __fdividef(g, 1.0f + __expf(-p.slope * g)) * (u + p.shift);       // for results that are rounded to 16 bits right away
 }
 
 // the same for callers that carry an activation's own numbers along

@@ -81,6 +81,19 @@ __device__ __forceinline__ void moe_argmax(const float* sc, int first, int last,
     if (at == 0x7fffffff) at = first;        // (no number among them: an index inside the range all the same)
 }
 
+// how many of v[0..n) come before v[i] (larger, or equal and earlier): its place in the order
+__device__ __forceinline__ int moe_rank(const float* v, int n, int i) {
+    const float mine = v[i];
+    int r = 0;
+#pragma unroll 8
+    for (int j = 0; j < n; ++j) r += (v[j] > mine || (v[j] == mine && j < i)) ? 1 : 0;
+    return r;
+}
+
+// entries up to which every lane counts its own entries' places (no round depends on the one before); above, rounds of
+// a maximum over the warp
+#define MOE_RANK_MAX 128
+
 __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float* gsc, int t, int lane) {
     float* prob = gsc + a.groups;                            // [E] (ROUTE_SOFTMAX_ALL)
     if (a.mode == ROUTE_SOFTMAX_ALL) {
@@ -96,7 +109,21 @@ __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float*
         }
         __syncwarp();
     }
-    if (a.groups > 1 && a.keep < a.groups) {
+    if (a.groups > 1 && a.keep < a.groups && a.group_largest && a.groups <= MOE_RANK_MAX) {
+        const int per = a.E / a.groups;
+        for (int g = lane; g < a.groups; g += 32) {
+            float b = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, sc[e]);
+            gsc[g] = b;
+        }
+        __syncwarp();
+        unsigned stays = 0;                                  // bit i: group lane + 32 i stays
+        for (int g = lane, i = 0; g < a.groups; g += 32, ++i) stays |= (moe_rank(gsc, a.groups, g) < a.keep ? 1u : 0u) << i;
+        for (int g = lane, i = 0; g < a.groups; g += 32, ++i)
+            if (!((stays >> i) & 1u))
+                for (int e = g * per; e < (g + 1) * per; ++e) sc[e] = -INFINITY;
+        __syncwarp();
+    } else if (a.groups > 1 && a.keep < a.groups) {
         const int per = a.E / a.groups;
         for (int g = 0; g < a.groups; ++g) {
             float b1, b2 = 0.f;
@@ -127,6 +154,16 @@ __device__ __forceinline__ void moe_choose(const RouteArgs& a, float* sc, float*
         for (int e = lane; e < a.E; e += 32)
             if (gsc[e / per] != -INFINITY) sc[e] = -INFINITY;
         __syncwarp();
+    }
+    if (a.mode == ROUTE_SOFTMAX_ALL && a.E <= MOE_RANK_MAX) {
+        for (int e = lane; e < a.E; e += 32) {
+            const int k = moe_rank(sc, a.E, e);
+            if (k < a.top) {
+                a.ids[(size_t)t * a.top + k] = e;
+                a.weights[(size_t)t * a.top + k] = prob[e] * a.scale;
+            }
+        }
+        return;
     }
     if (a.mode == ROUTE_SOFTMAX_ALL) {
         for (int k = 0; k < a.top; ++k) {
@@ -270,11 +307,29 @@ struct PlanArgs {
     int A, E, max_tiles;
 };
 
-__global__ void __launch_bounds__(1024)
-moe_plan_kernel(PlanArgs a) {
-    extern __shared__ int ism[];
-    gl_grid_launch_dependents();
-    gl_grid_wait();
+// Warp 0: exclusive sums over the experts of two numbers of each (rows and tiles), a run of experts a lane.
+template <typename F>
+__device__ __forceinline__ int moe_scan_experts(const int* count, int E, int tile_m, const F& store) {
+    const int lane = threadIdx.x & 31, each = (E + 31) / 32, e0 = min(E, lane * each), e1 = min(E, e0 + each);
+    int rows = 0, tiles = 0;
+    for (int e = e0; e < e1; ++e) { rows += count[e]; tiles += (count[e] + tile_m - 1) / tile_m; }
+    int r = rows, t = tiles;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int pr = __shfl_up_sync(0xffffffffu, r, o), pt = __shfl_up_sync(0xffffffffu, t, o);
+        if (lane >= o) { r += pr; t += pt; }
+    }
+    const int all = __shfl_sync(0xffffffffu, t, 31);
+    r -= rows; t -= tiles;
+    for (int e = e0; e < e1; ++e) {
+        store(e, r, t);
+        r += count[e];
+        t += (count[e] + tile_m - 1) / tile_m;
+    }
+    return all;
+}
+
+__device__ __forceinline__ void moe_plan_block(const PlanArgs& a, int* ism) {
     int* count = ism;                 // [E]
     int* start = count + a.E;         // [E] first place of the expert's rows, then the running cursor
     int* tile0 = start + a.E;         // [E] first tile of the expert
@@ -285,15 +340,9 @@ moe_plan_kernel(PlanArgs a) {
         if ((unsigned)e < (unsigned)a.E) atomicAdd(&count[e], 1);
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        int at = 0, tiles = 0;
-        for (int e = 0; e < a.E; ++e) {
-            start[e] = at;
-            tile0[e] = tiles;
-            at += count[e];
-            tiles += (count[e] + MOE_TM - 1) / MOE_TM;
-        }
-        *a.n_tiles = tiles < a.max_tiles ? tiles : a.max_tiles;
+    if (threadIdx.x < 32) {
+        const int tiles = moe_scan_experts(count, a.E, MOE_TM, [&](int e, int row, int tile) { start[e] = row; tile0[e] = tile; });
+        if (threadIdx.x == 0) *a.n_tiles = tiles < a.max_tiles ? tiles : a.max_tiles;
     }
     __syncthreads();
     for (int e = threadIdx.x; e < a.E; e += blockDim.x) {
@@ -311,6 +360,47 @@ moe_plan_kernel(PlanArgs a) {
         const int e = a.ids[i];
         if ((unsigned)e < (unsigned)a.E) a.order[atomicAdd(&start[e], 1)] = i;
     }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(PlanArgs a) {
+    extern __shared__ int ism[];
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    moe_plan_block(a, ism);
+}
+
+// Few tokens: the choice and the plan in one block (a warp a token in turn, then the plan of what they chose).
+__global__ void __launch_bounds__(1024)
+moe_route_plan_kernel(RouteArgs r, PlanArgs a) {
+    extern __shared__ float smem[];
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    float* sc = smem + (size_t)warp * moe_choice_floats(r);
+    for (int t = warp; t < r.T; t += warps) {
+        for (int e = lane; e < r.E; e += 32) sc[e] = moe_score(r, r.logits[(size_t)t * r.E + e], e);
+        __syncwarp();
+        moe_choose(r, sc, sc + r.E, t, lane);
+        __syncwarp();
+    }
+    __syncthreads();
+    moe_plan_block(a, (int*)smem);
+}
+
+// threads: a warp for every token up to 32 of them (fewer where they do not fit); ids of both records are the same array
+GL_API int gl_moe_route_plan(const RouteArgs* route, const PlanArgs* plan, cudaStream_t stream) {
+    const RouteArgs& r = *route;
+    const PlanArgs& a = *plan;
+    if (r.T <= 0) return GL_OK;
+    if (!route_possible(r) || a.ids != r.ids || a.A != r.T * r.top || a.E <= 0 || a.E > r.E) return GL_ERR_SHAPE;
+    if (a.max_tiles < (a.A + MOE_TM - 1) / MOE_TM + (a.E < a.A ? a.E : a.A)) return GL_ERR_SHAPE;
+    int warps = r.T >= 32 ? 32 : (r.T < 4 ? 4 : r.T);
+    while (warps > 4 && (size_t)warps * moe_choice_floats(r) * sizeof(float) > 48 * 1024) --warps;
+    size_t smem = (size_t)warps * moe_choice_floats(r) * sizeof(float);
+    if (smem < 3 * (size_t)a.E * sizeof(int)) smem = 3 * (size_t)a.E * sizeof(int);
+    if (smem > 48 * 1024) return GL_ERR_SMEM;
+    return gl_launch(moe_route_plan_kernel, dim3(1), dim3(warps * 32), smem, stream, 1, r, a) == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 GL_API int gl_moe_plan(const PlanArgs* args, cudaStream_t stream) {
@@ -347,27 +437,51 @@ moe_plan_padded_kernel(PadPlanArgs a) {
     for (int i = threadIdx.x; i < a.max_tiles; i += blockDim.x) a.tile_expert[i] = -1;
     for (int i = threadIdx.x; i < a.max_tiles * a.tile_m; i += blockDim.x) a.order[i] = -1;
     __syncthreads();
-    for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        const int e = a.ids[i];
-        if ((unsigned)e < (unsigned)a.E) atomicAdd(&count[e], 1);
-    }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        int tiles = 0;
-        for (int e = 0; e < a.E; ++e) {
-            start[e] = tiles * a.tile_m;
-            const int n = (count[e] + a.tile_m - 1) / a.tile_m;
-            for (int i = 0; i < n && tiles + i < a.max_tiles; ++i) a.tile_expert[tiles + i] = e;
-            tiles += n;
+    // (a warp's assignments to one expert are one addition: the experts are few and the assignments thousands)
+    const int lane = threadIdx.x & 31;
+    // ... and eight of a thread's are asked for at once: one block's trips to memory are what this kernel's time is
+    constexpr int AT_ONCE = 8;
+    int e8[AT_ONCE];
+    auto fetch = [&](int base) {
+#pragma unroll
+        for (int j = 0; j < AT_ONCE; ++j) {
+            const int i = base + j * (int)blockDim.x + (int)threadIdx.x;
+            e8[j] = i < a.A ? a.ids[i] : -1;
+        }
+    };
+    for (int base = 0; base < a.A; base += AT_ONCE * (int)blockDim.x) {
+        fetch(base);
+#pragma unroll
+        for (int j = 0; j < AT_ONCE; ++j) {
+            const unsigned same = __match_any_sync(0xffffffffu, e8[j]);
+            if ((unsigned)e8[j] < (unsigned)a.E && lane == __ffs(same) - 1) atomicAdd(&count[e8[j]], __popc(same));
         }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < a.A; i += blockDim.x) {
-        const int e = a.ids[i];
-        if ((unsigned)e >= (unsigned)a.E) { a.place[i] = -1; continue; }
-        const int row = atomicAdd(&start[e], 1);
-        if (row < a.max_tiles * a.tile_m) a.order[row] = i;
-        a.place[i] = row;
+    if (threadIdx.x < 32)
+        moe_scan_experts(count, a.E, a.tile_m, [&](int e, int, int tile) {
+            start[e] = tile * a.tile_m;
+            const int n = (count[e] + a.tile_m - 1) / a.tile_m;
+            for (int i = 0; i < n && tile + i < a.max_tiles; ++i) a.tile_expert[tile + i] = e;
+        });
+    __syncthreads();
+    for (int base = 0; base < a.A; base += AT_ONCE * (int)blockDim.x) {
+        if (a.A > AT_ONCE * (int)blockDim.x) fetch(base);            // (else they are still here)
+#pragma unroll
+        for (int j = 0; j < AT_ONCE; ++j) {
+            const int i = base + j * (int)blockDim.x + (int)threadIdx.x, e = e8[j];
+            const unsigned same = __match_any_sync(0xffffffffu, e);
+            const bool mine = (unsigned)e < (unsigned)a.E;
+            int first = 0;
+            if (mine && lane == __ffs(same) - 1) first = atomicAdd(&start[e], __popc(same));
+            first = __shfl_sync(0xffffffffu, first, __ffs(same) - 1);
+            const int row = first + __popc(same & ((1u << lane) - 1));
+            if (i < a.A) {
+                if (mine && row < a.max_tiles * a.tile_m) a.order[row] = i;
+                a.place[i] = mine ? row : -1;
+            }
+            __syncwarp();
+        }
     }
 }
 
@@ -382,10 +496,11 @@ GL_API int gl_moe_plan_padded(const PadPlanArgs* args, cudaStream_t stream) {
 
 // rows of the padded, sorted input: xs[row] = x[order[row] / top], zeros where order[row] < 0; bfloat16, K % 8 == 0
 __global__ void __launch_bounds__(128)
-moe_gather_rows_kernel(const __nv_bfloat16* x, const int* order, __nv_bfloat16* xs, int K, int top) {
+moe_gather_rows_kernel(const __nv_bfloat16* x, const int* order, const int* tile_expert, int tile_m, __nv_bfloat16* xs, int K, int top) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     const int row = blockIdx.x;
+    if (tile_expert[row / tile_m] < 0) return;             // a tile not in use: nobody reads it
     const int src = order[row];
     uint4* dst = (uint4*)(xs + (size_t)row * K);
     if (src < 0) {
@@ -396,11 +511,12 @@ moe_gather_rows_kernel(const __nv_bfloat16* x, const int* order, __nv_bfloat16* 
     for (int i = threadIdx.x; i < K / 8; i += blockDim.x) dst[i] = from[i];
 }
 
-GL_API int gl_moe_gather_rows(const void* x, const int* order, void* xs, int rows, int K, int top, cudaStream_t stream) {
+GL_API int gl_moe_gather_rows(const void* x, const int* order, const int* tile_expert, int tile_m, void* xs, int rows, int K, int top,
+                              cudaStream_t stream) {
     if (rows <= 0) return GL_OK;
-    if (K <= 0 || K % 8 || top <= 0) return GL_ERR_SHAPE;
+    if (K <= 0 || K % 8 || top <= 0 || tile_m <= 0) return GL_ERR_SHAPE;
     return gl_launch(moe_gather_rows_kernel, dim3(rows), dim3(128), 0, stream, 1, (const __nv_bfloat16*)x, order,
-                     (__nv_bfloat16*)xs, K, top) == 0 ? GL_OK : GL_ERR_LAUNCH;
+                     tile_expert, tile_m, (__nv_bfloat16*)xs, K, top) == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 // out[t, :] = sum_k weights[t, k] * y[place[t, k], :] (+ add[t, :]), in the order of the choices; a place of -1 is the
@@ -675,17 +791,18 @@ moe_expert_tc_kernel(ExpertArgs a) {
 
 // ---------------------------------------------------------------------------
 // Few rows an expert (single tokens of a few sequences): the products are a stream of the chosen experts'
-// weights, every weight row met by one to a few input rows.  A warp owns an output column: its lanes stride
-// over k with 16-byte loads of the weight row (gate and up rows together), the tile's input rows wait in shared
-// memory (eight at a time, 2,048 columns at a time), and a butterfly sum ends each row's dot product.  32-bit
+// weights, every weight row met by one to a few input rows.  A warp owns two weight rows, a column's gate and up rows
+// (gate_up) or two columns' rows (down): its lanes stride over k with 16-byte loads of both, the tile's input rows wait
+// in shared memory (eight at a time, 2,048 columns at a time), and a butterfly sum ends each row's dot product.  32-bit
 // accumulation in a fixed order; bfloat16 operands, K a multiple of 8.
 // ---------------------------------------------------------------------------
 #define MV_ROWS 8
 #define MV_KCH 2048
-#define MV_COLS 8
+#define MV_COLS 8                                  // output columns of a block
+#define MV_WARPS(gated) ((gated) ? 8 : 4)
 
 template <bool GATED>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(MV_WARPS(GATED) * 32)
 moe_expert_rows_kernel(ExpertArgs a) {
     __shared__ __align__(16) __nv_bfloat16 xs[MV_ROWS][MV_KCH];
     __shared__ int rows[MOE_TM];
@@ -698,81 +815,74 @@ moe_expert_rows_kernel(ExpertArgs a) {
     if (tid < MOE_TM) rows[tid] = tid < nrows ? (GATED ? a.order[start + tid] / a.top : start + tid) : -1;
     __syncthreads();
     const __nv_bfloat16* X = (const __nv_bfloat16*)a.x;
-    const __nv_bfloat16* Wg = (const __nv_bfloat16*)a.w + (size_t)e * (GATED ? 2 : 1) * a.N * a.K;
-    const __nv_bfloat16* Wu = Wg + (size_t)a.N * a.K;
-    const int n_first = blockIdx.x * MV_COLS;
+    const __nv_bfloat16* We = (const __nv_bfloat16*)a.w + (size_t)e * (GATED ? 2 : 1) * a.N * a.K;
+    const int n0 = blockIdx.x * MV_COLS + warp, n1 = GATED ? n0 : n0 + MV_WARPS(GATED);      // this warp's columns
+    // (a column past the last is computed as column 0 and dropped)
+    const __nv_bfloat16* w0 = We + (size_t)(n0 < a.N ? n0 : 0) * a.K;
+    const __nv_bfloat16* w1 = We + (size_t)((n1 < a.N ? n1 : 0) + (GATED ? a.N : 0)) * a.K;
     for (int r0 = 0; r0 < nrows; r0 += MV_ROWS) {
         const int nr = min(MV_ROWS, nrows - r0);
-        float accg[MV_COLS / 4][MV_ROWS], accu[MV_COLS / 4][MV_ROWS];
+        float acc0[MV_ROWS], acc1[MV_ROWS];
 #pragma unroll
-        for (int c = 0; c < MV_COLS / 4; ++c)
-#pragma unroll
-            for (int r = 0; r < MV_ROWS; ++r) accg[c][r] = accu[c][r] = 0.f;
+        for (int r = 0; r < MV_ROWS; ++r) acc0[r] = acc1[r] = 0.f;
         for (int k0 = 0; k0 < a.K; k0 += MV_KCH) {
             const int kn = min(MV_KCH, a.K - k0);
+            // A lane's first pieces of both weight rows are asked for before the tokens' rows are staged: the trip to
+            // memory runs under the staging, and after it the next pieces' under the arithmetic of this step.
+            const uint4 none = make_uint4(0, 0, 0, 0);
+            uint4 next0 = lane * 8 < kn ? *(const uint4*)(w0 + k0 + lane * 8) : none;
+            uint4 next1 = lane * 8 < kn ? *(const uint4*)(w1 + k0 + lane * 8) : none;
             __syncthreads();
-            for (int el = tid; el < nr * (kn / 8); el += 128) {
+            for (int el = tid; el < nr * (kn / 8); el += MV_WARPS(GATED) * 32) {
                 const int r = el / (kn / 8), c = (el - r * (kn / 8)) * 8;
                 *(uint4*)&xs[r][c] = *(const uint4*)(X + (size_t)rows[r0 + r] * a.K + k0 + c);
             }
             __syncthreads();
-#pragma unroll
-            for (int c = 0; c < MV_COLS / 4; ++c) {
-                const int n = n_first + warp + 4 * c;
-                if (n >= a.N) continue;
-                const __nv_bfloat16* wg = Wg + (size_t)n * a.K + k0;
-                const __nv_bfloat16* wu = Wu + (size_t)n * a.K + k0;
 #pragma unroll 2
-                for (int k = lane * 8; k < kn; k += 256) {
-                    const uint4 rg = *(const uint4*)(wg + k);
-                    uint4 ru = make_uint4(0, 0, 0, 0);
-                    if (GATED) ru = *(const uint4*)(wu + k);
-                    const __nv_bfloat162* pg = (const __nv_bfloat162*)&rg;
-                    const __nv_bfloat162* pu = (const __nv_bfloat162*)&ru;
-                    float g[8], u[8];
+            for (int k = lane * 8; k < kn; k += 256) {
+                const uint4 ra = next0, rb = next1;
+                if (k + 256 < kn) {
+                    next0 = *(const uint4*)(w0 + k0 + k + 256);
+                    next1 = *(const uint4*)(w1 + k0 + k + 256);
+                }
+                const __nv_bfloat162* pa = (const __nv_bfloat162*)&ra;
+                const __nv_bfloat162* pb = (const __nv_bfloat162*)&rb;
+                float wa[8], wb[8];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 fa = __bfloat1622float2(pa[i]), fb = __bfloat1622float2(pb[i]);
+                    wa[2 * i] = fa.x; wa[2 * i + 1] = fa.y;
+                    wb[2 * i] = fb.x; wb[2 * i + 1] = fb.y;
+                }
+#pragma unroll
+                for (int r = 0; r < MV_ROWS; ++r) {
+                    if (r >= nr) break;
+                    const uint4 rx = *(const uint4*)&xs[r][k];
+                    const __nv_bfloat162* px = (const __nv_bfloat162*)&rx;
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        const float2 fg = __bfloat1622float2(pg[i]);
-                        g[2 * i] = fg.x; g[2 * i + 1] = fg.y;
-                        if (GATED) {
-                            const float2 fu = __bfloat1622float2(pu[i]);
-                            u[2 * i] = fu.x; u[2 * i + 1] = fu.y;
-                        }
-                    }
-#pragma unroll
-                    for (int r = 0; r < MV_ROWS; ++r) {
-                        if (r >= nr) break;
-                        const uint4 rx = *(const uint4*)&xs[r][k];
-                        const __nv_bfloat162* px = (const __nv_bfloat162*)&rx;
-#pragma unroll
-                        for (int i = 0; i < 4; ++i) {
-                            const float2 fx = __bfloat1622float2(px[i]);
-                            accg[c][r] = fmaf(fx.x, g[2 * i], accg[c][r]);
-                            accg[c][r] = fmaf(fx.y, g[2 * i + 1], accg[c][r]);
-                            if (GATED) {
-                                accu[c][r] = fmaf(fx.x, u[2 * i], accu[c][r]);
-                                accu[c][r] = fmaf(fx.y, u[2 * i + 1], accu[c][r]);
-                            }
-                        }
+                        const float2 fx = __bfloat1622float2(px[i]);
+                        acc0[r] = fmaf(fx.x, wa[2 * i], acc0[r]);
+                        acc0[r] = fmaf(fx.y, wa[2 * i + 1], acc0[r]);
+                        acc1[r] = fmaf(fx.x, wb[2 * i], acc1[r]);
+                        acc1[r] = fmaf(fx.y, wb[2 * i + 1], acc1[r]);
                     }
                 }
             }
         }
 #pragma unroll
-        for (int c = 0; c < MV_COLS / 4; ++c) {
-            const int n = n_first + warp + 4 * c;
-#pragma unroll
-            for (int r = 0; r < MV_ROWS; ++r) {
-                if (r >= nr) break;
-                const float g = gl_warp_sum(accg[c][r]);
-                const float u = GATED ? gl_warp_sum(accu[c][r]) : 0.f;
-                if (lane != 0 || n >= a.N) continue;
-                if (GATED) {
-                    ((__nv_bfloat16*)a.out)[(size_t)(start + r0 + r) * a.N + n] = __float2bfloat16_rn(gl_gated<false>(g, u, a.act));
-                } else {
-                    const int asg = a.order[start + r0 + r];
-                    ((float*)a.out)[(size_t)asg * a.N + n] = g * a.weights[asg];
-                }
+        for (int r = 0; r < MV_ROWS; ++r) {
+            if (r >= nr) break;
+            const float y0 = gl_warp_sum(acc0[r]), y1 = gl_warp_sum(acc1[r]);
+            if (lane != 0) continue;
+            if (GATED) {
+                if (n0 < a.N)
+                    ((__nv_bfloat16*)a.out)[(size_t)(start + r0 + r) * a.N + n0] = __float2bfloat16_rn(gl_gated<false>(y0, y1, a.act));
+            } else {
+                const int asg = a.order[start + r0 + r];
+                float* o = (float*)a.out + (size_t)asg * a.N;
+                if (n0 < a.N) o[n0] = y0 * a.weights[asg];
+                if (n1 < a.N) o[n1] = y1 * a.weights[asg];
             }
         }
     }
@@ -788,7 +898,7 @@ static int launch_expert(const ExpertArgs& a, int x_dtype, int w_dtype, cudaStre
     if (x_dtype == GL_BF16 && w_dtype == GL_BF16 && a.K % 8 == 0 && a.A <= MV_MAX_ROWS_PER_EXPERT * a.E) {
         const dim3 grid((a.N + MV_COLS - 1) / MV_COLS, a.max_tiles);
         if (grid.y > 65535) return GL_ERR_SHAPE;
-        return gl_launch(moe_expert_rows_kernel<GATED>, grid, dim3(128), 0, stream, 1, a) == 0 ? GL_OK : GL_ERR_LAUNCH;
+        return gl_launch(moe_expert_rows_kernel<GATED>, grid, dim3(MV_WARPS(GATED) * 32), 0, stream, 1, a) == 0 ? GL_OK : GL_ERR_LAUNCH;
     }
     if (x_dtype == GL_BF16 && w_dtype == GL_BF16 && a.K % 8 == 0) {
         const dim3 grid((a.N + MOE_TN - 1) / MOE_TN, a.max_tiles);

@@ -224,10 +224,22 @@ qkv_headnorm_bf16_kernel(QkvCacheArgs a) {
     const int t = live ? (int)(item / heads) : 0, j = live ? (int)(item - (long long)t * heads) : 0;
     const int kind = j < a.nH ? 0 : (j < a.nH + a.nKV ? 1 : 2);           // q, k, v
     float gm[8];                                                          // (a weight: asked for before the wait)
-#pragma unroll
-    for (int e = 0; e < 8; ++e) gm[e] = (live && kind != 2) ? (kind == 0 ? a.q_gamma : a.k_gamma)[c * 8 + e] : 0.f;
+    const float* gamma = (kind == 0 ? a.q_gamma : a.k_gamma) + c * 8;
+    *(float4*)&gm[0] = (live && kind != 2) ? *(const float4*)gamma : make_float4(0.f, 0.f, 0.f, 0.f);
+    *(float4*)&gm[4] = (live && kind != 2) ? *(const float4*)(gamma + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     gl_grid_wait();
     uint4 raw = make_uint4(0, 0, 0, 0);
+    float co[4] = {1.f, 1.f, 1.f, 1.f}, si[4] = {0.f, 0.f, 0.f, 0.f};     // this lane's four pairs
+    if (live && kind != 2 && a.cosv && c * 4 < a.half) {
+        const float* cs = a.cosv + (size_t)t * a.half + c * 4;
+        const float* sn = a.sinv + (size_t)t * a.half + c * 4;
+        if (a.half % 4 == 0) {                                            // (rows of whole 16-byte units)
+            *(float4*)co = *(const float4*)cs;
+            *(float4*)si = *(const float4*)sn;
+        } else {
+            for (int e = 0; e < 4 && c * 4 + e < a.half; ++e) { co[e] = cs[e]; si[e] = sn[e]; }
+        }
+    }
     if (live) raw = *(const uint4*)((const __nv_bfloat16*)a.qkv + (size_t)t * a.ld + (size_t)j * a.hd + c * 8);
     float v[8], s = 0.f;
     const __nv_bfloat162* p2 = (const __nv_bfloat162*)&raw;
@@ -246,12 +258,8 @@ qkv_headnorm_bf16_kernel(QkvCacheArgs a) {
         const float sc = kind == 0 ? a.q_scale : 1.0f;
         __nv_bfloat162 o2[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = c * 4 + e;                                      // the pair's index
-            float co = 1.f, si = 0.f;
-            if (i < a.half && a.cosv) { co = a.cosv[(size_t)t * a.half + i]; si = a.sinv[(size_t)t * a.half + i]; }
-            o2[e] = __floats2bfloat162_rn((v[2 * e] * co - v[2 * e + 1] * si) * sc, (v[2 * e + 1] * co + v[2 * e] * si) * sc);
-        }
+        for (int e = 0; e < 4; ++e)
+            o2[e] = __floats2bfloat162_rn((v[2 * e] * co[e] - v[2 * e + 1] * si[e]) * sc, (v[2 * e + 1] * co[e] + v[2 * e] * si[e]) * sc);
         out = *(const uint4*)o2;
     }
     if (kind == 0) {
@@ -280,7 +288,8 @@ GL_API int gl_qkv_cache(const QkvCacheArgs* args, int act_dtype, int cache_dtype
     if (a.ld < 0 || (a.ld > 0 && a.ld < (a.nH + (a.v_from_k ? 1 : 2) * a.nKV) * a.hd) || (a.v_from_k && a.ld == 0)) return GL_ERR_SHAPE;
     const bool aligned = !(((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15);
     if (act_dtype == GL_BF16 && cache_dtype == GL_BF16 && a.q_gamma && a.k_gamma && !a.q_beta && !a.k_beta && a.norm_rms &&
-        (a.interleaved || a.half == 0) && a.hd % 8 == 0 && a.hd <= 256 && aligned) {
+        (a.interleaved || a.half == 0) && a.hd % 8 == 0 && a.hd <= 256 && aligned &&
+        !(((uintptr_t)a.q_gamma | (uintptr_t)a.k_gamma | (uintptr_t)a.cosv | (uintptr_t)a.sinv) & 15)) {
         QkvCacheArgs b = a;
         if (b.ld == 0) b.ld = (a.nH + 2 * a.nKV) * a.hd;
         const int chunks = a.hd / 8;

@@ -487,12 +487,14 @@ gated_act_kernel(const TA* gu, TA* __restrict__ out, long long n, int F, GlGated
 
 // bfloat16 rows whose halves are whole 16-byte units: eight columns a thread, 16-byte loads and stores
 __global__ void __launch_bounds__(256)
-gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out, long long n8, int F8, GlGated act) {
+gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out, long long n8, int F8, GlGated act, const int* tile_group,
+                        int tile_m) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n8; i += (long long)gridDim.x * blockDim.x) {
         const long long t = i / F8;
         const int j = (int)(i - t * F8);
+        if (tile_group && tile_group[t / tile_m] < 0) continue;        // rows of a tile not in use
         const uint4* row = (const uint4*)(gu + (size_t)t * 16 * F8);
         const uint4 g = row[j], u = row[F8 + j];
         const __nv_bfloat162* g2 = (const __nv_bfloat162*)&g;
@@ -502,14 +504,16 @@ gated_act_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* __restrict__ out
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const float2 gf = __bfloat1622float2(g2[e]), uf = __bfloat1622float2(u2[e]);
-            o2[e] = __floats2bfloat162_rn(gl_gated<true>(gf.x, uf.x, act), gl_gated<true>(gf.y, uf.y, act));
+            o2[e] = __floats2bfloat162_rn(gl_gated<false>(gf.x, uf.x, act), gl_gated<false>(gf.y, uf.y, act));
         }
         ((uint4*)out)[i] = o;
     }
 }
 
+// tile_group (or null): rows are tiles of tile_m, and a tile with a negative entry is left out (bfloat16 in whole 16-byte
+// units only; other rows are all computed)
 GL_API int gl_gated_act(const void* gu, void* out, int T, int F, int act_code, float limit, float slope, float shift,
-                        int act_dtype, cudaStream_t stream) {
+                        int act_dtype, const int* tile_group, int tile_m, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
     if (F <= 0) return GL_ERR_SHAPE;
     const GlGated act = {act_code, limit, slope, shift};
@@ -517,7 +521,7 @@ GL_API int gl_gated_act(const void* gu, void* out, int T, int F, int act_code, f
     if (act_dtype == GL_BF16 && F % 8 == 0 && !(((uintptr_t)gu | (uintptr_t)out) & 15)) {
         const long long n8 = n / 8, want8 = (n8 + 255) / 256;
         return gl_launch(gated_act_bf16x8_kernel, dim3((unsigned)(want8 > 8192 ? 8192 : want8)), dim3(256), 0, stream, 1,
-                         (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n8, F / 8, act);
+                         (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n8, F / 8, act, tile_group, tile_m);
     }
     const long long want = (n + 255) / 256;
     const dim3 grid((unsigned)(want > 8192 ? 8192 : want));

@@ -1621,11 +1621,13 @@ def _gated_code(act):
     return ACTIVATIONS[act], 0.0, 0.0, 0.0
 
 
-def gated_act(gu: torch.Tensor, act, inner: Optional[int] = None, row_gate: Optional[int] = None) -> torch.Tensor:
+def gated_act(gu: torch.Tensor, act, inner: Optional[int] = None, row_gate: Optional[int] = None,
+              tile_group: Optional[torch.Tensor] = None, tile_rows: int = 128) -> torch.Tensor:
     """act(gate) * up (or another gated form, see _gated_code) for rows that hold the gate's columns and then the up
     projection's.  ``inner``: the rows
     are longer than that, the gate's ``inner`` columns first, the up projection's behind them; ``row_gate``: the
-    column of such a row whose sigmoid multiplies the whole row's result."""
+    column of such a row whose sigmoid multiplies the whole row's result.  ``tile_group``: rows of tiles of ``tile_rows`` whose
+    entry is negative may be left out (their result stays as it is)."""
     _need(gu, "gu")
     T, F2 = gu.shape
     if inner is not None:
@@ -1642,7 +1644,7 @@ def gated_act(gu: torch.Tensor, act, inner: Optional[int] = None, row_gate: Opti
     out = empty((T, F2 // 2), gu.dtype, gu.device)
     fn = _lib("rowwise.cu").gl_gated_act
     _check(_launch(fn, _ptr(gu), _ptr(out), c_int(T), c_int(F2 // 2), c_int(code), c_float(limit), c_float(slope), c_float(shift),
-                   c_int(dtype_code(gu.dtype)), _stream()), "gated_act")
+                   c_int(dtype_code(gu.dtype)), _ptr(tile_group), c_int(tile_rows), _stream()), "gated_act")
     return out
 
 
@@ -1832,17 +1834,59 @@ class _PadPlanArgs(Structure):
                 ("A", c_int), ("E", c_int), ("max_tiles", c_int), ("tile_m", c_int)]
 
 
-MOE_ROWS_KERNEL_PER_EXPERT = 4     # up to this many (token, choice) pairs an expert on average: the few-rows kernel
+MOE_ROUTE_PLAN_MAX_TOKENS = 64     # up to this many tokens the choice and the plan are one kernel
+# up to this many (token, choice) pairs an expert on average: the few-rows kernel.  (Ten Dibedra layers at width 2,048 with
+# 32 experts, 4 a token, ms a step, few-rows kernel / grouped products: 16 tokens 1.03 / 0.88, 24 tokens 1.34 / 0.98,
+# 32 tokens 1.59 / 1.02; at width 1,024 0.54 / 0.57, 0.66 / 0.60, 0.78 / 0.63.)
+MOE_ROWS_KERNEL_PER_EXPERT = 2
 USE_MOE_GROUPED = True             # many rows an expert in bfloat16: one grouped product on tcgen05 (False: tiles on mma.sync)
 USE_MOE_TC = True        # bfloat16 experts on the tensor cores (False: the CUDA-core kernels, for comparison)
 
 
+def _plan_buffers(A: int, E: int, dev):
+    """(order, tile_expert, tile_start, tile_rows, n_tiles, most tiles) of a plan of tiles of MOE_TILE_ROWS rows; each a
+    tensor of its own: a tape of launches knows temporaries by their first address."""
+    max_tiles = -(-A // MOE_TILE_ROWS) + min(E, A)
+    order = empty((A,), torch.int32, dev)
+    tile_expert, tile_start, tile_rows = (empty((max_tiles,), torch.int32, dev) for _ in range(3))
+    return order, tile_expert, tile_start, tile_rows, empty((1,), torch.int32, dev), max_tiles
+
+
+def moe_plans_tiles(T: int, top: int, E: int, x_dtype, w_dtype, K: int, F: int, hidden: int) -> bool:
+    """Whether ``moe_experts`` works on tiles of MOE_TILE_ROWS rows for these sizes (else every expert's rows start on a
+    tile of 128 of their own)."""
+    return not (USE_MOE_TC and USE_TCGEN05 and USE_MOE_GROUPED and x_dtype == torch.bfloat16 and w_dtype == torch.bfloat16
+                and T * top > MOE_ROWS_KERNEL_PER_EXPERT * E and K % 8 == 0 and F % 8 == 0 and hidden % 4 == 0)
+
+
+def moe_route_plan(logits: torch.Tensor, top: int, experts: int, groups: int = 1, keep: int = 1, scale: float = 1.0,
+                   bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False, softmax_all: bool = False,
+                   correction: Optional[torch.Tensor] = None, group_largest: bool = False):
+    """``moe_route`` of few tokens and the plan of the experts' tiles (``experts`` of the logits' columns; choices behind
+    them are the identity) in one kernel: (ids, weights, plan for ``moe_experts``)."""
+    _need(logits, "logits", torch.float32)
+    T, E = logits.shape
+    mode = _route_mode(E, top, groups, keep, bias, softmax_chosen, softmax_all, correction)
+    ids = empty((T, top), torch.int32, logits.device)
+    weights = empty((T, top), torch.float32, logits.device)
+    r = _RouteArgs(logits.data_ptr(), ids.data_ptr(), weights.data_ptr(), T, E, top, groups, keep, scale, _addr(bias), mode,
+                   _addr(correction), 1 if group_largest else 0)
+    plan = _plan_buffers(T * top, experts, logits.device)
+    order, tile_expert, tile_start, tile_rows, n_tiles, max_tiles = plan
+    p = _PlanArgs(ids.data_ptr(), order.data_ptr(), tile_expert.data_ptr(), tile_start.data_ptr(), tile_rows.data_ptr(),
+                  n_tiles.data_ptr(), T * top, experts, max_tiles)
+    _check(_launch(_lib("moe.cu").gl_moe_route_plan, byref(r), byref(p), _stream()), "moe_route_plan")
+    return ids, weights, plan
+
+
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, add: Optional[torch.Tensor] = None,
-                out: Optional[torch.Tensor] = None, act="silu", identity: bool = False) -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, act="silu", identity: bool = False,
+                plan=None) -> torch.Tensor:
     """out[t] = sum_k weights[t, k] * down_e(silu(gate_e(x[t])) * up_e(x[t])) + add[t], e = ids[t, k]; float32
     [T, hidden].  ``act``: another gated form in silu's place (see gated_act).  ``identity``: a choice e >= E is the
-    identity: its part is weights[t, k] * x[t], and it takes no part in the products.  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
+    identity: its part is weights[t, k] * x[t], and it takes no part in the products.  ``plan``: what ``moe_route_plan``
+    returned for these choices (where ``moe_plans_tiles``).  w_gate_up [E, 2F, K] holds every expert's gate rows and then its up rows, w_down [E, hidden, F].
     The step's (token, choice) pairs are sorted by expert on the device and cut into tiles of rows; the grids
     cover the most tiles any choice can make, so nothing depends on the host knowing what the router chose.
     Which kernels run depends on the step's size alone: up to MOE_ROWS_KERNEL_PER_EXPERT pairs an expert on
@@ -1877,8 +1921,9 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     A = T * top
     dev = x.device
     lib = _lib("moe.cu")
-    if (USE_MOE_TC and USE_TCGEN05 and USE_MOE_GROUPED and x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16
-            and A > MOE_ROWS_KERNEL_PER_EXPERT * E and K % 8 == 0 and F % 8 == 0 and hidden % 4 == 0):
+    if not moe_plans_tiles(T, top, E, x.dtype, w_gate_up.dtype, K, F, hidden):
+        if plan is not None:
+            raise KernelError("moe_experts: a plan of small tiles where the experts' rows go on tiles of 128")
         # many rows an expert: rows sorted by expert, every expert on tiles of 128 rows of its own, and each of
         # the two products one product with grouped weights
         tiles = -(-A // 128) + min(E, A)
@@ -1888,10 +1933,10 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         p = _PadPlanArgs(ids.data_ptr(), order.data_ptr(), place.data_ptr(), tile_expert.data_ptr(), A, E, tiles, 128)
         _check(_launch(lib.gl_moe_plan_padded, byref(p), _stream()), "moe_plan")
         xs = empty((tiles * 128, K), torch.bfloat16, dev)
-        _check(_launch(lib.gl_moe_gather_rows, _ptr(x), _ptr(order), _ptr(xs), c_int(tiles * 128), c_int(K), c_int(top),
+        _check(_launch(lib.gl_moe_gather_rows, _ptr(x), _ptr(order), _ptr(tile_expert), c_int(128), _ptr(xs), c_int(tiles * 128), c_int(K), c_int(top),
                        _stream()), "moe_gather_rows")
         gu = gemm_tcgen05_grouped(xs, w_gate_up, tile_expert, torch.bfloat16)
-        h = gated_act(gu, act)
+        h = gated_act(gu, act, tile_group=tile_expert, tile_rows=128)
         y = gemm_tcgen05_grouped(h, w_down, tile_expert, torch.float32)
         if late_add is not None:
             add = late_add()
@@ -1899,14 +1944,11 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         _check(_launch(lib.gl_moe_combine_placed, _ptr(y), _ptr(place), _ptr(weights), _ptr(x_id), _ptr(add), _ptr(out), c_int(T),
                        c_int(hidden), c_int(top), _stream()), "moe_combine")
         return out
-    max_tiles = -(-A // MOE_TILE_ROWS) + min(E, A)
-    # (each a tensor of its own: a tape of launches knows temporaries by their first address)
-    order = empty((A,), torch.int32, dev)
-    tile_expert, tile_start, tile_rows = (empty((max_tiles,), torch.int32, dev) for _ in range(3))
-    n_tiles = empty((1,), torch.int32, dev)
-    p = _PlanArgs(ids.data_ptr(), order.data_ptr(), tile_expert.data_ptr(), tile_start.data_ptr(), tile_rows.data_ptr(),
-                  n_tiles.data_ptr(), A, E, max_tiles)
-    _check(_launch(lib.gl_moe_plan, byref(p), _stream()), "moe_plan")
+    order, tile_expert, tile_start, tile_rows, n_tiles, max_tiles = plan if plan is not None else _plan_buffers(A, E, dev)
+    if plan is None:
+        p = _PlanArgs(ids.data_ptr(), order.data_ptr(), tile_expert.data_ptr(), tile_start.data_ptr(), tile_rows.data_ptr(),
+                      n_tiles.data_ptr(), A, E, max_tiles)
+        _check(_launch(lib.gl_moe_plan, byref(p), _stream()), "moe_plan")
     h = empty((A, F), x.dtype, dev)
     y = empty((A, hidden), torch.float32, dev)
     xd, wd = c_int(dtype_code(x.dtype)), c_int(dtype_code(w_gate_up.dtype))

@@ -260,16 +260,20 @@ class MixtureOfExperts(FeedForward):
         return out
 
     def route(self, xn, ctx=None):
-        """(experts int32 [T, top], weights float32 [T, top]) of the step's tokens."""
+        """(experts int32 [T, top], weights float32 [T, top], a plan of the experts' tiles or None) of the step's tokens."""
         if self.router == "table":
-            return ops.moe_route_table(ctx.tokens, self.table, self.E)
+            return *ops.moe_route_table(ctx.tokens, self.table, self.E), None
         how = dict(groups=self.groups, keep=self.keep, scale=self.scale, bias=self.b_router,
                    softmax_chosen=self.weights_by == "softmax_chosen", softmax_all=self.weights_by == "softmax_all",
                    correction=self.correction, group_largest=self.group_largest)
         if xn.dtype == torch.bfloat16 and self.w_router_16 is not None and xn.shape[1] % 8 == 0:
             logits = ops.linear(xn, self.w_router_16, None, out_dtype=torch.float32)
-            return ops.moe_route(logits, self.top, **how)
-        return ops.moe_route_from(xn, self.w_router, self.top, **how)
+            s = self.spec
+            if (xn.shape[0] <= ops.MOE_ROUTE_PLAN_MAX_TOKENS and self.outputs <= 1024
+                    and ops.moe_plans_tiles(xn.shape[0], self.top, self.E, xn.dtype, self.w_gu.dtype, s.hidden, s.intermediate, s.hidden)):
+                return ops.moe_route_plan(logits, self.top, self.E, **how)
+            return *ops.moe_route(logits, self.top, **how), None
+        return *ops.moe_route_from(xn, self.w_router, self.top, **how), None
 
     def forward(self, xn, ctx, add: Sequence[torch.Tensor], out=None) -> torch.Tensor:
         if len(add) > (2 if self.shared else 1):
@@ -295,12 +299,12 @@ class MixtureOfExperts(FeedForward):
                 main.wait_event(join)
                 return ys
 
-            ids, weights = self.route(xn, ctx)
+            ids, weights, plan = self.route(xn, ctx)
             return ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=shared, out=out, act=self.act,
-                                   identity=self.identity > 0)
-        ids, weights = self.route(xn, ctx)
+                                   identity=self.identity > 0, plan=plan)
+        ids, weights, plan = self.route(xn, ctx)
         out = ops.moe_experts(xn, ids, weights, self.w_gu, self.w_down, add=add[0] if len(add) > 0 else None, out=out,
-                              act=self.act, identity=self.identity > 0)
+                              act=self.act, identity=self.identity > 0, plan=plan)
         if self.shared:
             gu = ops.linear(xn, self.ws_gu, None, out_dtype=ctx.act_dtype)
             hs = (ops.gated_act(gu, "silu", inner=self.shared, row_gate=2 * self.shared) if self.shared_gate
