@@ -615,3 +615,40 @@ def test_one_token_attention_with_normed_heads(heads, kv, dim, half, window, gat
         at[int(pages[b, (n - 1) // 64]), (n - 1) % 64] = True
     assert not (changed & ~at).any()
     ops.check_wait_failures()
+
+
+@pytest.mark.parametrize("tiles", [1, 2])
+@pytest.mark.parametrize("heads,kv,dim,window,gated", [(4, 2, 64, 0, True), (2, 1, 80, 100, True), (3, 3, 16, 64, False), (2, 2, 96, 0, True),
+                                                      (2, 1, 128, 300, True)])
+def test_prompt_attention_with_a_gate_in_both_block_forms(heads, kv, dim, window, gated, tiles):
+    """The tcgen05 prompt kernel with blocks of one tile and of two (where the head size has both), unequal runs behind
+    cached positions, with and without a window and a gate, against the 32-bit kernel and the gate's own pass."""
+    from ctypes import c_int
+    from gopherllm_b200 import ops
+    from gopherllm_b200.csrc import catalog
+    dev = torch.device("cuda:0")
+    g = torch.Generator().manual_seed(13)
+    qlens, ctxs = [300, 1, 129, 64], [0, 70, 130, 5]
+    B, T, pages_each = len(qlens), sum(qlens), 5
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    q = (0.4 * torch.randn(T, heads * dim, generator=g)).to(dev, torch.bfloat16)
+    k = torch.randn(B * pages_each, kv, 64, dim, generator=g).to(dev, torch.bfloat16)
+    v = torch.randn(B * pages_each, kv, 64, dim, generator=g).to(dev, torch.bfloat16)
+    gate = torch.randn(T, 8 + heads * dim, generator=g).to(dev, torch.bfloat16)
+    pages = torch.randperm(B * pages_each, generator=g).view(B, pages_each).to(dev, torch.int32)
+    starts = [sum(qlens[:b]) for b in range(B)]
+    args = (i32(starts), i32(qlens), i32(ctxs), pages, heads, kv, dim, max(qlens))
+    want = torch.empty_like(q)
+    ops.attention_generic(q, want, k, v, *args, window=window)
+    if gated:
+        ops.sigmoid_gate(want, gate, 8)
+    lib = ops._lib("attention_prefill_tc.cu", catalog.head_dim_defines(dim))
+    lib.gl_attention_prefill_tc_tiles(c_int(tiles))
+    try:
+        got = torch.empty_like(q)
+        ops.attention_prefill_tc(q, got, k, v, *args, window, gate if gated else None, 8)
+        torch.cuda.synchronize()
+    finally:
+        lib.gl_attention_prefill_tc_tiles(c_int(0))
+    ops.check_wait_failures()
+    assert (got.float() - want.float()).abs().max() <= 3e-2
