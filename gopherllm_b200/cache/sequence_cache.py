@@ -7,8 +7,9 @@ row of every state tensor.  Cache entries whose mixers ask for the same shape
 of its own; a model whose layers differ (all keys here, a window there, state
 elsewhere) gets several groups.  When a sequence ends its slot and pages go back
 to the pools and are handed to the next sequence without being cleared;
-a group whose mixers see a window of the last w positions gives a sequence's
-pages back as soon as they lie wholly before every window still to come:
+a group whose mixers see a window of the last w positions, or their own chunk of
+positions, gives a sequence's pages back as soon as they lie wholly before everything
+still to be seen:
 positions past a sequence's length are never read (the reference's argument for
 not clearing its cache, runtime.go:1530-1531), and state rows are zeroed when a
 slot is taken (runtime.go:1526-1539).
@@ -119,7 +120,7 @@ class SequenceCache:
         # per-slot bookkeeping
         self._length = [0] * self.max_slots
         self._pages: List[List[List[int]]] = [[[] for _ in self.groups] for _ in range(self.max_slots)]
-        # per slot and group: pages before this index have been released (groups with a window only)
+        # per slot and group: pages before this index have been released (groups with a window or chunks only)
         self._first_page: List[List[int]] = [[0 for _ in self.groups] for _ in range(self.max_slots)]
 
     # -- sizes ------------------------------------------------------------
@@ -213,16 +214,18 @@ class SequenceCache:
         """Record that positions up to new_len are now written.  In a group with a window w the next
         token (at position new_len) sees keys from new_len - w + 1 on and every later token later ones,
         so pages that end before that position are given back at once: a long sequence holds about
-        w / 64 + 1 pages of such a group, not all of its positions."""
+        w / 64 + 1 pages of such a group, not all of its positions.  With chunks of n positions it sees keys from
+        its chunk's start on, a multiple of n."""
         self._held(slot)
         if -(-new_len // PAGE) > (len(self._pages[slot][0]) if self.groups else new_len):
             raise ValueError(f"slot {slot}: length {new_len} was not reserved")
         self._length[slot] = new_len
         for g in self.groups:
-            w = g.req.window
-            if w > 0:
+            w, chunk = g.req.window, g.req.chunk
+            if w > 0 or chunk > 0:
                 pg = self._pages[slot][g.gid]
-                keep_from = min(max(0, new_len - w + 1) // PAGE, len(pg))
+                first_seen = new_len - new_len % chunk if chunk > 0 else max(0, new_len - w + 1)
+                keep_from = min(first_seen // PAGE, len(pg))
                 for i in range(self._first_page[slot][g.gid], keep_from):
                     g.pool.give(pg[i])
                     pg[i] = RELEASED

@@ -20,6 +20,8 @@ from . import darusun as _darusun  # registers the architecture
 from .darusun import DarusunConfig
 from . import dibedra as _dibedra  # registers the architecture
 from .dibedra import DibedraConfig
+from . import nakurax as _nakurax  # registers the architecture
+from .nakurax import NakuraxConfig
 
 
 def read_config_json(folder: str) -> dict:

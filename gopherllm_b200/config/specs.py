@@ -162,6 +162,9 @@ class ModelSpec:
     pass_vectors: int = 0
     # an embedding of the pair (token before, token) added to the token's own; None: none
     pair_embedding: Optional[HashedPairSpec] = None
+    # residual streams a token has where they are more than the one (0): the embedding's output fills them all, the blocks
+    # work on [tokens, streams, hidden], and the final norm reads their sum
+    streams: int = 0
 
     def __post_init__(self):
         if self.position_table and self.position_table < self.max_positions:
@@ -169,6 +172,11 @@ class ModelSpec:
                              f"{self.max_positions} positions")
         if self.logit_softcap < 0 or not self.logit_scale > 0:
             raise ValueError("logit_softcap must be >= 0 and logit_scale > 0")
+        if self.streams < 0 or any((b.option("streams", 0) or 0) != self.streams for b in self.layers):
+            raise ValueError("every block works on as many residual streams as the model has")
+        if self.streams and (self.position_table or self.pair_embedding or self.embedding_norm or self.pass_vectors
+                             or any(e.enter is not None for e in self.schedule)):
+            raise ValueError("several residual streams come with a plain embedding and plain passes")
         for e in self.schedule:
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule names layer {e.layer}, model has {len(self.layers)}")
@@ -204,11 +212,11 @@ def default_schedule(num_layers: int) -> Tuple[ScheduleEntry, ...]:
     return tuple(ScheduleEntry(layer=i, cache=i) for i in range(num_layers))
 
 
-def looped_schedule(num_layers: int, start: int, stop: int, times: int) -> Tuple[ScheduleEntry, ...]:
+def looped_schedule(num_layers: int, start: int, stop: int, times: int, marked: bool = True) -> Tuple[ScheduleEntry, ...]:
     """Layers 0..start-1 once, then layers start..stop-1 ``times`` times in a row with the same weights,
     then the rest once.  Every run has a cache entry of its own (a pass never sees another pass's keys or
     state).  The first run of each pass is marked: pass t adds the model's pass vector t, and every pass
-    but the first adds the embedding's output before that."""
+    but the first adds the embedding's output before that.  ``marked`` False: nothing happens between passes."""
     if not (0 <= start <= stop <= num_layers) or times < 1:
         raise ValueError(f"loop over layers {start}..{stop} x {times} does not fit {num_layers} layers")
     runs = []
@@ -216,7 +224,7 @@ def looped_schedule(num_layers: int, start: int, stop: int, times: int) -> Tuple
         runs.append(ScheduleEntry(layer=i, cache=len(runs)))
     for t in range(times):
         for i in range(start, stop):
-            enter = PassEntry(index=t, add_embedding=t > 0) if i == start else None
+            enter = PassEntry(index=t, add_embedding=t > 0) if marked and i == start else None
             runs.append(ScheduleEntry(layer=i, cache=len(runs), enter=enter))
     for i in range(stop, num_layers):
         runs.append(ScheduleEntry(layer=i, cache=len(runs)))

@@ -8,7 +8,7 @@
 // the first kernel computes A for every pair (query head, value head) with a running maximum and
 // sum (a pair's scores come from the query head's own key head), the second mixes.  Without a table
 // the pairs are (g, c(g)) alone and the second kernel only converts.  A query at position p sees keys
-// lo..p, lo = 0 or p-window+1.
+// lo..p, lo = 0, p-window+1 or the start of p's chunk.
 //
 // A score may be shaped before the softmax: s = (q . k) * score_scale; with softcap > 0,
 // s <- softcap * tanh(s / softcap); with a slope per query head, s <- s - slope_h * (p - j) for the
@@ -41,6 +41,7 @@ struct MixedAttnArgs {
                               // without a table, query head g then takes the values of head g / (nH / nVH)
     int vs;                   // numbers between two positions' values of a head (0: vd).  A cache whose values are the
                               // first vd columns of its key rows is read with v_cache = k_cache and vs = hd
+    int chunk;                // > 0: a query sees the keys of its own chunk of positions alone (window is then 0)
 };
 
 __host__ __device__ __forceinline__ int am_value_stride(const MixedAttnArgs& a) { return a.vs > 0 ? a.vs : a.vd; }
@@ -93,10 +94,10 @@ attn_pairs_kernel(MixedAttnArgs a, int stage_rows) {
     const int idx = row0 + warp;
     const bool live = idx < qlen;
     const int p = ctx + idx;
-    const int lo = (a.window > 0 && p - a.window + 1 > 0) ? p - a.window + 1 : 0;
+    const int lo = gl_first_key(p, a.window, a.chunk);
     const int rows_here = min(AM_ROWS, qlen - row0);
     const int p_first = ctx + row0, p_last = ctx + row0 + rows_here - 1;
-    const int lo_cta = (a.window > 0 && p_first - a.window + 1 > 0) ? p_first - a.window + 1 : 0;
+    const int lo_cta = gl_first_key(p_first, a.window, a.chunk);
 
     float* qv = Qs + warp * hd;
     const float slope = a.slopes ? a.slopes[g] : 0.f;
@@ -191,7 +192,7 @@ attn_pairs_decode_kernel(MixedAttnArgs a) {
     const int nvh = am_value_heads(a);
     const int vh = a.mix ? blockIdx.x - g * nVal : g / (a.nH / nvh);
     const int p = a.seq_ctx[b];                         // the token's position; keys lo..p
-    const int lo = (a.window > 0 && p - a.window + 1 > 0) ? p - a.window + 1 : 0;
+    const int lo = gl_first_key(p, a.window, a.chunk);
     const int row = a.seq_qstart[b];
     const TA* qsrc = (const TA*)a.q + ((size_t)row * a.nH + g) * hd;
     const float slope = a.slopes ? a.slopes[g] : 0.f;
@@ -317,7 +318,7 @@ attn_group_decode_kernel(MixedAttnArgs a) {
     const int head0 = kh * group + (blockIdx.x - kh * chunks) * gq;      // this block's first query head
     const int nVal = a.mix ? a.nKV : 1;
     const int p = a.seq_ctx[b];
-    const int lo = (a.window > 0 && p - a.window + 1 > 0) ? p - a.window + 1 : 0;
+    const int lo = gl_first_key(p, a.window, a.chunk);
     const int row = a.seq_qstart[b];
     const int page_first = lo / GL_PAGE + split * a.pages_per_split;
     const int page_last = min(p / GL_PAGE, page_first + a.pages_per_split - 1);      // may lie before page_first: nothing to do
@@ -573,14 +574,14 @@ static int dispatch_mixed(const MixedAttnArgs& a, cudaStream_t stream) {
         case 6: return launch_mixed<TA, TC, 6>(a, stream);
         case 7: return launch_mixed<TA, TC, 7>(a, stream);
         case 8: return launch_mixed<TA, TC, 8>(a, stream);
-        default: return GL_ERR_SHAPE;
+        default: return a.vd <= 512 ? launch_mixed<TA, TC, 16>(a, stream) : GL_ERR_SHAPE;
     }
 }
 
 GL_API int gl_attention_mixed(const MixedAttnArgs* args, int act_dtype, int cache_dtype, cudaStream_t stream) {
     const MixedAttnArgs& a = *args;
     if (a.B <= 0 || a.max_qlen <= 0 || a.T <= 0) return GL_OK;
-    if (a.hd <= 0 || a.hd > 1024 || a.vd <= 0 || a.vd > 256 || a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV) return GL_ERR_SHAPE;
+    if (a.hd <= 0 || a.hd > 1024 || a.vd <= 0 || a.vd > 512 || a.chunk < 0 || a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV) return GL_ERR_SHAPE;
     if (a.nVH < 0 || (a.nVH > 0 && (a.nVH % a.nKV || a.nH % a.nVH || (a.mix && a.nVH != a.nKV)))) return GL_ERR_SHAPE;
     if (a.vs < 0 || (a.vs > 0 && a.vs < a.vd)) return GL_ERR_SHAPE;
     if (a.B > 65535 || a.nH * a.nKV > 65535) return GL_ERR_SHAPE;

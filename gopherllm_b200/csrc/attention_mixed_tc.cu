@@ -52,6 +52,7 @@ struct PairsArgs {
                               // are the first columns of its key rows is read with v_cache = k_cache and vs = the key size
     int v_in_k;               // such a cache with one row of values a key head: no value tile is fetched, the second
                               // product reads the key tile
+    int chunk;                // > 0: a query sees the keys of its own chunk of positions alone (window is then 0)
 };
 
 __device__ __forceinline__ unsigned ap_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -123,7 +124,7 @@ attn_pairs_tc_kernel(PairsArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int grp = lane >> 2, t = lane & 3;
     const int p_first = ctx + q0, p_last = ctx + q0 + rows - 1;
-    const int lo_first = (a.window > 0 && p_first - a.window + 1 > 0) ? p_first - a.window + 1 : 0;
+    const int lo_first = gl_first_key(p_first, a.window, a.chunk);
     const int page_begin = lo_first / GL_PAGE, page_end = p_last / GL_PAGE + 1;
     const int* pg = a.pages + (size_t)b * a.max_pages;
     const __nv_bfloat16* K = (const __nv_bfloat16*)a.k_cache;
@@ -164,8 +165,8 @@ attn_pairs_tc_kernel(PairsArgs a) {
     const float two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
     const int r_lo = warp * 16 + grp, r_hi = r_lo + 8;        // this thread's two rows inside the tile
     const int pos_lo = p_first + r_lo, pos_hi = p_first + r_hi;
-    const int wlo_lo = (a.window > 0 && pos_lo - a.window + 1 > 0) ? pos_lo - a.window + 1 : 0;
-    const int wlo_hi = (a.window > 0 && pos_hi - a.window + 1 > 0) ? pos_hi - a.window + 1 : 0;
+    const int wlo_lo = gl_first_key(pos_lo, a.window, a.chunk);
+    const int wlo_hi = gl_first_key(pos_hi, a.window, a.chunk);
 
     for (int p = page_begin; p < page_end; ++p) {
         const int st = (p - page_begin) & 1;
@@ -210,8 +211,8 @@ attn_pairs_tc_kernel(PairsArgs a) {
                     }
                 }
             }
-            // mask: a row at position x sees keys max(0, x-window+1) .. x
-            const bool need_mask = (j0 + GL_PAGE - 1 > p_first + warp * 16) || (a.window > 0 && j0 < wlo_hi + 8);
+            // mask: a row at position x sees keys gl_first_key(x) .. x (this thread's first key never lies behind its second's)
+            const bool need_mask = (j0 + GL_PAGE - 1 > p_first + warp * 16) || j0 < wlo_hi;
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
@@ -343,6 +344,7 @@ struct RowsDecodeArgs {
     float* ml;                // [B, nH, splits, 2] each range's maximum and sum
     int B, nH, nKV, nVH, max_pages, window, splits, pages_per_split, rows, v_in_k;
     float score_scale;
+    int chunk;
 };
 
 __global__ void __launch_bounds__(AP_THREADS)
@@ -358,7 +360,7 @@ attn_rows_decode_tc_kernel(RowsDecodeArgs a) {
     const int head0 = blockIdx.x * a.rows;
     const int kh = head0 / (a.nH / a.nKV), vh = head0 / (a.nH / a.nVH);
     const int p = a.seq_ctx[b];                                   // the token's position; keys lo..p
-    const int lo = (a.window > 0 && p - a.window + 1 > 0) ? p - a.window + 1 : 0;
+    const int lo = gl_first_key(p, a.window, a.chunk);
     const int page_first = lo / GL_PAGE + split * a.pages_per_split;
     const int page_last = min(p / GL_PAGE, page_first + a.pages_per_split - 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;

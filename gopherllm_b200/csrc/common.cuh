@@ -125,6 +125,16 @@ GL_API int gl_bounds_status(int* out4, int clear) {
 #define gl_checked(v, limit, kind) (v)
 #endif
 
+#ifdef __CUDACC__
+// The first position whose key a query at position p sees (it sees that one to p): all of them, the last ``window``
+// positions, or, with chunk > 0, the positions of its own chunk, chunks of that many positions counted from a
+// sequence's start.  Never decreases with p.
+__device__ __forceinline__ int gl_first_key(int p, int window, int chunk) {
+    if (chunk > 0) return p - p % chunk;
+    return (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+}
+#endif
+
 static inline int gl_check_launch() {
     return cudaGetLastError() == cudaSuccess ? GL_OK : GL_ERR_LAUNCH;
 }

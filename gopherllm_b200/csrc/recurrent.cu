@@ -604,7 +604,7 @@ __device__ __forceinline__ void mc_store16(__nv_bfloat16* dst, const float* v) {
 }
 
 // ---------------------------------------------------------------------------
-// Short causal convolution per channel with bias and silu.  The filter's last tap is the current
+// Short causal convolution per channel with bias and silu (or without an activation).  The filter's last tap is the current
 // token's; inputs before the run come from the sequence's state row (the last taps-1 inputs, oldest
 // first, zero at a sequence's start).  A second kernel then moves the run's last inputs into the row.
 // ---------------------------------------------------------------------------
@@ -619,6 +619,7 @@ struct ConvArgs {
     const int* seq_qstart;
     const int* seq_qlen;
     int T, B, C, taps, ld, x_off, state_stride, tail_off;
+    int silu;                 // 0: the sum as it is
 };
 
 template <typename TA>
@@ -639,7 +640,7 @@ conv_silu_kernel(ConvArgs a) {
         const float v = rel >= 0 ? gl_load((const TA*)a.x + (size_t)(t - back + j) * a.ld + a.x_off + c) : tail[rel + back];
         acc = fmaf(a.w[(size_t)c * a.taps + j], v, acc);
     }
-    gl_store((TA*)a.out + (size_t)t * a.C + c, rc_silu(acc));
+    gl_store((TA*)a.out + (size_t)t * a.C + c, a.silu ? rc_silu(acc) : acc);
 }
 
 // The same with 16 bytes of channels a thread (4 or 8 of them): columns, pitch and offset are whole pieces, and
@@ -677,8 +678,10 @@ conv_silu_wide_kernel(ConvArgs a) {
 #pragma unroll
         for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w[k * TAPS + j], v[k], acc[k]);
     }
+    if (a.silu) {
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) acc[k] = rc_silu(acc[k]);
+        for (int k = 0; k < VEC; ++k) acc[k] = rc_silu(acc[k]);
+    }
     mc_store16((TA*)a.out + (size_t)t * a.C + c0, acc);
 }
 
@@ -729,7 +732,7 @@ conv_silu_step_kernel(ConvArgs a) {
     }
     acc = fmaf(a.w[(size_t)c * a.taps + back], x, acc);
     if (back > 0) tail[back - 1] = x;
-    gl_store((TA*)a.out + (size_t)t * a.C + c, rc_silu(acc));
+    gl_store((TA*)a.out + (size_t)t * a.C + c, a.silu ? rc_silu(acc) : acc);
 }
 
 GL_API int gl_conv_silu(const ConvArgs* args, int act_dtype, cudaStream_t stream) {

@@ -6,12 +6,13 @@
 
 // ---------------------------------------------------------------------------
 // Embedding: out[t, :] = scale * table[tokens[t], :]          (model.go:2642-2651)
+// A model with several residual streams starts with ``copies`` equal ones: out [T, copies, D].
 // ---------------------------------------------------------------------------
 // (tokens, index, x below: what an earlier kernel of the step wrote is not declared restrict: loads through a
 // const restrict pointer count as loads of memory nobody writes, which the compiler may move above the wait)
 template <typename TW>
 __global__ void embed_kernel(const TW* __restrict__ table, const int* tokens,
-                             float* __restrict__ out, int D, int V, float scale) {
+                             float* __restrict__ out, int D, int V, float scale, int copies) {
     const int t = blockIdx.x;
     gl_grid_launch_dependents();
     gl_grid_wait();
@@ -19,20 +20,23 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* tokens,
     // ids are checked on the host; a bad id must still not read outside the table
     tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
     const TW* row = table + (size_t)tok * D;
-    float* o = out + (size_t)t * D;
-    for (int d = threadIdx.x; d < D; d += blockDim.x) o[d] = gl_load(row + d) * scale;
+    float* o = out + (size_t)t * D * copies;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const float v = gl_load(row + d) * scale;
+        for (int s = 0; s < copies; ++s) o[(size_t)s * D + d] = v;
+    }
 }
 
 GL_API int gl_embed(const void* table, int table_dtype, const int* tokens, float* out,
-                    int T, int D, int V, float scale, cudaStream_t stream) {
+                    int T, int D, int V, float scale, int copies, cudaStream_t stream) {
     if (T <= 0) return GL_OK;
-    if (D <= 0 || V <= 0) return GL_ERR_SHAPE;
+    if (D <= 0 || V <= 0 || copies <= 0) return GL_ERR_SHAPE;
     const int threads = D >= 1024 ? 256 : 128;
     if (table_dtype == GL_F32)
-        return gl_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, stream, 1, (const float*)table, tokens, out, D, V, scale);
+        return gl_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, stream, 1, (const float*)table, tokens, out, D, V, scale, copies);
     if (table_dtype == GL_BF16)
         return gl_launch(embed_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, 1,
-                         (const __nv_bfloat16*)table, tokens, out, D, V, scale);
+                         (const __nv_bfloat16*)table, tokens, out, D, V, scale, copies);
     return GL_ERR_DTYPE;
 }
 

@@ -51,6 +51,7 @@ class DecoderModel:
         self.positions: Optional[torch.Tensor] = None          # learned absolute positions, if the spec has them
         self.head_weight: Optional[torch.Tensor] = None
         self.head_bias: Optional[torch.Tensor] = None
+        self._ones: Optional[torch.Tensor] = None              # weights of a sum of all streams
         self._held: Dict[int, Dict[str, int]] = {}             # layer -> addresses of its tensors (see run)
 
     # -- parameters -------------------------------------------------------
@@ -93,6 +94,7 @@ class DecoderModel:
         self.pass_vectors = tensors["pass_vectors"] if self.spec.pass_vectors else None
         self.head_weight = self.embedding if self.spec.tie_embeddings else tensors["head/weight"]
         self.head_bias = tensors.get("head/bias")
+        self._ones = torch.ones(self.spec.streams, dtype=torch.float32, device=self.embedding.device) if self.spec.streams else None
         self._held = {}
 
     @property
@@ -161,7 +163,7 @@ class DecoderModel:
             x = ops.embed_pair(self.embedding, self.pair_embedding, ctx, last, pair.mul_prev, pair.mul_cur,
                                self.spec.embedding_scale)
         else:
-            x = ops.embed(self.embedding, ctx.tokens, self.spec.embedding_scale)
+            x = ops.embed(self.embedding, ctx.tokens, self.spec.embedding_scale, copies=self.spec.streams)
         if self.positions is not None:
             ops.add_rows(self.positions, ctx.tok_pos, x)
         if self.embedding_norm is not None:
@@ -171,6 +173,10 @@ class DecoderModel:
             # context (a captured step's context lives as long as its graphs)
             ctx.scratch["embedding_output"] = x
             x = x.clone()
+        if self.spec.streams and self.spec.schedule:
+            # a run's input is read from the streams by what comes before it; one buffer serves all runs
+            h = ops.empty((ctx.n_tokens, self.spec.hidden), ctx.act_dtype, x.device)
+            ctx.scratch["streams_input"] = ops.streams_read(x, *self.blocks[self.spec.schedule[0].layer].opening(), h=h)
         return x
 
     def run(self, x, ctx, cache, start: int, stop: int) -> None:
@@ -184,10 +190,16 @@ class DecoderModel:
         run's tensors in place of the recorded ones.  Runs that fork onto a second stream are left
         alone: their events are no launches."""
         repeat = ops.REPEAT_LAYERS and getattr(ctx, "side_stream", None) is None and stop - start > 2
-        kinds: List[list] = []            # [block, writes, view type, tape, pointers, state, tries]
-        for e in self.spec.schedule[start:stop]:
+        kinds: List[list] = []            # [block, (writes, view type, how it hands on), tape, pointers, state, tries]
+        for i in range(start, stop):
+            e = self.spec.schedule[i]
             view = cache.view(e.cache, e.writes) if e.cache is not None else None
             block = self.blocks[e.layer]
+            after = None
+            if self.spec.streams:                 # a block of several streams reads them for the run behind it
+                nxt = self.spec.schedule[i + 1].layer if i + 1 < len(self.spec.schedule) else None
+                ctx.next_block = self.blocks[nxt] if nxt is not None else None
+                after = None if nxt is None else (nxt == e.layer, ctx.next_block.opening()[2])
             if not getattr(block, "takes_rounded_stream", False) or e.enter is not None:
                 ctx.scratch.pop("stream_rounded", None)      # (a rounded copy of the stream a layer left for the next one)
             if e.enter is not None:
@@ -197,12 +209,15 @@ class DecoderModel:
                 block.forward(x, ctx, view)
                 continue
             ptrs = self._pointers(e.layer, view)
-            kind = next((k for k in kinds if type(k[0]) is type(block) and k[0].spec == block.spec
-                         and k[1] == e.writes and k[2] is type(view)), None)
-            if kind is not None and kind[5] == "repeat":
-                kind[3].repeat(ptrs)
+            if after is not None:
+                opening = ctx.next_block.opening()
+                ptrs = dict(ptrs, **{"next/in": opening[0].data_ptr(), "next/gamma": opening[1].data_ptr()})
+            how = (e.writes, type(view), after)
+            kind = next((k for k in kinds if type(k[0]) is type(block) and k[0].spec == block.spec and k[1] == how), None)
+            if kind is not None and kind[4] == "repeat":
+                kind[2].repeat(ptrs)
                 continue
-            if kind is not None and kind[5] == "own":
+            if kind is not None and kind[4] == "own":
                 block.forward(x, ctx, view)
                 continue
             tape = ops.LaunchTape().start()
@@ -211,16 +226,16 @@ class DecoderModel:
             finally:
                 tape.stop()
             if kind is None:
-                kinds.append([block, e.writes, type(view), tape, ptrs, "recorded", 0])
-            elif kind[3].same_as(tape, kind[4], ptrs):
-                kind[3].bind(kind[4])
-                kind[5] = "repeat"
+                kinds.append([block, how, tape, ptrs, "recorded", 0])
+            elif kind[2].same_as(tape, kind[3], ptrs):
+                kind[2].bind(kind[3])
+                kind[4] = "repeat"
             else:
                 # (the first run of a step may do what later ones find done: tables of the step's
                 # positions, say; so the later run becomes the one to compare with, a few times)
-                kind[3], kind[4], kind[6] = tape, ptrs, kind[6] + 1
-                if kind[6] >= 3:
-                    kind[5] = "own"
+                kind[2], kind[3], kind[5] = tape, ptrs, kind[5] + 1
+                if kind[5] >= 3:
+                    kind[4] = "own"
 
     def _pointers(self, layer: int, view) -> Dict[str, int]:
         """name -> address of every tensor block ``layer`` holds, and of the cache entry it runs on."""
@@ -237,11 +252,24 @@ class DecoderModel:
             ptrs.update(_tensor_addresses(view, "cache/"))
         return ptrs
 
+    def _norm_of_streams(self, x, ctx) -> torch.Tensor:
+        """The final norm of the sum of a token's streams, at the wanted places."""
+        norm = self.final_norm
+        if getattr(norm, "rms", False) and norm.fusable is not None and not norm.spec.bias:
+            gamma, _, eps, _ = norm.fusable()
+            h = ops.empty((ctx.n_want, self.spec.hidden), ctx.act_dtype, x.device)
+            return ops.streams_read(x, self._ones, gamma, eps, h, rows=ctx.want_rows)
+        total = ops.empty((ctx.n_want, self.spec.hidden), torch.float32, x.device)
+        return norm.forward(ops.streams_read(x, self._ones, None, 0.0, total, rows=ctx.want_rows), ctx.act_dtype)
+
     def finish(self, x, ctx) -> torch.Tensor:
         s = self.spec
         if ctx.n_want == 0:
             return torch.empty((0, s.vocab), dtype=torch.float32, device=x.device)
-        xn = self.final_norm.forward(x, ctx.act_dtype, rows=ctx.want_rows)
+        if s.streams:
+            xn = self._norm_of_streams(x, ctx)
+        else:
+            xn = self.final_norm.forward(x, ctx.act_dtype, rows=ctx.want_rows)
         logits = ops.linear(xn, self.head_weight, self.head_bias, out_dtype=torch.float32)
         if s.logit_scale != 1.0 or s.logit_softcap > 0.0:
             ops.scale_softcap(logits, s.logit_scale, s.logit_softcap)

@@ -42,6 +42,7 @@ class StepContext:
         self.n_tokens = self.n_seqs = self.n_want = 0
         self.max_qlen = self.max_len = 0
         self.is_decode = False
+        self.next_block = None           # the block of the run behind the current one (models of several residual streams)
         self.side_stream = None          # a second stream blocks may fork onto (decode steps only)
 
 

@@ -251,18 +251,18 @@ def _lib(source: str, defines=()):
 
 # ---------------------------------------------------------------------------
 def embed(table: torch.Tensor, tokens: torch.Tensor, scale: float = 1.0,
-          out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = scale * table[tokens[t]] as float32."""
+          out: Optional[torch.Tensor] = None, copies: int = 0) -> torch.Tensor:
+    """out[t] = scale * table[tokens[t]] as float32; with ``copies`` n > 0 n times, [T, n, D]."""
     _need(table, "table")
     _need(tokens, "tokens", torch.int32)
     V, D = table.shape
     T = tokens.numel()
     if out is None:
-        out = empty((T, D), torch.float32, table.device)
-    _need(out, "out", torch.float32, (T, D))
+        out = empty((T, copies, D) if copies else (T, D), torch.float32, table.device)
+    _need(out, "out", torch.float32, (T, copies, D) if copies else (T, D))
     fn = _lib("rowwise.cu").gl_embed
     _check(_launch(fn, _ptr(table), c_int(dtype_code(table.dtype)), _ptr(tokens), _ptr(out),
-              c_int(T), c_int(D), c_int(V), c_float(scale), _stream()), "embed")
+              c_int(T), c_int(D), c_int(V), c_float(scale), c_int(max(1, copies)), _stream()), "embed")
     return out
 
 
@@ -1294,12 +1294,12 @@ class _ConvArgs(Structure):
     _fields_ = [("x", c_void_p), ("out", c_void_p), ("w", c_void_p), ("bias", c_void_p), ("state", c_void_p),
                 ("tok_seq", c_void_p), ("seq_slot", c_void_p), ("seq_qstart", c_void_p), ("seq_qlen", c_void_p),
                 ("T", c_int), ("B", c_int), ("C", c_int), ("taps", c_int), ("ld", c_int), ("x_off", c_int),
-                ("state_stride", c_int), ("tail_off", c_int)]
+                ("state_stride", c_int), ("tail_off", c_int), ("silu", c_int)]
 
 
 def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, tail_off: int, ctx,
-              x_off: int = 0) -> torch.Tensor:
-    """silu of a causal per-channel convolution over columns x_off.. of ``x`` [T, ld]; ``w`` [C, taps] with the
+              x_off: int = 0, silu: bool = True) -> torch.Tensor:
+    """silu (``silu`` False: the sum itself) of a causal per-channel convolution over columns x_off.. of ``x`` [T, ld]; ``w`` [C, taps] with the
     current token's tap last.  The inputs before a run come from ``state`` (the last taps-1 inputs of each
     channel from column tail_off of the sequence's row on), which then takes the run's last inputs."""
     _need(x, "x")
@@ -1314,10 +1314,61 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], st
     out = empty((T, C), x.dtype, x.device)
     a = _ConvArgs(x.data_ptr(), out.data_ptr(), w.data_ptr(), _addr(bias), state.data_ptr(),
                   ctx.tok_seq.data_ptr(), ctx.seq_slot.data_ptr(), ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(),
-                  T, ctx.n_seqs, C, taps, ld, x_off, state.shape[1], tail_off)
+                  T, ctx.n_seqs, C, taps, ld, x_off, state.shape[1], tail_off, 1 if silu else 0)
     fn = _lib("recurrent.cu").gl_conv_silu
     _check(_launch(fn, byref(a), c_int(dtype_code(x.dtype)), _stream()), "conv_silu",
            2 if taps > 1 and T != ctx.n_seqs else 1)
+    return out
+
+
+# ---------------------------------------------------------------------------
+# A real-gated linear recurrent unit (csrc/gated_unit.cu)
+class _UnitGatesArgs(Structure):
+    _fields_ = [("u", c_void_p), ("w", c_void_p), ("bias", c_void_p), ("rate", c_void_p), ("ab", c_void_p),
+                ("y", c_void_p), ("out", c_void_p), ("state", c_void_p), ("tok_seq", c_void_p), ("seq_slot", c_void_p),
+                ("T", c_int), ("C", c_int), ("blocks", c_int), ("y_ld", c_int), ("y_off", c_int), ("state_stride", c_int),
+                ("step", c_int)]
+
+
+class _UnitScanArgs(Structure):
+    _fields_ = [("ab", c_void_p), ("y", c_void_p), ("out", c_void_p), ("state", c_void_p), ("seq_slot", c_void_p),
+                ("seq_qstart", c_void_p), ("seq_qlen", c_void_p),
+                ("B", c_int), ("C", c_int), ("y_ld", c_int), ("y_off", c_int), ("state_stride", c_int)]
+
+
+def gated_unit(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor, y_off: int,
+               state: torch.Tensor, ctx) -> torch.Tensor:
+    """A diagonal recurrence whose decay the input sets.  u [T, C] falls into blocks of C / blocks channels; ``w``
+    [blocks, 2 * size, size] and ``bias`` [2 * C] float32 hold both gates' rows channel by channel (r, then i);
+    r, i = sigmoid(w u + bias), a = e^(rate r) (``rate`` [C] float32, not positive), S <- a S + sqrt(1 - a^2) i u.
+    Returns S * gelu(y) (tanh form), y the C columns y_off.. of its tensor, [T, C] in u's type; S [C] stands first in the
+    sequences' rows of ``state``."""
+    _need(u, "u")
+    T, C = u.shape
+    _need(w, "w")
+    blocks, rows, size = w.shape
+    if blocks * size != C or rows != 2 * size:
+        raise KernelError(f"gated_unit: matrices {tuple(w.shape)} do not fit {C} channels")
+    _need(bias, "bias", torch.float32, (2 * C,))
+    _need(rate, "rate", torch.float32, (C,))
+    _need(y, "y", u.dtype)
+    if y.shape[0] != T or y_off < 0 or y_off + C > y.shape[1]:
+        raise KernelError("gated_unit: the other branch's columns do not fit its rows")
+    _need(state, "state", torch.float32)
+    if state.shape[1] < C:
+        raise KernelError("gated_unit: the state row is too small")
+    out = empty((T, C), u.dtype, u.device)
+    step = ctx.max_qlen == 1
+    ab = None if step else empty((T, C, 2), torch.float32, u.device)
+    lib = _lib("gated_unit.cu")
+    g = _UnitGatesArgs(u.data_ptr(), w.data_ptr(), bias.data_ptr(), rate.data_ptr(), _addr(ab), y.data_ptr(), out.data_ptr(),
+                       state.data_ptr(), ctx.tok_seq.data_ptr(), ctx.seq_slot.data_ptr(), T, C, blocks, y.shape[1], y_off,
+                       state.shape[1], 1 if step else 0)
+    _check(_launch(lib.gl_unit_gates, byref(g), c_int(dtype_code(u.dtype)), c_int(dtype_code(w.dtype)), _stream()), "unit_gates")
+    if not step:
+        s = _UnitScanArgs(ab.data_ptr(), y.data_ptr(), out.data_ptr(), state.data_ptr(), ctx.seq_slot.data_ptr(),
+                          ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.n_seqs, C, y.shape[1], y_off, state.shape[1])
+        _check(_launch(lib.gl_unit_scan, byref(s), c_int(dtype_code(u.dtype)), _stream()), "unit_scan")
     return out
 
 
@@ -1443,7 +1494,7 @@ class _MixedAttnArgs(Structure):
                 ("max_pages", c_int), ("window", c_int), ("max_qlen", c_int), ("n_pages", c_int),
                 ("parts", c_void_p), ("ml", c_void_p), ("splits", c_int), ("pages_per_split", c_int),
                 ("score_scale", c_float), ("softcap", c_float), ("slopes", c_void_p), ("sinks", c_void_p), ("nVH", c_int),
-                ("vs", c_int)]
+                ("vs", c_int), ("chunk", c_int)]
 
 
 # A block of the one-token kernel walks its pages one after the other and waits for each: what hides the trips to
@@ -1466,7 +1517,7 @@ class _PairsArgs(Structure):
                 ("seq_qstart", c_void_p), ("seq_qlen", c_void_p), ("seq_ctx", c_void_p), ("pages", c_void_p),
                 ("B", c_int), ("nH", c_int), ("nKV", c_int), ("nVal", c_int), ("max_pages", c_int), ("window", c_int),
                 ("max_qlen", c_int), ("score_scale", c_float), ("softcap", c_float), ("slopes", c_void_p),
-                ("out", c_void_p), ("sinks", c_void_p), ("nVH", c_int), ("vs", c_int), ("v_in_k", c_int)]
+                ("out", c_void_p), ("sinks", c_void_p), ("nVH", c_int), ("vs", c_int), ("v_in_k", c_int), ("chunk", c_int)]
 
 
 USE_PAIRS_TC = True
@@ -1477,7 +1528,7 @@ class _RowsDecodeArgs(Structure):
     _fields_ = [("q", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("seq_qstart", c_void_p), ("seq_ctx", c_void_p),
                 ("pages", c_void_p), ("parts", c_void_p), ("ml", c_void_p),
                 ("B", c_int), ("nH", c_int), ("nKV", c_int), ("nVH", c_int), ("max_pages", c_int), ("window", c_int),
-                ("splits", c_int), ("pages_per_split", c_int), ("rows", c_int), ("v_in_k", c_int), ("score_scale", c_float)]
+                ("splits", c_int), ("pages_per_split", c_int), ("rows", c_int), ("v_in_k", c_int), ("score_scale", c_float), ("chunk", c_int)]
 
 
 def rows_decode_smem(head_dim: int, value_dim: int, values_in_keys: bool) -> int:
@@ -1498,7 +1549,8 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
                     mix: Optional[torch.Tensor] = None, window: int = 0, score_scale: float = 1.0,
                     softcap: float = 0.0, slopes: Optional[torch.Tensor] = None,
-                    sinks: Optional[torch.Tensor] = None, value_heads: int = 0, values_in_keys: bool = False) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, value_heads: int = 0, values_in_keys: bool = False,
+                    chunk: int = 0) -> torch.Tensor:
     """Causal softmax attention of scaled queries [T, nH*hd] over the paged cache; with ``mix`` [nH, nH]
     head h applies sum_g mix[h, g] * (head g's softmax weights) to the values of its own key/value
     head.  A score is (q . k) * score_scale, then softcap * tanh(score / softcap) when softcap > 0, then
@@ -1507,7 +1559,8 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     ``value_heads`` > 0: the value cache has that many heads (a multiple of the key heads), and without a table
     query head h takes the values of head h / (nH / value_heads): many query heads on one wide key head, each
     with one of several value heads.  ``values_in_keys``: a position's values are the first ``value_dim`` numbers of its
-    key row (``v_cache`` is the key cache).
+    key row (``v_cache`` is the key cache).  ``chunk`` n > 0 (with window 0): a query sees the keys of its own chunk of
+    n positions alone, chunks counted from a sequence's start.
     Returns [T, nH*vd] in q's type.  Prompts in bfloat16 with key and value sizes that are
     multiples of 16 compute the (query head, value head) pairs on the tensor cores (a library per pair
     of sizes); everything else runs the 32-bit kernels."""
@@ -1520,8 +1573,14 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         _need(slopes, "slopes", torch.float32, (num_heads,))
     if sinks is not None:
         _need(sinks, "sinks", torch.float32, (num_heads,))
+    if chunk < 0 or (chunk > 0 and window > 0):
+        raise KernelError("attention_mixed: keys are limited by a window or by chunks, not by both")
     n_val = num_kv_heads if mix is not None else 1
     nvh = int(value_heads)
+    # pages a token's keys can lie on
+    span = max(1, -(-int(ctx.max_len) // PAGE))
+    if window > 0 or chunk > 0:
+        span = min(span, -(-(window or chunk) // PAGE) + 1)
     if nvh and (nvh % num_kv_heads or num_heads % nvh or (mix is not None and nvh != num_kv_heads)):
         raise KernelError(f"attention_mixed: {nvh} value heads do not fit {num_heads} query heads on {num_kv_heads} key heads")
     vs = 0
@@ -1541,7 +1600,7 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         p = _PairsArgs(q.data_ptr(), None, k_cache.data_ptr(), v_cache.data_ptr(),
                        ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.seq_ctx.data_ptr(), pages.data_ptr(),
                        ctx.n_seqs, num_heads, num_kv_heads, 1, pages.shape[-1], window, ctx.max_qlen,
-                       score_scale, softcap, _addr(slopes), out.data_ptr(), _addr(sinks), nvh, vs, 1 if values_in_keys else 0)
+                       score_scale, softcap, _addr(slopes), out.data_ptr(), _addr(sinks), nvh, vs, 1 if values_in_keys else 0, chunk)
         fn = _lib("attention_mixed_tc.cu", catalog.pair_dim_defines(head_dim, value_dim)).gl_attention_pairs_tc
         _check(_launch(fn, byref(p), _stream()), "attention_pairs_tc")
         return out
@@ -1549,19 +1608,18 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     a = _MixedAttnArgs(q.data_ptr(), pairs.data_ptr(), out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _addr(mix),
                        ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.seq_ctx.data_ptr(), pages.data_ptr(),
                        T, ctx.n_seqs, num_heads, num_kv_heads, head_dim, value_dim, pages.shape[-1], window,
-                       ctx.max_qlen, k_cache.shape[0], None, None, 0, 0, score_scale, softcap, _addr(slopes), _addr(sinks), nvh, vs)
+                       ctx.max_qlen, k_cache.shape[0], None, None, 0, 0, score_scale, softcap, _addr(slopes), _addr(sinks), nvh, vs,
+                       chunk)
     group, share = num_heads // num_kv_heads, num_heads // (nvh or num_kv_heads)
-    rows = min(share, 16)
+    # query heads that share a value head, in equal runs of up to sixteen
+    rows = max(n for n in range(1, 17) if share % n == 0)
     if (USE_ROWS_DECODE_TC and ctx.max_qlen == 1 and mix is None and softcap == 0.0 and slopes is None and not DEBUG_BOUNDS
             and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and head_dim % 16 == 0 and value_dim % 16 == 0
-            and head_dim <= 256 and value_dim <= 256 and group >= 8 and rows >= 4 and share % rows == 0
+            and head_dim <= 256 and value_dim <= 256 and (group >= 8 or values_in_keys) and rows >= 4
             and rows_decode_smem(head_dim, value_dim, values_in_keys) <= 227 * 1024):
         # one token a sequence and many query heads on a key head: runs of heads that share a value head are the rows
         # of a tensor-core product over the key head's pages; the ranges are put together by the mixing kernel
         smem = rows_decode_smem(head_dim, value_dim, values_in_keys)
-        span = max(1, -(-int(ctx.max_len) // PAGE))          # pages a token's keys can lie on
-        if window > 0:
-            span = min(span, -(-window // PAGE) + 1)
         splits = rows_decode_splits(ctx.n_seqs, num_heads // rows, span, q.device, smem)
         a.splits = splits
         a.pages_per_split = -(-span // splits)
@@ -1571,7 +1629,7 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         r = _RowsDecodeArgs(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), ctx.seq_qstart.data_ptr(),
                             ctx.seq_ctx.data_ptr(), pages.data_ptr(), parts.data_ptr(), ml.data_ptr(), ctx.n_seqs, num_heads,
                             num_kv_heads, nvh or num_kv_heads, pages.shape[-1], window, splits, a.pages_per_split, rows,
-                            1 if values_in_keys else 0, score_scale)
+                            1 if values_in_keys else 0, score_scale, chunk)
         fn = _lib("attention_mixed_tc.cu", catalog.pair_dim_defines(head_dim, value_dim)).gl_attention_rows_decode_tc
         _check(_launch(fn, byref(r), _stream()), "attention_rows_decode_tc")
         _check(_launch(_lib("attention_mixed.cu").gl_head_mix_split, byref(a), c_int(dtype_code(q.dtype)), _stream()), "head_mix_split")
@@ -1585,9 +1643,9 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     if ctx.max_qlen == 1 and by_key_head and value_dim <= 128:
         # one token a sequence: the context in ranges of pages, a block each (sized for the step's longest
         # sequence; a captured step is sized for its bucket's longest), put together by the mixing kernel
-        splits = mixed_decode_splits(ctx.n_seqs, num_kv_heads * max(1, group // 8), ctx.max_len, q.device)
+        splits = mixed_decode_splits(ctx.n_seqs, num_kv_heads * max(1, group // 8), span * PAGE, q.device)
         a.splits = splits
-        a.pages_per_split = -(-max(1, -(-int(ctx.max_len) // PAGE)) // splits)
+        a.pages_per_split = -(-span // splits)
         parts = empty((ctx.n_seqs, num_heads, n_val, splits, value_dim), torch.float32, q.device)
         ml = empty((ctx.n_seqs, num_heads, splits, 2), torch.float32, q.device)
         a.parts, a.ml = parts.data_ptr(), ml.data_ptr()
@@ -1596,7 +1654,7 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         p = _PairsArgs(q.data_ptr(), pairs.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                        ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.seq_ctx.data_ptr(), pages.data_ptr(),
                        ctx.n_seqs, num_heads, num_kv_heads, n_val, pages.shape[-1], window, ctx.max_qlen,
-                       score_scale, softcap, _addr(slopes), None, _addr(sinks), nvh, vs, 0)
+                       score_scale, softcap, _addr(slopes), None, _addr(sinks), nvh, vs, 0, chunk)
         fn = _lib("attention_mixed_tc.cu", catalog.pair_dim_defines(head_dim, value_dim)).gl_attention_pairs_tc
         _check(_launch(fn, byref(p), _stream()), "attention_pairs_tc")
         _check(_launch(lib.gl_head_mix, byref(a), c_int(dtype_code(q.dtype)), _stream()), "head_mix")
@@ -1667,14 +1725,14 @@ class _LatentPrepareArgs(Structure):
 
 
 def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, ctx, pages: torch.Tensor,
-                   q_rank: int, kv_rank: int, rot: int, q_gamma: torch.Tensor, kv_gamma: torch.Tensor, eps: float,
+                   q_rank: int, kv_rank: int, rot: int, q_gamma: Optional[torch.Tensor], kv_gamma: torch.Tensor, eps: float,
                    cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], interleaved: bool,
-                   write_kv: bool = True) -> torch.Tensor:
+                   write_kv: bool = True) -> Optional[torch.Tensor]:
     """A token's down projections proj [T, ld] = [query latent (q_rank) | c (kv_rank) | key part (rot) | ...]: both
     latents RMS-normed with their weights (32-bit), the key part rotated by the token's angles; the row [c | key part]
     goes to the token's place in k_cache [pages, 1, PAGE, kv_rank + rot], c to v_cache [pages, 1, PAGE, kv_rank]
     (``v_cache`` None or the key cache itself: the values are read from the key rows, nothing more is written).
-    Returns the normed query latent [T, q_rank]."""
+    Returns the normed query latent [T, q_rank] (``q_rank`` 0: there is none, None)."""
     _need(proj, "proj")
     T, ld = proj.shape
     if ld < q_rank + kv_rank + rot:
@@ -1683,14 +1741,15 @@ def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         v_cache = None
     if tuple(k_cache.shape[1:]) != (1, PAGE, kv_rank + rot) or (v_cache is not None and tuple(v_cache.shape[1:]) != (1, PAGE, kv_rank)):
         raise KernelError(f"cache pages do not fit: keys {tuple(k_cache.shape)}, values {tuple(v_cache.shape)}")
-    _need(q_gamma, "q_gamma", torch.float32, (q_rank,))
+    if q_rank:
+        _need(q_gamma, "q_gamma", torch.float32, (q_rank,))
     _need(kv_gamma, "kv_gamma", torch.float32, (kv_rank,))
     if cos is not None:
         _need(cos, "cos", torch.float32, (T, rot // 2))
         _need(sin, "sin", torch.float32, (T, rot // 2))
-    cq = empty((T, q_rank), proj.dtype, proj.device)
-    a = _LatentPrepareArgs(proj.data_ptr(), cq.data_ptr(), k_cache.data_ptr(), _addr(v_cache), _addr(cos), _addr(sin),
-                           q_gamma.data_ptr(), kv_gamma.data_ptr(), ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(),
+    cq = empty((T, q_rank), proj.dtype, proj.device) if q_rank else None
+    a = _LatentPrepareArgs(proj.data_ptr(), _addr(cq), k_cache.data_ptr(), _addr(v_cache), _addr(cos), _addr(sin),
+                           _addr(q_gamma), kv_gamma.data_ptr(), ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(),
                            pages.data_ptr(), T, ld, q_rank, kv_rank, rot, pages.shape[-1], k_cache.shape[0],
                            1 if interleaved else 0, 1 if write_kv else 0, eps)
     _check(_launch(_lib("latent.cu").gl_latent_prepare, byref(a), c_int(dtype_code(proj.dtype)),
@@ -1707,16 +1766,16 @@ class _HeadLinearArgs(Structure):
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, x_head: int, tail: int = 0, cos: Optional[torch.Tensor] = None,
                 sin: Optional[torch.Tensor] = None, interleaved: bool = False, gate: Optional[torch.Tensor] = None,
-                gate_off: int = 0) -> torch.Tensor:
-    """A product per head: out[t, h, :N] = w[h] x[t, h, :K] for x [T, H * x_head] (head h's K inputs start at column
-    h * x_head) and w [H, N, K].  ``tail`` > 0: the columns x[t, h, K:K + tail] are copied behind the result, turned by
+                gate_off: int = 0, x_off: int = 0) -> torch.Tensor:
+    """A product per head: out[t, h, :N] = w[h] x[t, h, :K] for rows x [T, >= x_off + H * x_head] (head h's K inputs start
+    at column x_off + h * x_head) and w [H, N, K].  ``tail`` > 0: the columns x[t, h, K:K + tail] are copied behind the result, turned by
     the token's angles when cos/sin [T, tail / 2] are given; out is [T, H * (N + tail)].  ``gate`` [T, ld]: the result
     of head h is multiplied by sigmoid(gate[t, gate_off + h])."""
     _need(x, "x")
     _need(w, "w")
     T = x.shape[0]
     H, N, K = w.shape
-    if x.shape[1] != H * x_head or K + tail > x_head:
+    if x_off < 0 or x.shape[1] < x_off + H * x_head or K + tail > x_head:
         raise KernelError(f"head_linear: x {tuple(x.shape)} does not hold {H} heads of {K} + {tail} columns")
     if cos is not None:
         _need(cos, "cos", torch.float32, (T, tail // 2))
@@ -1729,7 +1788,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, x_head: int, tail: int = 0, co
             raise KernelError("head_linear: the gate's rows do not hold a column for every head")
     out = empty((T, H * (N + tail)), x.dtype, x.device)
     a = _HeadLinearArgs(x.data_ptr(), w.data_ptr(), out.data_ptr(), _addr(gate), _addr(cos), _addr(sin), T, H, N, K,
-                        x.shape[1], x_head, 0, H * (N + tail), N + tail, 0, g_row, gate_off, tail, 1 if interleaved else 0)
+                        x.shape[1], x_head, x_off, H * (N + tail), N + tail, 0, g_row, gate_off, tail, 1 if interleaved else 0)
     _check(_launch(_lib("latent.cu").gl_head_linear, byref(a), c_int(dtype_code(x.dtype)), c_int(dtype_code(w.dtype)),
                    _stream()), "head_linear")
     return out
@@ -1981,6 +2040,62 @@ def enter_pass(x: torch.Tensor, base: Optional[torch.Tensor], table: Optional[to
     fn = _lib("rowwise.cu").gl_enter_pass
     _check(_launch(fn, _ptr(x), _ptr(base), _ptr(table), c_int(T), c_int(D), c_int(row), _stream()), "enter_pass")
     return x
+
+
+class _StreamArgs(Structure):
+    _fields_ = [("x", c_void_p), ("a", c_void_p), ("b", c_void_p), ("mix", c_void_p), ("out_share", c_void_p),
+                ("in_share", c_void_p), ("gamma", c_void_p), ("h", c_void_p), ("rows", c_void_p),
+                ("R", c_int), ("S", c_int), ("W", c_int), ("fa", c_float), ("fb", c_float), ("eps", c_float)]
+
+
+MAX_STREAMS = 16         # ST_MAX_STREAMS
+
+
+def streams_read(x: torch.Tensor, in_share: torch.Tensor, gamma: Optional[torch.Tensor], eps: float, h: torch.Tensor,
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """h = u / sqrt(mean(u^2) + eps) * gamma (``gamma`` None: u itself) with u = sum_s in_share[s] x[:, s], for float32
+    streams x [T, S, W]; ``rows`` picks tokens."""
+    return _streams(x, None, None, None, None, in_share, gamma, eps, h, rows)
+
+
+def streams_join(x: torch.Tensor, branches, mix: torch.Tensor, out_share: torch.Tensor, in_share: Optional[torch.Tensor] = None,
+                 gamma: Optional[torch.Tensor] = None, eps: float = 0.0, h: Optional[torch.Tensor] = None) -> None:
+    """A sublayer's result joins the streams, x [T, S, W] in place: x_t <- sum_s mix[s, t] x_s + out_share[t] y with y the
+    sum of ``branches``, one or two (float32 [T, W], factor).  With ``in_share`` the same pass reads the new streams for
+    the next sublayer into ``h`` (see streams_read)."""
+    branches = list(branches)
+    if not 1 <= len(branches) <= 2:
+        raise KernelError("streams_join takes one branch or two")
+    _streams(x, branches[0], branches[1] if len(branches) > 1 else None, mix, out_share, in_share, gamma, eps, h, None)
+
+
+def _streams(x, first, second, mix, out_share, in_share, gamma, eps, h, rows):
+    _need(x, "x", torch.float32)
+    if x.dim() != 3:
+        raise KernelError(f"streams [tokens, streams, width] expected, got {tuple(x.shape)}")
+    T, S, W = x.shape
+    for n, t in (("branch", first), ("second branch", second)):
+        if t is not None:
+            _need(t[0], n, torch.float32, (T, W))
+    if first is not None:
+        _need(mix, "mix", torch.float32, (S, S))
+        _need(out_share, "out_share", torch.float32, (S,))
+    R = T
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+        R = rows.numel()
+    if in_share is not None:
+        _need(in_share, "in_share", torch.float32, (S,))
+        _need(h, "h", shape=(R, W))
+        if gamma is not None:
+            _need(gamma, "gamma", torch.float32, (W,))
+    a = _StreamArgs(x.data_ptr(), first[0].data_ptr() if first else None, second[0].data_ptr() if second else None,
+                    _addr(mix), _addr(out_share), _addr(in_share), _addr(gamma) if in_share is not None else None,
+                    _addr(h) if in_share is not None else None, _addr(rows), R, S, W, first[1] if first else 0.0,
+                    second[1] if second else 0.0, eps)
+    _check(_launch(_lib("streams.cu").gl_streams, byref(a), c_int(dtype_code(h.dtype) if in_share is not None else F32), _stream()),
+           "streams")
+    return h
 
 
 def rms_norm_pair(x: torch.Tensor, g1: torch.Tensor, g2: torch.Tensor, eps: float, out_dtype: torch.dtype):

@@ -189,7 +189,8 @@ class MixedHeadAttention(Mixer):
     rotation every head of q and of k is divided by its own root mean square (``norm_eps`` inside the root, no
     weight).  ``sink``: a learned score per head ("sink" [heads]) whose exponential joins the softmax's
     denominator once, with no key and no value, unscaled.  ``out_bias``: the output projection has a bias.
-    ``spec.window`` w > 0: a query sees itself and the w - 1 positions before it.
+    ``spec.window`` w > 0: a query sees itself and the w - 1 positions before it.  ``chunk`` n > 0 (window 0 then): a
+    query at position p sees the positions from n floor(p / n) on to its own.
     ``talk_scores``: a learned table T ("talk" [heads, heads]) mixes the heads' SCORES before the softmax,
     s'_h = sum_g T[h, g] s_g, and head h applies its own softmax of s'_h to the values of its own key/value head.
     The sum is taken on the queries: with q'_h,c = sum of T[h, g] q_g over the query heads g of key head c,
@@ -209,13 +210,13 @@ class MixedHeadAttention(Mixer):
         self.vdim = spec.value_dim or spec.head_dim
         self.talk_scores = bool(spec.option("talk_scores", False))
         if self.talk_scores:
-            if spec.head_dim * spec.num_kv_heads > 1024 or self.vdim > 256:
+            if spec.head_dim * spec.num_kv_heads > 1024 or self.vdim > 512:
                 raise ValueError(f"{spec.num_kv_heads} key heads of {spec.head_dim} side by side exceed what the attention "
-                                 f"kernels take (1024), or values of {self.vdim} do (256)")
+                                 f"kernels take (1024), or values of {self.vdim} do (512)")
             if spec.option("talk", False):
                 raise ValueError("a table mixes the heads' scores or their softmax weights, not both")
-        elif spec.head_dim > 256 or self.vdim > 256:
-            raise ValueError(f"head sizes {spec.head_dim}/{self.vdim} exceed what the attention kernels take (256)")
+        elif spec.head_dim > 1024 or self.vdim > 512:
+            raise ValueError(f"head sizes {spec.head_dim}/{self.vdim} exceed what the attention kernels take (1024/512)")
         scope = spec.option("qk_norm", None)
         if scope not in (None, "projection", "head_unit"):
             raise ValueError(f"qk_norm {scope!r}: this mixer norms over the whole projection, every head to unit "
@@ -224,6 +225,9 @@ class MixedHeadAttention(Mixer):
         self.head_unit = scope == "head_unit"
         self.sink = bool(spec.option("sink", False))
         self.out_bias = bool(spec.option("out_bias", False))
+        self.chunk = int(spec.option("chunk", 0))
+        if self.chunk < 0 or (self.chunk and spec.window):
+            raise ValueError("keys are limited by a window or by chunks of positions, not by both")
         self.talk = bool(spec.option("talk", False))
         self.eps = float(spec.option("norm_eps", 1e-6))
         self.position = build_position(spec.position)
@@ -294,8 +298,9 @@ class MixedHeadAttention(Mixer):
         if self.talk_scores:
             wide = s.num_kv_heads * s.head_dim
             return KVRequest(1, wide, s.window, value_dim=0 if self.vdim == wide else self.vdim,
-                             value_heads=0 if s.num_kv_heads == 1 else s.num_kv_heads)
-        return KVRequest(s.num_kv_heads, s.head_dim, s.window, value_dim=0 if self.vdim == s.head_dim else self.vdim)
+                             value_heads=0 if s.num_kv_heads == 1 else s.num_kv_heads, chunk=self.chunk)
+        return KVRequest(s.num_kv_heads, s.head_dim, s.window, value_dim=0 if self.vdim == s.head_dim else self.vdim,
+                         chunk=self.chunk)
 
     def products(self):
         return [("qkv", self.w_qkv, self.b_qkv, None), ("o", self.w_out, self.b_out, None)]
@@ -320,7 +325,7 @@ class MixedHeadAttention(Mixer):
             o = ops.attention_mixed(q, cache.k, cache.v, ctx, pages, s.num_heads, 1, s.num_kv_heads * s.head_dim,
                                     self.vdim, mix=None, window=s.window, score_scale=self.score_scale,
                                     softcap=self.softcap, slopes=self.slopes, sinks=self.sinks,
-                                    value_heads=s.num_kv_heads)
+                                    value_heads=s.num_kv_heads, chunk=self.chunk)
             return o, self.w_out, self.b_out
         q = ops.qkv_rownorm_to_cache(qkv, cache.k, cache.v, ctx, pages, s.num_heads, s.num_kv_heads, s.head_dim,
                                      self.vdim, s.q_scale, cos, sin, s.position.interleaved,
@@ -328,7 +333,7 @@ class MixedHeadAttention(Mixer):
                                      q_temp=self.q_temp, q_only=self.shared_kv, head_unit=self.head_unit)
         o = ops.attention_mixed(q, cache.k, cache.v, ctx, pages, s.num_heads, s.num_kv_heads, s.head_dim, self.vdim,
                                 mix=self.mix, window=s.window, score_scale=self.score_scale, softcap=self.softcap,
-                                slopes=self.slopes, sinks=self.sinks)
+                                slopes=self.slopes, sinks=self.sinks, chunk=self.chunk)
         return o, self.w_out, self.b_out
 
     def forward(self, xn, ctx, cache, add: Sequence[torch.Tensor], out=None) -> torch.Tensor:
@@ -354,8 +359,8 @@ class LatentAttention(Mixer):
     every query head becomes a row [W_uk,h^T q_h | its rotated part] of kv_rank + rot numbers, attention runs as
     ``num_heads`` query heads on ONE key head with values of size kv_rank, and W_uv,h is applied to a head's result.
     The three down projections (query latent, [c' | k_r], gates) are one product; the per-head products are
-    csrc/latent.cu's.  Options: ``q_rank``, ``kv_rank``, ``rot`` (the position encoding's rotary size),
-    ``score_scale``, ``norm_eps``, ``sink``, ``gate``."""
+    csrc/latent.cu's.  Options: ``q_rank`` (0: there is no query latent, q = W_q x, and its rows ride in the first product),
+    ``kv_rank``, ``rot`` (the position encoding's rotary size), ``score_scale``, ``norm_eps``, ``sink``, ``gate``."""
 
     deferred_add = True
     capturable = True
@@ -363,15 +368,16 @@ class LatentAttention(Mixer):
 
     def __init__(self, spec: MixerSpec):
         self.spec = spec
-        self.q_rank, self.kv_rank = int(spec.option("q_rank")), int(spec.option("kv_rank"))
+        self.q_rank, self.kv_rank = int(spec.option("q_rank", 0)), int(spec.option("kv_rank"))
         self.rot = int(spec.option("rot", 0))
         self.vdim = spec.value_dim or spec.head_dim
-        if min(self.q_rank, self.kv_rank, spec.num_heads, spec.head_dim, self.vdim) < 1 or self.rot < 0 or self.rot % 2:
+        if (min(self.kv_rank, spec.num_heads, spec.head_dim, self.vdim) < 1 or self.q_rank < 0 or self.rot < 0
+                or self.rot % 2):
             raise ValueError("latent attention: ranks, heads and head sizes are positive, the rotated part is even")
         if spec.position.kind != "none" and spec.position.rotary_dim != self.rot:
             raise ValueError("latent attention: the rotation covers the rotated part exactly")
-        if self.kv_rank + self.rot > 1024 or self.kv_rank > 256:
-            raise ValueError(f"a latent of {self.kv_rank} + {self.rot} exceeds what the attention kernels take (256 + 768)")
+        if self.kv_rank + self.rot > 1024 or self.kv_rank > 512:
+            raise ValueError(f"a latent of {self.kv_rank} + {self.rot} exceeds what the attention kernels take (512, 1024 in all)")
         self.sink = bool(spec.option("sink", False))
         self.gate = bool(spec.option("gate", False))
         self.eps = float(spec.option("norm_eps", 1e-6))
@@ -379,15 +385,21 @@ class LatentAttention(Mixer):
         self.position = build_position(spec.position)
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_out = None
         self.q_gamma = self.kv_gamma = self.sinks = None
+        self.q_off = self.gate_off = 0           # columns of the first product: queries (without a query latent), gates
 
     def parameters(self) -> Dict[str, ParamSpec]:
         s, H = self.spec, self.spec.num_heads
-        p = {"dq.weight": ParamSpec((self.q_rank, s.hidden)), "dq.norm.weight": ParamSpec((self.q_rank,), "vector", "gamma"),
-             "uq.weight": ParamSpec((H * (s.head_dim + self.rot), self.q_rank)),
+        wide = H * (s.head_dim + self.rot)
+        if self.q_rank:
+            p = {"dq.weight": ParamSpec((self.q_rank, s.hidden)), "dq.norm.weight": ParamSpec((self.q_rank,), "vector", "gamma"),
+                 "uq.weight": ParamSpec((wide, self.q_rank))}
+        else:
+            p = {"q.weight": ParamSpec((wide, s.hidden))}
+        p.update({
              "dkv.weight": ParamSpec((self.kv_rank + self.rot, s.hidden)),
              "dkv.norm.weight": ParamSpec((self.kv_rank,), "vector", "gamma"),
              "uk.weight": ParamSpec((H * s.head_dim, self.kv_rank)), "uv.weight": ParamSpec((H * self.vdim, self.kv_rank)),
-             "o.weight": ParamSpec((s.hidden, H * self.vdim))}
+             "o.weight": ParamSpec((s.hidden, H * self.vdim))})
         if self.sink:
             p["sink"] = ParamSpec((H,), "vector", "wide")
         if self.gate:
@@ -396,27 +408,39 @@ class LatentAttention(Mixer):
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         s, H = self.spec, self.spec.num_heads
-        ws = [t["dq.weight"], t["dkv.weight"]] + ([t["g.weight"]] if self.gate else [])
+        # rows of the first product: [query latent] | c | rotated key part | [gates] or [queries | gates]; queries start at,
+        # and the rows end on, whole 16-byte units
+        ws = ([t["dq.weight"]] if self.q_rank else []) + [t["dkv.weight"]]
+
+        def pad():
+            n = sum(w.shape[0] for w in ws) % 8
+            if n:
+                ws.append(torch.zeros((8 - n, ws[0].shape[1]), dtype=ws[0].dtype, device=ws[0].device))
+        if not self.q_rank:
+            pad()
+            self.q_off = sum(w.shape[0] for w in ws)
+            ws.append(t["q.weight"])
+        self.gate_off = sum(w.shape[0] for w in ws)
+        if self.gate:
+            ws.append(t["g.weight"])
+        pad()
         if len({w.dtype for w in ws}) > 1:
             ws = [w.float() for w in ws]
-        n = sum(w.shape[0] for w in ws)
-        pad = (8 - n % 8) % 8                           # output rows of whole 16-byte units
-        if pad:
-            ws.append(torch.zeros((pad, ws[0].shape[1]), dtype=ws[0].dtype, device=ws[0].device))
         self.w_down = torch.cat(ws, dim=0).contiguous()
-        self.w_uq = t["uq.weight"]
+        self.w_uq = t["uq.weight"] if self.q_rank else None
         # W_uk,h^T as a product's weight [out = kv_rank, in = head_dim], head by head
         self.w_uk_t = t["uk.weight"].view(H, s.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = t["uv.weight"].view(H, self.vdim, self.kv_rank).contiguous()
         self.w_out = t["o.weight"]
-        self.q_gamma, self.kv_gamma = t["dq.norm.weight"], t["dkv.norm.weight"]
+        self.q_gamma, self.kv_gamma = t.get("dq.norm.weight"), t["dkv.norm.weight"]
         self.sinks = t.get("sink")
 
     def cache_request(self):
         return KVRequest(1, self.kv_rank + self.rot, self.spec.window, value_dim=self.kv_rank, values_in_keys=True)
 
     def products(self):
-        return [("down", self.w_down, None, None), ("uq", self.w_uq, None, None), ("o", self.w_out, None, None)]
+        up = [("uq", self.w_uq, None, None)] if self.q_rank else []
+        return [("down", self.w_down, None, None), *up, ("o", self.w_out, None, None)]
 
     def first_product(self):
         return self.w_down, None, None
@@ -429,13 +453,13 @@ class LatentAttention(Mixer):
         pages = ctx.pages[cache.group]
         cq = ops.latent_prepare(proj, cache.k, cache.v, ctx, pages, self.q_rank, self.kv_rank, self.rot, self.q_gamma,
                                 self.kv_gamma, self.eps, cos, sin, s.position.interleaved, write_kv=cache.writes)
-        q = ops.linear(cq, self.w_uq, None, out_dtype=ctx.act_dtype)
+        q = ops.linear(cq, self.w_uq, None, out_dtype=ctx.act_dtype) if self.q_rank else proj
         wide = ops.head_linear(q, self.w_uk_t, s.head_dim + self.rot, tail=self.rot, cos=cos, sin=sin,
-                               interleaved=s.position.interleaved)
+                               interleaved=s.position.interleaved, x_off=self.q_off)
         mixed = ops.attention_mixed(wide, cache.k, cache.v, ctx, pages, H, 1, self.kv_rank + self.rot, self.kv_rank,
                                     window=s.window, score_scale=self.score_scale, sinks=self.sinks, values_in_keys=True)
         o = ops.head_linear(mixed, self.w_uv, self.kv_rank, gate=proj if self.gate else None,
-                            gate_off=self.q_rank + self.kv_rank + self.rot)
+                            gate_off=self.gate_off)
         return o, self.w_out, None
 
     def forward(self, xn, ctx, cache, add: Sequence[torch.Tensor], out=None) -> torch.Tensor:

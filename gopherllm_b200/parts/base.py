@@ -37,13 +37,15 @@ class ParamSpec:
 @dataclass(frozen=True)
 class KVRequest:
     """A mixer's need for cached keys and values: per position ``num_kv_heads``
-    rows of ``head_dim``; ``window`` 0 keeps every position, w > 0 the last w."""
+    rows of ``head_dim``; ``window`` 0 keeps every position, w > 0 the last w; ``chunk`` n > 0 (window 0 then) the
+    positions of the chunk of n the next token lies in, chunks counted from position 0."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     value_dim: int = 0        # size of a head's values where it differs from head_dim (0: the same)
     value_heads: int = 0      # rows of values per position where they differ from the rows of keys (0: the same)
     values_in_keys: bool = False   # a position's values are the first value_dim numbers of its key rows: nothing more is kept
+    chunk: int = 0
 
 
 @dataclass(frozen=True)
@@ -157,7 +159,17 @@ class FeedForward(Part):
 class Block(Part):
     """One layer: owns a norm (or two), a mixer and a feed-forward and runs them
     in its arrangement.  forward(x, ctx, cache) updates the float32 residual
-    stream x [T, hidden] in place."""
+    stream x [T, hidden] in place.
+
+    streams: how many residual streams the arrangement works on (0: one, x as above).  With n > 0 streams x is
+    [T, n, hidden], and a layer's input is prepared by what runs before it: ``opening()`` gives the tensors for that,
+    (weights of the streams [n], norm weight [hidden], eps); a block finds its own input in
+    ctx.scratch["streams_input"] and leaves the next run's there, with the opening of ctx.next_block (None behind
+    the last run)."""
+    streams = 0
+
+    def opening(self):
+        raise NotImplementedError
 
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         raise NotImplementedError

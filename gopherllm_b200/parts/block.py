@@ -7,7 +7,7 @@ import torch
 
 from .. import ops
 from ..config.specs import BlockSpec
-from .base import Block, ParamSpec, build_feed_forward, build_mixer, build_norm, register_block
+from .base import Block, ParamSpec, Part, build_feed_forward, build_mixer, build_norm, register_block
 
 
 class AssembledBlock(Block):
@@ -258,7 +258,74 @@ class PostNormBlock(AssembledBlock):
         return x
 
 
+class StreamsBlock(AssembledBlock):
+    """Hyper-connections: the residual is n streams x_1 .. x_n (option ``streams``) in one tensor [T, n, hidden].  A
+    sublayer reads a weighted sum of them and what it returns joins all of them at once,
+        u = sum_s in[s] x_s;  y = sublayer(norm(u));  x_t <- sum_s mix[s, t] x_s + out[t] y   (mix is [from, to]),
+    with weights of its own for the mixer ("hc1") and the feed-forward ("hc2"); a layer without a feed-forward
+    (``spec.ffn`` None, no norm2) is the first half alone.  One kernel joins a sublayer's result, reads the streams for
+    the next sublayer and norms what it read, across layers too: a run finds its input in the step's context and leaves
+    the next run's there (see Block).  A mixer that offers ``branches`` is summed inside that kernel."""
+
+    def __init__(self, spec: BlockSpec):
+        if (spec.ffn is None) != (spec.norm2 is None):
+            raise ValueError("the second norm comes with the feed-forward: both or neither")
+        super().__init__(spec)
+        for n in (self.norm, self.norm2):
+            if n is not None and not (getattr(n, "rms", False) and n.fusable is not None and not n.spec.bias):
+                raise ValueError("a block of several streams takes RMS norms without bias")
+        self.streams = int(spec.option("streams", 1))
+        if not 1 <= self.streams <= ops.MAX_STREAMS:
+            raise ValueError(f"a block works on 1 to {ops.MAX_STREAMS} streams, not {self.streams}")
+        self.hc1 = StreamWeights(self.streams)
+        self.hc2 = StreamWeights(self.streams) if self.ffn is not None else None
+
+    def children(self) -> Dict[str, object]:
+        c = super().children()
+        c["hc1"] = self.hc1
+        if self.hc2 is not None:
+            c["hc2"] = self.hc2
+        return c
+
+    def opening(self):
+        gamma, _, eps, _ = self.norm.fusable()
+        return self.hc1.weight_in, gamma, eps
+
+    def forward(self, x, ctx, cache):
+        h = ctx.scratch["streams_input"]                # every run's input passes through this one buffer
+        branches = getattr(self.mixer, "branches", None)
+        y = branches(h, ctx, cache) if branches is not None else [(self.mixer.forward(h, ctx, cache, (), None), 1.0)]
+        after = ctx.next_block.opening() if ctx.next_block is not None else (None, None, 0.0)
+        if self.ffn is None:
+            ops.streams_join(x, y, self.hc1.mix, self.hc1.weight_out, *after, h=h)
+            return x
+        gamma, _, eps, _ = self.norm2.fusable()
+        ops.streams_join(x, y, self.hc1.mix, self.hc1.weight_out, self.hc2.weight_in, gamma, eps, h=h)
+        y = self.ffn.forward(h, ctx, (), None)
+        ops.streams_join(x, [(y, 1.0)], self.hc2.mix, self.hc2.weight_out, *after, h=h)
+        return x
+
+
+class StreamWeights(Part):
+    """How a sublayer reads n streams ("in" [n]) and how its result joins them ("mix" [n, n], from and to; "out" [n])."""
+    capturable = True
+    launches_only = True
+
+    def __init__(self, streams: int):
+        self.n = streams
+        self.weight_in = self.weight_out = self.mix = None
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        n = self.n
+        return {"in": ParamSpec((n,), "vector", "share"), "out": ParamSpec((n,), "vector", "gamma"),
+                "mix": ParamSpec((n, n), "vector", "near_identity")}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight_in, self.weight_out, self.mix = tensors["in"], tensors["out"], tensors["mix"]
+
+
 register_block("parallel", ParallelBlock)
 register_block("parallel_two_norms", TwoNormParallelBlock)
 register_block("sequential", SequentialBlock)
 register_block("post_norm", PostNormBlock)
+register_block("streams", StreamsBlock)

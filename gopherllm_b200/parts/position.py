@@ -38,12 +38,23 @@ def stretched_frequencies(rotary_dim: int, theta: float, factor: float, original
     return inv / factor * ramp + inv * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
+def banded_frequencies(rotary_dim: int, theta: float, factor: float, low: float, high: float, original: float) -> np.ndarray:
+    """64-bit frequencies [rotary_dim / 2] of a rotation stretched to longer contexts band by band, as Llama 3.1 does: with
+    n = how often a pair turns over ``original`` positions, pairs with n > high keep theta^(-2i/d), pairs with n < low
+    turn ``factor`` times slower, those between are blended linearly in n."""
+    inv = np.float64(theta) ** (-2.0 * np.arange(rotary_dim // 2, dtype=np.float64) / rotary_dim)
+    turns = original * inv / (2.0 * math.pi)
+    share = np.clip((turns - low) / (high - low), 0.0, 1.0) if high > low else (turns >= low).astype(np.float64)
+    return (1.0 - share) * inv / factor + share * inv
+
+
 class Rope(PositionEncoding):
     """Rotary embedding over the first ``rotary_dim`` dims of a head.  The
     angle float32(pos) * inv[i] is a 32-bit product; sine and cosine are taken
     in 64-bit (prepareRopeScratch, model.go:3041-3046).  The tables depend on
     the step's positions only, so every layer of a step shares them.  Option ``exact_angles``: frequencies and angles
-    in 64-bit; with it option ``yarn`` = (factor, original, fast, slow): see stretched_frequencies."""
+    in 64-bit; with it option ``yarn`` = (factor, original, fast, slow): see stretched_frequencies, or option ``bands`` =
+    (factor, low, high, original): see banded_frequencies."""
     capturable = True
     launches_only = True
 
@@ -53,18 +64,23 @@ class Rope(PositionEncoding):
         self.spec = spec
         self._inv = None
         self._gain = 1.0
-        if spec.option("yarn") is not None and not spec.option("exact_angles", False):
+        stretched = [k for k in ("yarn", "bands") if spec.option(k) is not None]
+        if stretched and not spec.option("exact_angles", False):
             raise ValueError("stretched frequencies come with exact angles")
+        if len(stretched) > 1:
+            raise ValueError("frequencies are stretched one way or the other, not both")
 
     def tables(self, ctx):
         exact = bool(self.spec.option("exact_angles", False))
-        yarn = self.spec.option("yarn")
-        key = ("rope", self.spec.rotary_dim, float(self.spec.theta), exact, yarn)
+        yarn, bands = self.spec.option("yarn"), self.spec.option("bands")
+        key = ("rope", self.spec.rotary_dim, float(self.spec.theta), exact, yarn, bands)
         hit = ctx.scratch.get(key)
         if hit is None:
             if self._inv is None or self._inv.device != ctx.device:
                 if yarn is not None:
                     inv, self._gain = stretched_frequencies(self.spec.rotary_dim, float(self.spec.theta), *yarn)
+                elif bands is not None:
+                    inv = banded_frequencies(self.spec.rotary_dim, float(self.spec.theta), *bands)
                 elif exact:
                     # frequencies theta^(-2i/d) and the angles pos * frequency in 64-bit: a table entry is then
                     # the rounded cosine of the true angle at any position (a 32-bit angle is off by up to

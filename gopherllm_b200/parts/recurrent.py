@@ -53,6 +53,11 @@ def _finish(o, w, add: Sequence, out: Optional[torch.Tensor]) -> torch.Tensor:
     return ops.linear(o, w, None, add0=a0, add1=a1, out_dtype=torch.float32, out=out)
 
 
+def _finish_product(until_last) -> torch.Tensor:
+    o, w, b = until_last
+    return ops.linear(o, w, b, out_dtype=torch.float32)
+
+
 class MatrixLstm(Mixer):
     """The matrix memory of xLSTM (mLSTM).  Per head: q = W_q h / sqrt(dim), k, v; log input gate
     gi = cap tanh((W_i h + b_i) / cap), log forget gate gf = logsigmoid(cap tanh((W_f h + b_f) / cap));
@@ -482,6 +487,76 @@ class StateSpaceDual(Mixer):
         return _finish(y, w, add, out)
 
 
+class GatedLinearUnit(Mixer):
+    """Griffin's recurrent block with a real-gated linear recurrent unit.  Two branches of ``width`` channels,
+        y = gelu(W_y h + b_y) (tanh form),  u = conv(W_x h + b_x),
+    the convolution causal and per channel (``conv`` taps, the last the current token's, zeros before the start, bias, no
+    activation).  u falls into ``blocks`` equal parts with a square matrix per part and gate:
+        r = sigmoid(R u + b_r),  i = sigmoid(I u + b_i),  log a = -``decay`` r softplus(lam),  a = e^(log a),
+        S <- a S + sqrt(1 - a^2) i u  from S = 0;  output W_o (S y).
+    The state row holds S [width] and the convolution's last taps - 1 inputs; gates, decays and the state are 32-bit.
+    Options: ``width``, ``blocks``, ``conv``, ``decay``."""
+    capturable = True
+    launches_only = True
+    deferred_add = True
+
+    def __init__(self, spec: MixerSpec):
+        self.spec = spec
+        self.C, self.blocks = int(spec.option("width")), int(spec.option("blocks", 1))
+        self.taps, self.decay = int(spec.option("conv", 1)), float(spec.option("decay", 8.0))
+        if self.C < 1 or self.blocks < 1 or self.C % self.blocks:
+            raise ValueError(f"gated_linear_unit: {self.C} channels do not form {self.blocks} equal parts")
+        if self.taps < 1:
+            raise ValueError("gated_linear_unit: the convolution has at least one tap")
+        if not self.decay > 0:
+            raise ValueError("gated_linear_unit: the decay's factor is positive")
+        self.y_off = _pad8(self.C)                     # columns of the first product: x, then y, each in whole 16-byte units
+        self.state_size = self.C + self.C * (self.taps - 1)
+        self.w_in = self.b_in = self.conv_w = self.conv_b = self.w_gates = self.b_gates = self.rate = self.w_o = None
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        C, W, B, n = self.C, self.spec.hidden, self.blocks, self.C // self.blocks
+        return {"y.weight": ParamSpec((C, W)), "y.bias": ParamSpec((C,), "vector", "bias"),
+                "x.weight": ParamSpec((C, W)), "x.bias": ParamSpec((C,), "vector", "bias"),
+                "conv.weight": ParamSpec((C, self.taps), "vector", "wide"), "conv.bias": ParamSpec((C,), "vector", "bias"),
+                "ra.weight": ParamSpec((B, n, n)), "ra.bias": ParamSpec((B, n), "vector", "wide"),
+                "ri.weight": ParamSpec((B, n, n)), "ri.bias": ParamSpec((B, n), "vector", "wide"),
+                "lam": ParamSpec((C,), "vector", "wide"), "o.weight": ParamSpec((W, C))}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        C, B, n = self.C, self.blocks, self.C // self.blocks
+        x = t["x.weight"]
+        gap = torch.zeros((self.y_off - C, x.shape[1]), dtype=x.dtype, device=x.device)
+        self.w_in, self.b_in = _joined([x, gap, t["y.weight"]], [t["x.bias"], None, t["y.bias"]], x)
+        self.conv_w, self.conv_b, self.w_o = t["conv.weight"], t["conv.bias"], t["o.weight"]
+        # the two gates' rows alternate, channel by channel
+        gates = [t["ra.weight"], t["ri.weight"]]
+        if gates[0].dtype != gates[1].dtype:
+            gates = [g.float() for g in gates]
+        self.w_gates = torch.stack(gates, 2).reshape(B, 2 * n, n).contiguous()
+        self.b_gates = torch.stack([t["ra.bias"].reshape(C), t["ri.bias"].reshape(C)], 1).reshape(2 * C).contiguous()
+        self.rate = (-self.decay * torch.nn.functional.softplus(t["lam"].double(), threshold=1e9)).float().contiguous()
+
+    def cache_request(self):
+        return StateRequest((self.state_size,))
+
+    def first_product(self):
+        return self.w_in, self.b_in, None
+
+    def products(self):
+        return [("in", self.w_in, self.b_in, None), ("o", self.w_o, None, None)]
+
+    def until_last(self, xn, ctx, cache, first=None):
+        proj = first if first is not None else ops.linear(xn, self.w_in, self.b_in, out_dtype=ctx.act_dtype)
+        u = ops.conv_silu(proj, self.conv_w, self.conv_b, cache.rows, self.C, ctx, x_off=0, silu=False)
+        y = ops.gated_unit(u, self.w_gates, self.b_gates, self.rate, proj, self.y_off, cache.rows, ctx)
+        return y, self.w_o, None
+
+    def forward(self, xn, ctx, cache, add: Sequence, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        y, w, _ = self.until_last(xn, ctx, cache)
+        return _finish(y, w, add, out)
+
+
 class ScaledPair(Mixer):
     """Two mixers side by side on the same input, summed with a factor each: left_scale * left(h) +
     right_scale * right(h).  The children are whole mixer specs (options ``left`` and ``right``); their cache
@@ -520,7 +595,28 @@ class ScaledPair(Mixer):
                 + [("right." + n, w, b, a) for n, w, b, a in self.right.products()])
 
     def branches(self, xn, ctx, cache):
-        """[(float32 output, factor)] of the two children."""
+        """[(float32 output, factor)] of the two children.  Children that offer their first products run them as one grid
+        for many tokens; in one-token steps, where every kernel is short, the right child runs on the step's second
+        stream beside the left one."""
+        side = getattr(ctx, "side_stream", None)
+        if side is not None and torch.cuda.current_stream() != side:
+            main = torch.cuda.current_stream()
+            yr = ops.empty((xn.shape[0], self.spec.hidden), torch.float32, xn.device)
+            fork, join = torch.cuda.Event(), torch.cuda.Event()
+            fork.record(main)
+            side.wait_event(fork)
+            with torch.cuda.stream(side):
+                self.right.forward(xn, ctx, cache[1], (), yr)
+                join.record(side)
+            yl = self.left.forward(xn, ctx, cache[0], (), None)
+            main.wait_event(join)
+            return [(yl, self.left_scale), (yr, self.right_scale)]
+        if all(c.until_last is not None and c.first_product is not None for c in (self.left, self.right)):
+            wl, bl, al = self.left.first_product()
+            wr, br, ar = self.right.first_product()
+            pl, pr = ops.linear_fork(xn, wl, bl, al, wr, br, ar, ctx.act_dtype)
+            return [(_finish_product(self.left.until_last(xn, ctx, cache[0], first=pl)), self.left_scale),
+                    (_finish_product(self.right.until_last(xn, ctx, cache[1], first=pr)), self.right_scale)]
         return [(self.left.forward(xn, ctx, cache[0], (), None), self.left_scale),
                 (self.right.forward(xn, ctx, cache[1], (), None), self.right_scale)]
 
@@ -537,4 +633,5 @@ register_mixer("normed_pair", NormedPair)
 register_mixer("gated_delta", GatedDeltaRule)
 register_mixer("retention", Retention)
 register_mixer("mamba2", StateSpaceDual)
+register_mixer("gated_linear_unit", GatedLinearUnit)
 register_mixer("scaled_pair", ScaledPair)

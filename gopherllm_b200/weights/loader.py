@@ -208,6 +208,10 @@ def random_tensor(name: str, spec: ParamSpec, seed: int, sigma: float, storage: 
         t = z.zero_()
     elif spec.init == "unit":                  # a bound or a share, strictly inside (0, 1)
         t = torch.sigmoid(z)
+    elif spec.init == "share":                 # weights of a sum of several equal things
+        t = z.mul_(0.1).add_(1.0).div_(max(1, spec.shape[-1]))
+    elif spec.init == "near_identity":
+        t = z.mul_(0.02).add_(torch.eye(*spec.shape))
     elif spec.init == "wide":                  # N(0, 1): biases of gates that should not all sit at one half
         t = z
     else:
