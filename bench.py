@@ -8,6 +8,7 @@
     python bench.py --design lilupel         the same for a Lilupel model, beside a Vopedra model of equal width and depth
     python bench.py --design darusun         the same for a Darusun model, beside a Gozolix model of equal width and depth
     python bench.py --design dibedra         the same for a Dibedra model, beside a Gozolix and a Phi model of equal width and depth
+    python bench.py --design nakurax         the same for a Nakurax model, beside a Darusun and a Vopedra model of equal width and depth
     python bench.py --design vopedra         prefill and decode of a Vopedra model at a few layer sizes beside a
                                              Phi model of equal width, depth and feed-forward weights
 
@@ -121,7 +122,7 @@ def main():
     ap.add_argument("--sections", default="decode,e2e,prefill,points",
                     help="which measurements to run (for profiling a part): decode,e2e,prefill,points")
     ap.add_argument("--model", default="phi-2", choices=sorted(MODELS), help="whose layer sizes to run")
-    ap.add_argument("--design", default=None, choices=["vopedra", "gozolix", "lilupel", "darusun", "dibedra"],
+    ap.add_argument("--design", default=None, choices=["vopedra", "gozolix", "lilupel", "darusun", "dibedra", "nakurax"],
                     help="instead: prefill and decode rates of another design at a few layer sizes, beside the Phi "
                          "model of equal width and depth")
     ap.add_argument("--ragged", action="store_true",
@@ -151,7 +152,7 @@ def main():
 
     if args.design == "vopedra":
         return design_vopedra(args)
-    if args.design in ("gozolix", "lilupel", "darusun", "dibedra"):
+    if args.design in ("gozolix", "lilupel", "darusun", "dibedra", "nakurax"):
         return design_vopedra(args, design=args.design)
     pk, pk_src = peaks()
     label, sizes, weight_seed = MODELS[args.model]
@@ -427,13 +428,31 @@ def dibedra_sizes(width, heads, ff):
             "initializer_range": 0.02, "layers": five + second}
 
 
+def nakurax_sizes(width, heads, ff):
+    """A Nakurax model whose layers resemble a real model's at this width, four residual streams, five layers run twice: a
+    latent attention (256 numbers a position, all positions), a chunked attention (512 positions, a quarter as many
+    key/value heads as query heads) beside a gated linear recurrence as wide as the model and a quarter, in blocks of
+    width / 8, two latent attentions, the pair again; dense feed-forwards of as many weights as the other designs'."""
+    hd = width // heads
+    latent = {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": 256, "scale": hd ** -0.5}
+    pair = {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": 512},
+                     "rot": {"dims": hd, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+            "right": {"width": 5 * width // 4, "blocks": 10, "conv": 4}, "left_scale": 1.0, "right_scale": 1.0}
+    dense = {"kind": "dense", "ff": (3 * ff // 2) // 64 * 64}
+    five = [{"type": t, "mixer": latent if t == "latent_attention" else pair, "mlp": dense}
+            for t in ("latent_attention", "parallel", "latent_attention", "latent_attention", "parallel")]
+    return {"architecture": "Nakurax", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "streams": 4,
+            "embedding": {"scale": 1.0}, "initializer_range": 0.02, "layers": five, "loop": {"start": 0, "stop": 5, "times": 2}}
+
+
 def design_vopedra(args, design="vopedra"):
     """Prefill and decode rates of Vopedra models (random weights) beside Phi models of the same width, the
     same number of layer runs and feed-forwards of the same number of weights; with ``design`` "gozolix" or
     "lilupel", of models of that design beside Vopedra models of the same width and number of layer runs; with
     "darusun", beside Gozolix models (the nearest relative: softmax attention, layers on another layer's keys, dense
     feed-forwards and routed mixtures with a shared expert); with "dibedra", beside Gozolix models (grouped attention,
-    dense feed-forwards, grouped routing) and Phi models (the same block).  One JSON line."""
+    dense feed-forwards, grouped routing) and Phi models (the same block); with "nakurax", beside Darusun models
+    (attention through a latent) and Vopedra models (recurrences, pairs of mixers, loops).  One JSON line."""
     import numpy as np
     import torch
     import gopherllm_b200 as gl
@@ -501,6 +520,11 @@ def design_vopedra(args, design="vopedra"):
             rows.append({"width": width, "heads": heads, design: d, "gozolix": measure(gozolix_sizes(width, heads, ff_gated)),
                          "phi": measure(phi)})
             continue
+        if design == "nakurax":
+            rows.append({"width": width, "heads": heads, design: measure(nakurax_sizes(width, heads, ff_gated)),
+                         "darusun": measure(darusun_sizes(width, heads, ff_gated)),
+                         "vopedra": measure(vopedra_sizes(width, heads, ff_gated))})
+            continue
         if design == "darusun":
             rows.append({"width": width, "heads": heads, design: measure(darusun_sizes(width, heads, ff_gated)),
                          "gozolix": measure(gozolix_sizes(width, heads, ff_gated))})
@@ -514,8 +538,8 @@ def design_vopedra(args, design="vopedra"):
         phi = dict(PHI15, hidden_size=width, num_attention_heads=heads, num_key_value_heads=heads,
                    intermediate_size=ff_plain, vocab_size=32000, num_hidden_layers=v["layer_runs"])
         rows.append({"width": width, "heads": heads, "vopedra": v, "phi": measure(phi)})
-    if design in ("gozolix", "lilupel", "darusun", "dibedra"):
-        beside = {"darusun": "Gozolix", "dibedra": "Gozolix and Phi"}.get(design, "Vopedra")
+    if design in ("gozolix", "lilupel", "darusun", "dibedra", "nakurax"):
+        beside = {"darusun": "Gozolix", "dibedra": "Gozolix and Phi", "nakurax": "Darusun and Vopedra"}.get(design, "Vopedra")
         print(json.dumps({"metric": f"prefill and decode rates of {design.capitalize()} layer sizes beside {beside} of equal width and depth (bf16)",
                           "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic: random weights seed 7, uniform token ids",
                           "decode_steps_timed": K, "decode_context": 1024, "peaks": pk_src, "clocks": clocks.stop(), "sizes": rows}))
