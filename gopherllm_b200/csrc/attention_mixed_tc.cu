@@ -53,6 +53,9 @@ struct PairsArgs {
     int v_in_k;               // such a cache with one row of values a key head: no value tile is fetched, the second
                               // product reads the key tile
     int chunk;                // > 0: a query sees the keys of its own chunk of positions alone (window is then 0)
+    const int* seq_base;      // [B] or null: keys and values are not in pages but rows of matrices kv_ld numbers apart, sequence
+                              // b's position 0 in row seq_base[b], a head's numbers side by side from column head * size on
+    int kv_ld, q_ld;          // q_ld > 0: numbers between two rows of q
 };
 
 __device__ __forceinline__ unsigned ap_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -133,13 +136,22 @@ attn_pairs_tc_kernel(PairsArgs a) {
     const size_t vs = a.vs > 0 ? (size_t)a.vs : (size_t)AP_VD;
     const size_t vhead_off = (size_t)vh * GL_PAGE * vs, vpage_stride = (size_t)nvh * GL_PAGE * vs;
     const int total = ctx + qlen;
+    const size_t k_row = a.seq_base ? (size_t)a.kv_ld : AP_HD, v_row = a.seq_base ? (size_t)a.kv_ld : vs;
+    const size_t first_row = a.seq_base ? (size_t)a.seq_base[b] : 0;
+    auto k_page = [&](int p) {
+        return a.seq_base ? K + (first_row + (size_t)p * GL_PAGE) * k_row + (size_t)g * AP_HD : K + (size_t)pg[p] * page_stride + head_off;
+    };
+    auto v_page = [&](int p) {
+        return a.seq_base ? V + (first_row + (size_t)p * GL_PAGE) * v_row + (size_t)vh * AP_VD : V + (size_t)pg[p] * vpage_stride + vhead_off;
+    };
+    const size_t q_row = a.q_ld > 0 ? (size_t)a.q_ld : (size_t)a.nH * AP_HD;
 
     // the query tile and the first page; the tile's fragments go to registers before its stage is used for keys
-    ap_load_rows<AP_HD>(sQ, (const __nv_bfloat16*)a.q + ((size_t)(qstart + q0) * a.nH + h) * AP_HD, (size_t)a.nH * AP_HD, rows);
+    ap_load_rows<AP_HD>(sQ, (const __nv_bfloat16*)a.q + (size_t)(qstart + q0) * q_row + (size_t)h * AP_HD, q_row, rows);
     {
         const int nv = min(GL_PAGE, total - page_begin * GL_PAGE);
-        ap_load_rows<AP_HD>(sK[0], K + (size_t)pg[page_begin] * page_stride + head_off, AP_HD, nv);
-        if (!a.v_in_k) ap_load_rows<AP_VD>(sV[0], V + (size_t)pg[page_begin] * vpage_stride + vhead_off, vs, nv);
+        ap_load_rows<AP_HD>(sK[0], k_page(page_begin), k_row, nv);
+        if (!a.v_in_k) ap_load_rows<AP_VD>(sV[0], v_page(page_begin), v_row, nv);
     }
     ap_commit();
     ap_wait<0>();
@@ -172,8 +184,8 @@ attn_pairs_tc_kernel(PairsArgs a) {
         const int st = (p - page_begin) & 1;
         if (p + 1 < page_end) {
             const int nv = min(GL_PAGE, total - (p + 1) * GL_PAGE);
-            ap_load_rows<AP_HD>(sK[st ^ 1], K + (size_t)pg[p + 1] * page_stride + head_off, AP_HD, nv);
-            if (!a.v_in_k) ap_load_rows<AP_VD>(sV[st ^ 1], V + (size_t)pg[p + 1] * vpage_stride + vhead_off, vs, nv);
+            ap_load_rows<AP_HD>(sK[st ^ 1], k_page(p + 1), k_row, nv);
+            if (!a.v_in_k) ap_load_rows<AP_VD>(sV[st ^ 1], v_page(p + 1), v_row, nv);
         }
         ap_commit();
         ap_wait<1>();
@@ -560,6 +572,7 @@ GL_API int gl_attention_pairs_tc(const PairsArgs* args, cudaStream_t stream) {
     if (a.nVH < 0 || (a.nVH > 0 && (a.nH % a.nVH || (a.nVal != 1 && a.nVH != a.nKV)))) return GL_ERR_SHAPE;
     if (a.vs < 0 || (a.vs > 0 && (a.vs < AP_VD || a.vs % 8))) return GL_ERR_SHAPE;
     if (a.v_in_k && (AP_VD > AP_HD || a.nVal != 1 || (a.nVH > 0 && a.nVH != a.nKV))) return GL_ERR_SHAPE;
+    if (a.q_ld % 8 || (a.seq_base && (a.kv_ld <= 0 || a.kv_ld % 8 || a.v_in_k))) return GL_ERR_SHAPE;
     if (a.B > 65535 || a.nH * a.nVal > 65535) return GL_ERR_SHAPE;
     const size_t smem = 2 * (size_t)AP_TILE + (a.v_in_k ? 0 : 2 * (size_t)AP_VTILE);
     static size_t configured = 0;

@@ -94,6 +94,17 @@ struct AttnGate {
     int ld, off;
 };
 
+// Where queries, keys and values lie when that is not the caller's compact q and the cache's pages, and which keys a
+// query sees when that is not a window.  A record of its own with an entry point of its own, as above; all zero: as if
+// it were not there.
+struct AttnPlace {
+    const int* seq_base;      // [B] or null: keys and values are rows of matrices, sequence b's position 0 in row seq_base[b],
+                              // key head g's numbers at columns g*hd.. of its row (k_cache, v_cache: the matrices' first columns)
+    int kv_ld, kv_rows;       // numbers between two rows (a multiple of 8), rows
+    int q_ld;                 // > 0: numbers between two rows of q (a multiple of 8)
+    int chunk;                // > 0: a query sees the keys of its own chunk of positions alone (window is then 0)
+};
+
 struct AttnMaps { CUtensorMap q[4], k[4], v; };
 
 __device__ __forceinline__ float at_exp2(float x) {
@@ -104,7 +115,7 @@ __device__ __forceinline__ float at_exp2(float x) {
 
 template <int NT>
 __global__ void __launch_bounds__(AT_THREADS(NT), 3 - NT)
-attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMaps maps) {
+attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, AttnPlace place, const __grid_constant__ AttnMaps maps) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ unsigned tmem_slot;
     __shared__ volatile int failed;
@@ -138,7 +149,7 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
     const int g = h / (a.nH / a.nKV);
     const int total = ctx + qlen;
     const int p_first = ctx + q0;
-    const int lo_first = (a.window > 0 && p_first - a.window + 1 > 0) ? p_first - a.window + 1 : 0;
+    const int lo_first = gl_first_key(p_first, a.window, place.chunk);
     const int page_begin = lo_first / GL_PAGE;
     // pages each tile needs: from the block's first page to the page of the tile's last row
     const int n0 = (p_first + min(AT_BM, rows_all) - 1) / GL_PAGE + 1 - page_begin;
@@ -182,17 +193,18 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
             for (int j = 0; j < n_max && !failed; ++j) {
                 const int st = j % AT_STAGES;
                 const unsigned par = ((j / AT_STAGES) - 1) & 1;
-                const int row = (pg[page_begin + j] * a.nKV + g) * GL_PAGE;
+                const int row = place.seq_base ? place.seq_base[b] + (page_begin + j) * GL_PAGE : (pg[page_begin + j] * a.nKV + g) * GL_PAGE;
+                const int col = place.seq_base ? g * AT_HD : 0;
                 if (j >= AT_STAGES && !mbar_wait(bar_ke + 8 * st, par)) { failed = 1; break; }
                 mbar_expect_tx(bar_kf + 8 * st, GL_PAGE * AT_HD * 2);
 #pragma unroll
                 for (int s = 0; s < AT_NSEG; ++s)
-                    tma_load_2d(sK + st * AT_K_BYTES + at_seg_base(s, GL_PAGE), &maps.k[s], at_seg(s).off, row, bar_kf + 8 * st);
+                    tma_load_2d(sK + st * AT_K_BYTES + at_seg_base(s, GL_PAGE), &maps.k[s], col + at_seg(s).off, row, bar_kf + 8 * st);
                 if (j >= AT_STAGES && !mbar_wait(bar_ve + 8 * st, par)) { failed = 1; break; }
                 mbar_expect_tx(bar_vf + 8 * st, AT_V_BYTES);                       // zero fill counts
 #pragma unroll
                 for (int c = 0; c < AT_VATOMS; ++c)
-                    tma_load_2d(sV + st * AT_V_BYTES + c * AT_VATOM_BYTES, &maps.v, 64 * c, row, bar_vf + 8 * st);
+                    tma_load_2d(sV + st * AT_V_BYTES + c * AT_VATOM_BYTES, &maps.v, col + 64 * c, row, bar_vf + 8 * st);
             }
         }
     } else if (warp > PRODUCER) {
@@ -264,11 +276,11 @@ attn_prefill_tc_kernel(AttnArgs a, AttnGate gate, const __grid_constant__ AttnMa
         const int r = quarter * 32 + lane;                                  // row inside the tile
         const int rows = min(AT_BM, rows_all - t * AT_BM);                  // valid rows of this tile (may be <= 0)
         const int pos = p_first + t * AT_BM + r;
-        const int wlo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+        const int wlo = gl_first_key(pos, a.window, place.chunk);
         const unsigned lane_off = (unsigned)(quarter * 32) << 16;
         const unsigned tS = tmem + 256 * t + lane_off, tO = tS + 128;
         const int nt = t ? n1 : n0;
-        const float LOG2E = 1.4426950408889634f;
+        const float LOG2E = 1.4426950408889634f * a.score_scale;           // (scores stay as they are, their exponents are scaled)
         float m_run = -INFINITY, l_run = 0.f;
         bool alive = true;
         for (int j = 0; j < nt; ++j) {
@@ -431,25 +443,28 @@ static bool at_allow() {
     return cudaFuncSetAttribute(attn_prefill_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)at_smem(NT)) == cudaSuccess;
 }
 template <int NT>
-static int at_launch(long long blocks, cudaStream_t stream, const AttnArgs& a, const AttnGate& gate, const AttnMaps& maps) {
-    return gl_launch(attn_prefill_tc_kernel<NT>, dim3((unsigned)blocks), dim3(AT_THREADS(NT)), at_smem(NT), stream, 1, a, gate, maps);
+static int at_launch(long long blocks, cudaStream_t stream, const AttnArgs& a, const AttnGate& gate, const AttnPlace& place,
+                     const AttnMaps& maps) {
+    return gl_launch(attn_prefill_tc_kernel<NT>, dim3((unsigned)blocks), dim3(AT_THREADS(NT)), at_smem(NT), stream, 1, a, gate, place, maps);
 }
 
 // Tiles a block.  Blocks of one tile, two an SM, overlap one's start and end with the other's pages and share the work
 // out in smaller pieces, at the price of every tile fetching its own pages: measured ahead with a window (32 heads of 64,
 // 2,048 tokens, 512 positions: 36.9 against 44.1 us; 8 x 1,024 tokens, 256 positions: 82 against 100) and where blocks
 // of two tiles do not fill the SMs (512 tokens: 17 against 18), behind without (2,048 tokens: 56 against 48).
-static int at_choose(const AttnArgs& a, int sms) {
+static int at_choose(const AttnArgs& a, const AttnPlace& place, int sms) {
     if (!AT_ONE_TILE) return 2;
     if (at_tiles) return at_tiles;
     const long long pairs = (long long)((a.max_qlen + 2 * AT_BM - 1) / (2 * AT_BM)) * a.nH * a.B;
-    return a.window > 0 || pairs < sms ? 1 : 2;
+    return a.window > 0 || place.chunk > 0 || pairs < sms ? 1 : 2;
 }
 
-static int prefill_tc(const AttnArgs& a, const AttnGate& gate, int n_tokens, int n_pages, cudaStream_t stream) {
+static int prefill_tc(const AttnArgs& a, const AttnGate& gate, const AttnPlace& place, int n_tokens, int n_pages, cudaStream_t stream) {
     if (a.B <= 0 || a.max_qlen <= 0) return GL_OK;
     if (a.hd != AT_HD || a.nH <= 0 || a.nKV <= 0 || a.nH % a.nKV) return GL_ERR_SHAPE;
-    if (a.score_scale != 1.0f) return GL_ERR_SHAPE;
+    if (!(a.score_scale > 0.f) || place.chunk < 0 || (place.chunk > 0 && a.window > 0)) return GL_ERR_SHAPE;
+    if (place.q_ld < 0 || place.q_ld % 8 || (place.q_ld > 0 && place.q_ld < a.nH * AT_HD)) return GL_ERR_SHAPE;
+    if (place.seq_base && (place.kv_ld % 8 || place.kv_ld < a.nKV * AT_HD || place.kv_rows <= 0)) return GL_ERR_SHAPE;
     if (((uintptr_t)a.q | (uintptr_t)a.out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15) return GL_ERR_ALIGN;
     static int sms = 0;
     if (!sms) {
@@ -463,35 +478,45 @@ static int prefill_tc(const AttnArgs& a, const AttnGate& gate, int n_tokens, int
             return GL_ERR_SMEM;
         }
     }
-    const int nt = at_choose(a, sms);
+    const int nt = at_choose(a, place, sms);
     AttnMaps maps;
-    const uint64_t kv_rows = (uint64_t)n_pages * a.nKV * GL_PAGE;
+    const uint64_t kv_rows = place.seq_base ? (uint64_t)place.kv_rows : (uint64_t)n_pages * a.nKV * GL_PAGE;
+    const uint64_t kv_cols = place.seq_base ? (uint64_t)a.nKV * AT_HD : AT_HD, kv_pitch = place.seq_base ? (uint64_t)place.kv_ld : 0;
     for (int s = 0; s < AT_NSEG; ++s) {
         const int w = at_seg(s).width;
-        int rc = gl_cached_map(&maps.q[s], a.q, (uint64_t)n_tokens, (uint64_t)a.nH * AT_HD, AT_BM, w, 2);
+        int rc = gl_cached_map(&maps.q[s], a.q, (uint64_t)n_tokens, (uint64_t)a.nH * AT_HD, AT_BM, w, 2, (uint64_t)place.q_ld);
         if (rc != GL_OK) return rc;
-        rc = gl_cached_map(&maps.k[s], a.k_cache, kv_rows, AT_HD, GL_PAGE, w, 2);
+        rc = gl_cached_map(&maps.k[s], a.k_cache, kv_rows, kv_cols, GL_PAGE, w, 2, kv_pitch);
         if (rc != GL_OK) return rc;
     }
     {   // values: 64 dims a box; what a box has beyond the head size reads as zero
-        int rc = gl_cached_map(&maps.v, a.v_cache, kv_rows, AT_HD, GL_PAGE, 64, 2);
+        int rc = gl_cached_map(&maps.v, a.v_cache, kv_rows, kv_cols, GL_PAGE, 64, 2, kv_pitch);
         if (rc != GL_OK) return rc;
     }
     const long long blocks = (long long)((a.max_qlen + nt * AT_BM - 1) / (nt * AT_BM)) * a.nH * a.B;
     if (blocks > 0x7fffffffLL) return GL_ERR_SHAPE;
-    const int rc = nt == 1 ? at_launch<(AT_ONE_TILE ? 1 : 2)>(blocks, stream, a, gate, maps) : at_launch<2>(blocks, stream, a, gate, maps);
+    const int rc = nt == 1 ? at_launch<(AT_ONE_TILE ? 1 : 2)>(blocks, stream, a, gate, place, maps)
+                           : at_launch<2>(blocks, stream, a, gate, place, maps);
     return rc == 0 ? GL_OK : GL_ERR_LAUNCH;
 }
 
 // n_tokens: rows of q; n_pages: pages of the cache entry
 GL_API int gl_attention_prefill_tc(const AttnArgs* args, int n_tokens, int n_pages, cudaStream_t stream) {
     const AttnGate none = {nullptr, 0, 0};
-    return prefill_tc(*args, none, n_tokens, n_pages, stream);
+    const AttnPlace cache = {nullptr, 0, 0, 0, 0};
+    return prefill_tc(*args, none, cache, n_tokens, n_pages, stream);
 }
 
 // the same with a gate on the result
 GL_API int gl_attention_prefill_tc_gated(const AttnArgs* args, const AttnGate* gate, int n_tokens, int n_pages, cudaStream_t stream) {
     if (!gate->gate || gate->ld % 8 || gate->off < 0 || gate->off % 8 || gate->off + args->nH * AT_HD > gate->ld) return GL_ERR_SHAPE;
     if ((uintptr_t)gate->gate & 15) return GL_ERR_ALIGN;
-    return prefill_tc(*args, *gate, n_tokens, n_pages, stream);
+    const AttnPlace cache = {nullptr, 0, 0, 0, 0};
+    return prefill_tc(*args, *gate, cache, n_tokens, n_pages, stream);
+}
+
+// the same with queries, keys and values where ``place`` says, or chunks
+GL_API int gl_attention_prefill_tc_placed(const AttnArgs* args, const AttnPlace* place, int n_tokens, int n_pages, cudaStream_t stream) {
+    const AttnGate none = {nullptr, 0, 0};
+    return prefill_tc(*args, none, *place, n_tokens, n_pages, stream);
 }

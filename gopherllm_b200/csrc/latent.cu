@@ -11,11 +11,12 @@
 //                       RMS-normed with a weight, the key part rotated; the query latent written out, the row
 //                       [c | key part] written to the token's place in the cache (the values are its first columns;
 //                       a cache that keeps values of its own gets c once more).
+//   gl_latent_rows      the latents of whole sequences as rows of one matrix, out of the pages.
 //   gl_head_linear      out[t, h, :] = W_h x[t, h, :] per head (strided rows on both sides), optionally followed by
 //                       a rotated copy of the columns behind x[t, h, :K] (the query's rotated part) and optionally
 //                       times sigmoid(gate[t, h]) (an output gate per head).
 // Norms, rotation, gates and all sums are 32-bit; one block a token in the first kernel, tiles of 64 x 64 in the
-// second: on the CUDA cores with sums over k in ascending order (the 32-bit path, and sizes the other form does not
+// last: on the CUDA cores with sums over k in ascending order (the 32-bit path, and sizes the other form does not
 // take), on the tensor cores for bfloat16 in whole 16-byte pieces.
 #include "common.cuh"
 
@@ -33,6 +34,7 @@ struct LatentPrepareArgs {
     const int* pages;         // [B, max_pages]
     int T, ld, q_rank, kv_rank, rot, max_pages, n_pages, interleaved, write_kv;
     float eps;
+    void* c_out;              // [T, kv_rank] cache type or null: c once more, a row a token
 };
 
 template <typename TA, typename TC>
@@ -76,6 +78,7 @@ latent_prepare_kernel(LatentPrepareArgs a) {
         const float y = c[i] * inv_k * a.kv_gamma[i];
         gl_store(kr + i, y);
         if (a.v_cache) gl_store(vr + i, y);
+        if (a.c_out) gl_store((TC*)a.c_out + (size_t)t * a.kv_rank + i, y);
     }
     const float* kp = c + a.kv_rank;
     const int half = a.rot / 2;
@@ -106,6 +109,39 @@ GL_API int gl_latent_prepare(const LatentPrepareArgs* args, int act_dtype, int c
     else if (act_dtype == GL_BF16) rc = gl_launch(latent_prepare_kernel<__nv_bfloat16, __nv_bfloat16>, g, b, smem, stream, 1, a);
     else return GL_ERR_DTYPE;
     return rc == 0 ? GL_OK : GL_ERR_LAUNCH;
+}
+
+// ---------------------------------------------------------------------------
+// out[base[b] + p, :] = the first n numbers of sequence b's cached row of position p, for all its positions (those of this
+// step too).  A warp a row.
+// ---------------------------------------------------------------------------
+template <typename TC>
+__global__ void __launch_bounds__(256)
+latent_rows_kernel(const TC* cache, const int* __restrict__ seq_base, const int* seq_qlen, const int* seq_ctx, const int* pages,
+                   TC* out, int wide, int n, int max_pages, int n_pages) {
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    const int b = blockIdx.y, p = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (p >= seq_ctx[b] + seq_qlen[b]) return;
+    const int slot = gl_checked(p / GL_PAGE, max_pages, GL_BAD_POSITION);
+    const int page = gl_checked(pages[(size_t)b * max_pages + slot], n_pages > 0 ? n_pages : 0x7fffffff, GL_BAD_PAGE);
+    const TC* src = cache + ((size_t)page * GL_PAGE + p % GL_PAGE) * wide;
+    TC* dst = out + ((size_t)seq_base[b] + p) * n;
+    for (int i = lane; i < n; i += 32) dst[i] = src[i];
+}
+
+GL_API int gl_latent_rows(const void* cache, const int* seq_base, const int* seq_qlen, const int* seq_ctx, const int* pages, void* out,
+                          int B, int wide, int n, int max_pages, int n_pages, int max_len, int dtype, cudaStream_t stream) {
+    if (B <= 0 || max_len <= 0) return GL_OK;
+    if (n <= 0 || wide < n || B > 65535) return GL_ERR_SHAPE;
+    const dim3 grid((unsigned)((max_len + 7) / 8), (unsigned)B);
+    if (dtype == GL_F32)
+        return gl_launch(latent_rows_kernel<float>, grid, dim3(256), 0, stream, 1, (const float*)cache, seq_base, seq_qlen, seq_ctx, pages,
+                         (float*)out, wide, n, max_pages, n_pages);
+    if (dtype == GL_BF16)
+        return gl_launch(latent_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, 1, (const __nv_bfloat16*)cache, seq_base, seq_qlen,
+                         seq_ctx, pages, (__nv_bfloat16*)out, wide, n, max_pages, n_pages);
+    return GL_ERR_DTYPE;
 }
 
 // ---------------------------------------------------------------------------

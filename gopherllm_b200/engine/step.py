@@ -26,9 +26,11 @@ class StepContext:
     tokens[T], tok_seq[T] (index of the token's sequence in this batch),
     tok_pos[T] (absolute position); seq_slot[B], seq_qstart[B] (row of the
     sequence's first token), seq_qlen[B], seq_ctx[B] (positions cached before
-    the step); want_rows[M]; pages[g] = [B, max_pages] page ids in cache group g.
+    the step), seq_base[B] (positions of the sequences before this one, after the
+    step); want_rows[M]; pages[g] = [B, max_pages] page ids in cache group g.
     Host-side: n_tokens, n_seqs, n_want, max_qlen, max_len (longest sequence
-    after the step), is_decode (every run is one token), act_dtype, device,
+    after the step), total_len (positions of all sequences after the step), query_keys
+    (pairs of a token of the step and a position it may see), is_decode (every run is one token), act_dtype, device,
     scratch (per-step memo shared by the parts, e.g. position tables).
     """
 
@@ -37,10 +39,10 @@ class StepContext:
         self.scratch: Dict = {}
         self.pages: List[torch.Tensor] = []
         self.tokens = self.tok_seq = self.tok_pos = None
-        self.seq_slot = self.seq_qstart = self.seq_qlen = self.seq_ctx = None
+        self.seq_slot = self.seq_qstart = self.seq_qlen = self.seq_ctx = self.seq_base = None
         self.want_rows = None
         self.n_tokens = self.n_seqs = self.n_want = 0
-        self.max_qlen = self.max_len = 0
+        self.max_qlen = self.max_len = self.total_len = self.query_keys = 0
         self.is_decode = False
         self.next_block = None           # the block of the run behind the current one (models of several residual streams)
         self.side_stream = None          # a second stream blocks may fork onto (decode steps only)
@@ -58,7 +60,7 @@ class _Layout:
         o = 0
         self.off: Dict[str, Tuple[int, int]] = {}
         for name, n in (("tokens", T), ("tok_seq", T), ("tok_pos", T), ("seq_slot", B),
-                        ("seq_qstart", B), ("seq_qlen", B), ("seq_ctx", B), ("want_rows", M)):
+                        ("seq_qstart", B), ("seq_qlen", B), ("seq_ctx", B), ("seq_base", B), ("want_rows", M)):
             self.off[name] = (o, n)
             o += _pad4(n)
         for g in range(groups):
@@ -157,12 +159,14 @@ class Engine:
         put("seq_qstart", np.concatenate([[0], np.cumsum(qlens)[:-1]]))
         put("seq_qlen", qlens)
         put("seq_ctx", ctxs)
+        put("seq_base", np.concatenate([[0], np.cumsum([c + q for c, q in zip(ctxs, qlens)])[:-1]]))
         put("want_rows", rows)
         for g in range(lay.groups):
             o, n = lay.off[f"pages{g}"]
             cache.page_rows(g, slots, out=buf[o:o + n].reshape(B, lay.max_pages))
         meta = dict(slots=slots, new_lens=[c + q for c, q in zip(ctxs, qlens)],
-                    max_qlen=max(qlens), is_decode=max(qlens) == 1)
+                    max_qlen=max(qlens), is_decode=max(qlens) == 1,
+                    query_keys=sum(q * c + q * (q + 1) // 2 for c, q in zip(ctxs, qlens)))
         return lay, buf, meta
 
     def _stage(self, buf: np.ndarray) -> torch.Tensor:
@@ -188,7 +192,7 @@ class Engine:
     def context(self, lay: _Layout, dev: torch.Tensor, meta: dict) -> StepContext:
         ctx = StepContext(self.device, self.act_dtype)
         for name in ("tokens", "tok_seq", "tok_pos", "seq_slot", "seq_qstart", "seq_qlen",
-                     "seq_ctx", "want_rows"):
+                     "seq_ctx", "seq_base", "want_rows"):
             o, n = lay.off[name]
             setattr(ctx, name, dev[o:o + n])
         for g in range(lay.groups):
@@ -197,6 +201,7 @@ class Engine:
         ctx.n_tokens, ctx.n_seqs, ctx.n_want = lay.T, lay.B, lay.M
         ctx.max_qlen, ctx.is_decode = meta["max_qlen"], meta["is_decode"]
         ctx.max_len = max(meta["new_lens"])
+        ctx.total_len, ctx.query_keys = sum(meta["new_lens"]), meta["query_keys"]
         if ctx.is_decode and self.overlap_branches and self.act_dtype == torch.bfloat16:
             if self._side_stream is None:
                 self._side_stream = torch.cuda.Stream(device=self.device)

@@ -124,8 +124,16 @@ class LaunchTape:
                 return False
             to[a.data_ptr()] = b.data_ptr()
 
+        def moved(u):
+            if u in to:
+                return to[u]
+            for a, b in zip(self.temps, other.temps):            # a place inside a temporary
+                if a.data_ptr() < u < a.data_ptr() + a.numel() * a.element_size():
+                    return u - a.data_ptr() + b.data_ptr()
+            return u
+
         def same_pointer(u, v):
-            return (not u and not v) or (bool(u) and to.get(u, u) == v)
+            return (not u and not v) or (bool(u) and moved(u) == v)
 
         for (f0, a0, w0, k0), (f1, a1, w1, k1) in zip(self.calls, other.calls):
             if f0 is not f1:
@@ -557,6 +565,61 @@ def attention_prefill_tc(q, out, k_cache, v_cache, seq_qstart, seq_qlen, seq_ctx
         return
     _check(_launch(lib.gl_attention_prefill_tc, byref(a), c_int(q.shape[0]), c_int(k_cache.shape[0]), _stream()),
            "attention_prefill_tc")
+
+
+class _AttnPlace(Structure):
+    _fields_ = [("seq_base", c_void_p), ("kv_ld", c_int), ("kv_rows", c_int), ("q_ld", c_int), ("chunk", c_int)]
+
+
+def prefill_tc_takes(dtype, head_dim: int, value_dim: int, score_scale: float) -> bool:
+    """Whether the tcgen05 prompt kernel takes these sizes (with queries, keys and values placed freely)."""
+    return (USE_TCGEN05 and dtype == torch.bfloat16 and value_dim == head_dim and head_dim % 16 == 0
+            and 16 <= head_dim <= TC_ATTENTION_MAX_HEAD_DIM and score_scale > 0)
+
+
+def attention_prefill_tc_chunked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, ctx, pages: torch.Tensor,
+                                 num_heads: int, num_kv_heads: int, head_dim: int, window: int = 0, chunk: int = 0,
+                                 score_scale: float = 1.0) -> torch.Tensor:
+    """attention_prefill_tc with a factor on the scores, and with chunks: a query sees the keys of its own chunk of
+    positions alone.  Returns [T, num_heads * head_dim]."""
+    out = empty((q.shape[0], num_heads * head_dim), q.dtype, q.device)
+    a = _attn_args(q, out, k_cache, v_cache, ctx.seq_qstart, ctx.seq_qlen, ctx.seq_ctx, pages, num_heads, num_kv_heads, head_dim,
+                   window, ctx.max_qlen, score_scale)
+    x = _AttnPlace(None, 0, 0, 0, chunk)
+    lib = _lib("attention_prefill_tc.cu", catalog.head_dim_defines(head_dim))
+    _check(_launch(lib.gl_attention_prefill_tc_placed, byref(a), byref(x), c_int(q.shape[0]), c_int(k_cache.shape[0]), _stream()),
+           "attention_prefill_tc")
+    return out
+
+
+def attention_rows(proj: torch.Tensor, q_off: int, kv: torch.Tensor, ctx, pages: torch.Tensor, num_heads: int, head_dim: int,
+                   value_dim: int, score_scale: float) -> torch.Tensor:
+    """Causal attention of a step's runs on keys and values that are rows of a matrix instead of cache pages: ``kv``
+    [ctx.total_len, heads * (head_dim + value_dim)] bfloat16 holds every position of every sequence, keys of all heads then
+    values of all heads, sequence b's position 0 in row ctx.seq_base[b]; queries are columns q_off.. of ``proj``.
+    Returns [T, heads * value_dim]."""
+    _need(proj, "proj", torch.bfloat16)
+    T, ld = proj.shape
+    nk, nv = num_heads * head_dim, num_heads * value_dim
+    _need(kv, "kv", torch.bfloat16, (ctx.total_len, nk + nv))
+    if q_off % 8 or ld % 8 or q_off + nk > ld or (nk + nv) % 8:
+        raise KernelError("attention_rows: rows of whole 16-byte units expected")
+    out = empty((T, nv), proj.dtype, proj.device)
+    es = proj.element_size()
+    q_ptr, k_ptr, v_ptr = proj.data_ptr() + q_off * es, kv.data_ptr(), kv.data_ptr() + nk * es
+    if prefill_tc_takes(proj.dtype, head_dim, value_dim, score_scale):
+        a = _AttnArgs(q_ptr, out.data_ptr(), k_ptr, v_ptr, ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.seq_ctx.data_ptr(),
+                      pages.data_ptr(), ctx.n_seqs, num_heads, num_heads, head_dim, pages.shape[-1], 0, ctx.max_qlen, score_scale, 0)
+        x = _AttnPlace(ctx.seq_base.data_ptr(), nk + nv, ctx.total_len, ld, 0)
+        lib = _lib("attention_prefill_tc.cu", catalog.head_dim_defines(head_dim))
+        _check(_launch(lib.gl_attention_prefill_tc_placed, byref(a), byref(x), c_int(T), c_int(0), _stream()), "attention_prefill_tc")
+        return out
+    p = _PairsArgs(q_ptr, None, k_ptr, v_ptr, ctx.seq_qstart.data_ptr(), ctx.seq_qlen.data_ptr(), ctx.seq_ctx.data_ptr(),
+                   pages.data_ptr(), ctx.n_seqs, num_heads, num_heads, 1, pages.shape[-1], 0, ctx.max_qlen, score_scale, 0.0, None,
+                   out.data_ptr(), None, 0, 0, 0, 0, ctx.seq_base.data_ptr(), nk + nv, ld)
+    fn = _lib("attention_mixed_tc.cu", catalog.pair_dim_defines(head_dim, value_dim)).gl_attention_pairs_tc
+    _check(_launch(fn, byref(p), _stream()), "attention_pairs_tc")
+    return out
 
 
 class _DecodeArgs(Structure):
@@ -1517,11 +1580,15 @@ class _PairsArgs(Structure):
                 ("seq_qstart", c_void_p), ("seq_qlen", c_void_p), ("seq_ctx", c_void_p), ("pages", c_void_p),
                 ("B", c_int), ("nH", c_int), ("nKV", c_int), ("nVal", c_int), ("max_pages", c_int), ("window", c_int),
                 ("max_qlen", c_int), ("score_scale", c_float), ("softcap", c_float), ("slopes", c_void_p),
-                ("out", c_void_p), ("sinks", c_void_p), ("nVH", c_int), ("vs", c_int), ("v_in_k", c_int), ("chunk", c_int)]
+                ("out", c_void_p), ("sinks", c_void_p), ("nVH", c_int), ("vs", c_int), ("v_in_k", c_int), ("chunk", c_int),
+                ("seq_base", c_void_p), ("kv_ld", c_int), ("q_ld", c_int)]
 
 
 USE_PAIRS_TC = True
 USE_ROWS_DECODE_TC = True      # one token a sequence, eight or more query heads on a key head: the heads as rows of a tensor-core product
+
+
+ROWS_DECODE_MIN_ROWS = 1
 
 
 class _RowsDecodeArgs(Structure):
@@ -1615,7 +1682,7 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     rows = max(n for n in range(1, 17) if share % n == 0)
     if (USE_ROWS_DECODE_TC and ctx.max_qlen == 1 and mix is None and softcap == 0.0 and slopes is None and not DEBUG_BOUNDS
             and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and head_dim % 16 == 0 and value_dim % 16 == 0
-            and head_dim <= 256 and value_dim <= 256 and (group >= 8 or values_in_keys) and rows >= 4
+            and head_dim <= 256 and value_dim <= 256 and rows >= ROWS_DECODE_MIN_ROWS
             and rows_decode_smem(head_dim, value_dim, values_in_keys) <= 227 * 1024):
         # one token a sequence and many query heads on a key head: runs of heads that share a value head are the rows
         # of a tensor-core product over the key head's pages; the ranges are put together by the mixing kernel
@@ -1721,17 +1788,18 @@ class _LatentPrepareArgs(Structure):
                 ("cosv", c_void_p), ("sinv", c_void_p), ("q_gamma", c_void_p), ("kv_gamma", c_void_p),
                 ("tok_seq", c_void_p), ("tok_pos", c_void_p), ("pages", c_void_p),
                 ("T", c_int), ("ld", c_int), ("q_rank", c_int), ("kv_rank", c_int), ("rot", c_int), ("max_pages", c_int),
-                ("n_pages", c_int), ("interleaved", c_int), ("write_kv", c_int), ("eps", c_float)]
+                ("n_pages", c_int), ("interleaved", c_int), ("write_kv", c_int), ("eps", c_float), ("c_out", c_void_p)]
 
 
 def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, ctx, pages: torch.Tensor,
                    q_rank: int, kv_rank: int, rot: int, q_gamma: Optional[torch.Tensor], kv_gamma: torch.Tensor, eps: float,
                    cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], interleaved: bool,
-                   write_kv: bool = True) -> Optional[torch.Tensor]:
+                   write_kv: bool = True, c_rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """A token's down projections proj [T, ld] = [query latent (q_rank) | c (kv_rank) | key part (rot) | ...]: both
     latents RMS-normed with their weights (32-bit), the key part rotated by the token's angles; the row [c | key part]
     goes to the token's place in k_cache [pages, 1, PAGE, kv_rank + rot], c to v_cache [pages, 1, PAGE, kv_rank]
     (``v_cache`` None or the key cache itself: the values are read from the key rows, nothing more is written).
+    ``c_rows`` [T, kv_rank]: receives c once more, a row a token.
     Returns the normed query latent [T, q_rank] (``q_rank`` 0: there is none, None)."""
     _need(proj, "proj")
     T, ld = proj.shape
@@ -1751,10 +1819,25 @@ def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     a = _LatentPrepareArgs(proj.data_ptr(), _addr(cq), k_cache.data_ptr(), _addr(v_cache), _addr(cos), _addr(sin),
                            _addr(q_gamma), kv_gamma.data_ptr(), ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(),
                            pages.data_ptr(), T, ld, q_rank, kv_rank, rot, pages.shape[-1], k_cache.shape[0],
-                           1 if interleaved else 0, 1 if write_kv else 0, eps)
+                           1 if interleaved else 0, 1 if write_kv else 0, eps, _addr(c_rows))
+    if c_rows is not None:
+        _need(c_rows, "c_rows", k_cache.dtype, (T, kv_rank))
     _check(_launch(_lib("latent.cu").gl_latent_prepare, byref(a), c_int(dtype_code(proj.dtype)),
                    c_int(dtype_code(k_cache.dtype)), _stream()), "latent_prepare")
     return cq
+
+
+def latent_rows(k_cache: torch.Tensor, ctx, pages: torch.Tensor, kv_rank: int) -> torch.Tensor:
+    """The cached latents of every position of the step's sequences (this step's too) as rows [ctx.total_len, kv_rank],
+    sequence b's position 0 in row ctx.seq_base[b]."""
+    wide = k_cache.shape[-1]
+    if tuple(k_cache.shape[1:3]) != (1, PAGE) or kv_rank > wide:
+        raise KernelError(f"latent_rows: cache pages {tuple(k_cache.shape)} do not hold latents of {kv_rank}")
+    out = empty((ctx.total_len, kv_rank), k_cache.dtype, k_cache.device)
+    _check(_launch(_lib("latent.cu").gl_latent_rows, _ptr(k_cache), _ptr(ctx.seq_base), _ptr(ctx.seq_qlen), _ptr(ctx.seq_ctx), _ptr(pages),
+                   _ptr(out), c_int(ctx.n_seqs), c_int(wide), c_int(kv_rank), c_int(pages.shape[-1]), c_int(k_cache.shape[0]),
+                   c_int(ctx.max_len), c_int(dtype_code(k_cache.dtype)), _stream()), "latent_rows")
+    return out
 
 
 class _HeadLinearArgs(Structure):

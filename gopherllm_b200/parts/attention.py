@@ -331,6 +331,11 @@ class MixedHeadAttention(Mixer):
                                      self.vdim, s.q_scale, cos, sin, s.position.interleaved,
                                      self.q_gamma, self.k_gamma, self.eps, write_kv=cache.writes,
                                      q_temp=self.q_temp, q_only=self.shared_kv, head_unit=self.head_unit)
+        if (not ctx.is_decode and self.mix is None and self.softcap == 0.0 and self.slopes is None and self.sinks is None
+                and ops.prefill_tc_takes(q.dtype, s.head_dim, self.vdim, self.score_scale) and not ops.DEBUG_BOUNDS):
+            o = ops.attention_prefill_tc_chunked(q, cache.k, cache.v, ctx, pages, s.num_heads, s.num_kv_heads, s.head_dim,
+                                                 window=s.window, chunk=self.chunk, score_scale=self.score_scale)
+            return o, self.w_out, self.b_out
         o = ops.attention_mixed(q, cache.k, cache.v, ctx, pages, s.num_heads, s.num_kv_heads, s.head_dim, self.vdim,
                                 mix=self.mix, window=s.window, score_scale=self.score_scale, softcap=self.softcap,
                                 slopes=self.slopes, sinks=self.sinks, chunk=self.chunk)
@@ -346,6 +351,9 @@ class MixedHeadAttention(Mixer):
         return ops.linear(o, w, b, add0=a0, add1=a1, out_dtype=torch.float32, out=out)
 
 
+LATENT_BUILDS_KEYS = True        # (False: prompts too run on the latents as they are; for comparison)
+
+
 class LatentAttention(Mixer):
     """Softmax attention whose keys and values are read out of a small latent per position.
 
@@ -359,7 +367,14 @@ class LatentAttention(Mixer):
     every query head becomes a row [W_uk,h^T q_h | its rotated part] of kv_rank + rot numbers, attention runs as
     ``num_heads`` query heads on ONE key head with values of size kv_rank, and W_uv,h is applied to a head's result.
     The three down projections (query latent, [c' | k_r], gates) are one product; the per-head products are
-    csrc/latent.cu's.  Options: ``q_rank`` (0: there is no query latent, q = W_q x, and its rows ride in the first product),
+    csrc/latent.cu's.
+
+    That form costs 2 (kv_rank + rot) + 2 kv_rank operations per head, query and key, keys and values built first cost
+    2 (head_dim + value_dim), and their building 2 kv_rank (head_dim + value_dim) per head and position.  Prompts in
+    bfloat16 without a rotated part, window, sink or gate therefore build all heads' keys and values of their sequences' positions
+    as one product of the latents (``_builds_keys`` weighs the two), and attention reads them as rows of its result.
+
+     Options: ``q_rank`` (0: there is no query latent, q = W_q x, and its rows ride in the first product),
     ``kv_rank``, ``rot`` (the position encoding's rotary size), ``score_scale``, ``norm_eps``, ``sink``, ``gate``."""
 
     deferred_add = True
@@ -383,7 +398,7 @@ class LatentAttention(Mixer):
         self.eps = float(spec.option("norm_eps", 1e-6))
         self.score_scale = float(spec.option("score_scale", 1.0))
         self.position = build_position(spec.position)
-        self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_out = None
+        self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_kv = self.w_out = None
         self.q_gamma = self.kv_gamma = self.sinks = None
         self.q_off = self.gate_off = 0           # columns of the first product: queries (without a query latent), gates
 
@@ -431,6 +446,14 @@ class LatentAttention(Mixer):
         # W_uk,h^T as a product's weight [out = kv_rank, in = head_dim], head by head
         self.w_uk_t = t["uk.weight"].view(H, s.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = t["uv.weight"].view(H, self.vdim, self.kv_rank).contiguous()
+        self.w_kv = None
+        D, V = s.head_dim, self.vdim
+        if (not self.q_rank and not self.rot and not self.sink and not self.gate and s.window == 0 and self.score_scale > 0
+                and t["uk.weight"].dtype == t["uv.weight"].dtype == torch.bfloat16 and self.kv_rank % 8 == 0
+                and D % 16 == 0 and V % 16 == 0 and D <= 256 and V <= 256):
+            # all heads' keys, then all heads' values, as one product of the latent
+            self.w_kv = torch.cat([t["uk.weight"], t["uv.weight"]], 0).contiguous()
+            self.w_uv = self.w_kv[H * D:].view(H, V, self.kv_rank)
         self.w_out = t["o.weight"]
         self.q_gamma, self.kv_gamma = t.get("dq.norm.weight"), t["dkv.norm.weight"]
         self.sinks = t.get("sink")
@@ -445,9 +468,28 @@ class LatentAttention(Mixer):
     def first_product(self):
         return self.w_down, None, None
 
+    def _builds_keys(self, ctx) -> bool:
+        s = self.spec
+        both = s.head_dim + self.vdim
+        if (ctx.max_qlen < 16 or self.w_kv is None or ctx.act_dtype != torch.bfloat16 or ops.DEBUG_BOUNDS or not ops.USE_PAIRS_TC
+                or not LATENT_BUILDS_KEYS):
+            return False
+        # (a product's operations are several times cheaper than the attention kernels')
+        return ctx.query_keys * (2 * self.kv_rank - both) > ctx.total_len * self.kv_rank * both / 4
+
     def until_last(self, xn, ctx, cache, first=None):
         s, H = self.spec, self.spec.num_heads
         proj = first if first is not None else ops.linear(xn, self.w_down, None, out_dtype=ctx.act_dtype)
+        if self._builds_keys(ctx):
+            pages = ctx.pages[cache.group]
+            fresh = cache.writes and ctx.total_len == ctx.n_tokens        # nothing was cached before: the step's own latents
+            c = ops.empty((ctx.n_tokens, self.kv_rank), ctx.act_dtype, xn.device) if fresh else None
+            ops.latent_prepare(proj, cache.k, cache.v, ctx, pages, 0, self.kv_rank, 0, None, self.kv_gamma, self.eps, None, None,
+                               False, write_kv=cache.writes, c_rows=c)
+            if c is None:
+                c = ops.latent_rows(cache.k, ctx, pages, self.kv_rank)
+            kv = ops.linear(c, self.w_kv, None, out_dtype=ctx.act_dtype)
+            return ops.attention_rows(proj, self.q_off, kv, ctx, pages, H, s.head_dim, self.vdim, self.score_scale), self.w_out, None
         tables = self.position.tables(ctx)
         cos, sin = tables if tables is not None else (None, None)
         pages = ctx.pages[cache.group]
