@@ -426,6 +426,114 @@ attn_group_decode_kernel(MixedAttnArgs a) {
     }
 }
 
+// The factors on a head's ranges' sums, by one warp: coef[s] = e^(m_s - m) / (sum of all ranges, the sink's share in it),
+// from each range's maximum and sum (ml [splits, 2]); up to 64 ranges.
+__device__ __forceinline__ void am_range_factors(const float* ml, int splits, const float* sinks, int h, float* coef) {
+    const int lane = threadIdx.x & 31;
+    const float m0 = lane < splits ? ml[2 * lane] : -INFINITY, m1 = lane + 32 < splits ? ml[2 * (lane + 32)] : -INFINITY;
+    const float l0 = lane < splits ? ml[2 * lane + 1] : 0.f, l1 = lane + 32 < splits ? ml[2 * (lane + 32) + 1] : 0.f;
+    const float m = gl_warp_max(fmaxf(m0, m1));
+    const float e0 = m0 > -INFINITY ? expf(m0 - m) : 0.f, e1 = m1 > -INFINITY ? expf(m1 - m) : 0.f;
+    const float inv = am_finish(m, gl_warp_sum(l0 * e0 + l1 * e1), sinks, h);
+    if (lane < splits) coef[lane] = e0 * inv;
+    if (lane + 32 < splits) coef[lane + 32] = e1 * inv;
+}
+
+// The ranges put together and a product per head behind them: out[b, h, :] = W_h y_h (times sigmoid(gate[b, h]) where there
+// is a gate) with y_h as above, 32-bit until out is rounded.  For attention on latents, whose values are read out of the
+// weighted latent: few tokens, so a block takes up to AP_TOKENS tokens of a head and a run of output rows; the merged
+// latents stay in shared memory, a warp an output row at a time (a lane 16 bytes of it), and the row is fetched before the
+// kernel waits for the one that leaves the ranges.
+#define AP_TOKENS 8
+#define AP_THREADS 256
+struct MergeProjectArgs {
+    const float* parts;       // [B, nH, splits, R]
+    const float* ml;          // [B, nH, splits, 2]
+    const void* w;            // [nH, N, R] weight type bf16
+    const void* gate;         // activation type or null, row pitch g_ld, head h's at column g_off + h
+    const float* sinks;       // [nH] or null
+    const int* seq_qstart;    // [B]
+    void* out;                // [T, nH*N] bf16
+    int B, nH, N, R, splits, rows_per_block, g_ld, g_off;
+};
+
+__global__ void __launch_bounds__(AP_THREADS)
+merge_project_kernel(MergeProjectArgs a) {
+    extern __shared__ float smem[];
+    float* coef = smem;                                 // [AP_TOKENS][64]
+    float* y = coef + AP_TOKENS * 64;                   // [AP_TOKENS][R]
+    gl_grid_launch_dependents();
+    const int h = blockIdx.y, b0 = blockIdx.z * AP_TOKENS, n0 = blockIdx.x * a.rows_per_block;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int tokens = min(AP_TOKENS, a.B - b0), n_end = min(a.N, n0 + a.rows_per_block);
+    const __nv_bfloat16* W = (const __nv_bfloat16*)a.w + (size_t)h * a.N * a.R;
+    uint4 first = make_uint4(0, 0, 0, 0);               // this warp's first row, first pieces
+    if (n0 + warp < n_end && lane * 8 < a.R) first = *(const uint4*)(W + (size_t)(n0 + warp) * a.R + lane * 8);
+    gl_grid_wait();
+    if (warp < tokens) am_range_factors(a.ml + ((size_t)(b0 + warp) * a.nH + h) * a.splits * 2, a.splits, a.sinks, h, coef + warp * 64);
+    __syncthreads();
+    for (int i = threadIdx.x; i < tokens * a.R; i += AP_THREADS) {
+        const int t = i / a.R, d = i - t * a.R;
+        const float* src = a.parts + ((size_t)(b0 + t) * a.nH + h) * a.splits * a.R + d;
+        const float* c = coef + t * 64;
+        float v = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < a.splits; ++s) v = fmaf(c[s], src[(size_t)s * a.R], v);
+        y[i] = v;
+    }
+    __syncthreads();
+    for (int n = n0 + warp; n < n_end; n += AP_THREADS / 32) {
+        float acc[AP_TOKENS];
+#pragma unroll
+        for (int t = 0; t < AP_TOKENS; ++t) acc[t] = 0.f;
+        for (int k = lane * 8; k < a.R; k += 256) {
+            const uint4 raw = (n == n0 + warp && k == lane * 8) ? first : *(const uint4*)(W + (size_t)n * a.R + k);
+            const __nv_bfloat162* p2 = (const __nv_bfloat162*)&raw;
+            float w[8];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(p2[e]);
+                w[2 * e] = f.x;
+                w[2 * e + 1] = f.y;
+            }
+#pragma unroll
+            for (int t = 0; t < AP_TOKENS; ++t) {
+                if (t < tokens) {
+                    const float4 u = *(const float4*)(y + t * a.R + k), v = *(const float4*)(y + t * a.R + k + 4);
+                    acc[t] = fmaf(w[0], u.x, fmaf(w[1], u.y, fmaf(w[2], u.z, fmaf(w[3], u.w, acc[t]))));
+                    acc[t] = fmaf(w[4], v.x, fmaf(w[5], v.y, fmaf(w[6], v.z, fmaf(w[7], v.w, acc[t]))));
+                }
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < AP_TOKENS; ++t) {
+            if (t < tokens) {
+                const float s = gl_warp_sum(acc[t]);
+                if (lane == 0) {
+                    const size_t row = (size_t)a.seq_qstart[b0 + t];
+                    const float mul = a.gate ? 1.0f / (1.0f + expf(-gl_load((const __nv_bfloat16*)a.gate + row * a.g_ld + a.g_off + h))) : 1.0f;
+                    ((__nv_bfloat16*)a.out)[(row * a.nH + h) * a.N + n] = __float2bfloat16_rn(s * mul);
+                }
+            }
+        }
+    }
+}
+
+GL_API int gl_merge_project(const MergeProjectArgs* args, cudaStream_t stream) {
+    MergeProjectArgs a = *args;
+    if (a.B <= 0) return GL_OK;
+    if (a.nH <= 0 || a.N <= 0 || a.R <= 0 || a.R % 8 || a.R > 1024 || a.splits <= 0 || a.splits > 64 || !a.parts || !a.ml) return GL_ERR_SHAPE;
+    if ((uintptr_t)a.w & 15) return GL_ERR_ALIGN;
+    const int groups = (a.B + AP_TOKENS - 1) / AP_TOKENS;
+    if (groups > 65535 || a.nH > 65535) return GL_ERR_SHAPE;
+    // every block of a head puts its tokens' ranges together again: more than one only where the grid would be small
+    a.rows_per_block = a.N;
+    while (a.rows_per_block > 8 && (long long)groups * a.nH * ((a.N + a.rows_per_block - 1) / a.rows_per_block) < 128) a.rows_per_block = (a.rows_per_block + 1) / 2;
+    const dim3 grid((a.N + a.rows_per_block - 1) / a.rows_per_block, a.nH, groups);
+    const size_t smem = (size_t)AP_TOKENS * (64 + a.R) * sizeof(float);
+    return gl_launch(merge_project_kernel, grid, dim3(AP_THREADS), smem, stream, 1, a) == 0 ? GL_OK : GL_ERR_LAUNCH;
+}
+
 // out[b, h, :] = sum_g M[h, g] * (sum_s parts[b, g, c(h), s, :] e^(m_gs - m_g)) / (sum_s l_gs e^(m_gs - m_g))
 template <typename TA>
 __global__ void __launch_bounds__(128)
@@ -434,6 +542,19 @@ head_mix_split_kernel(MixedAttnArgs a) {
     gl_grid_launch_dependents();
     gl_grid_wait();
     const int b = blockIdx.y, h = blockIdx.x;
+    if (!a.mix && a.splits <= 64) {                     // one head's ranges: a lane a range, or two
+        if (threadIdx.x < 32) am_range_factors(a.ml + ((size_t)b * a.nH + h) * a.splits * 2, a.splits, a.sinks, h, coef);
+        __syncthreads();
+        const float* src = a.parts + ((size_t)b * a.nH + h) * a.splits * a.vd;
+        const size_t row = (size_t)a.seq_qstart[b];
+        for (int d = threadIdx.x; d < a.vd; d += blockDim.x) {
+            float y = 0.f;
+#pragma unroll 8
+            for (int s = 0; s < a.splits; ++s) y = fmaf(coef[s], src[(size_t)s * a.vd + d], y);
+            gl_store((TA*)a.out + (row * a.nH + h) * a.vd + d, y);
+        }
+        return;
+    }
     const int nVal = a.mix ? a.nKV : 1;
     const int c = a.mix ? h / (a.nH / a.nKV) : 0;
     const int row = a.seq_qstart[b];

@@ -15,9 +15,23 @@
 // 1 - a^2 = d (2 - d).
 #include "common.cuh"
 
-__device__ __forceinline__ float gu_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+// FAST: the hardware's exponential, reciprocal and square root, each off by a few 2^-23 of its value.  They enter the
+// recurrence as errors of that size in log a and in what is written, which the 16-bit rounding of u outweighs by far;
+// the 32-bit path takes the exact forms.
+template <bool FAST>
+__device__ __forceinline__ float gu_sigmoid(float x) {
+    return FAST ? __fdividef(1.0f, 1.0f + __expf(-x)) : 1.0f / (1.0f + expf(-x));
+}
+template <bool FAST>
+__device__ __forceinline__ float gu_sqrt(float x) {
+    if (!FAST) return sqrtf(x);
+    float y;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 // 1 - e^x for x <= 0: near zero from the series of e^x - 1 to x^9/9! (below 2^-28 here), Horner in 32-bit
+template <bool FAST>
 __device__ __forceinline__ float gu_one_minus_exp(float x) {
     if (x > -0.5f) {
         float p = 2.755731922e-6f;
@@ -31,7 +45,7 @@ __device__ __forceinline__ float gu_one_minus_exp(float x) {
         p = fmaf(p, x, 1.0f);
         return -p * x;
     }
-    return 1.0f - expf(x);
+    return 1.0f - (FAST ? __expf(x) : expf(x));
 }
 
 struct UnitGatesArgs {
@@ -50,14 +64,30 @@ struct UnitGatesArgs {
 };
 
 // a channel's gates' sums to its decay and input
+template <bool FAST>
 __device__ __forceinline__ float2 gu_factors(float rs, float is, float u, float rate) {
-    const float d = gu_one_minus_exp(rate * gu_sigmoid(rs));
-    return make_float2(1.0f - d, sqrtf(d * (2.0f - d)) * gu_sigmoid(is) * u);
+    const float d = gu_one_minus_exp<FAST>(rate * gu_sigmoid<FAST>(rs));
+    return make_float2(1.0f - d, gu_sqrt<FAST>(d * (2.0f - d)) * gu_sigmoid<FAST>(is) * u);
+}
+
+// the other branch's activation, for results rounded to TA
+template <typename TA>
+__device__ __forceinline__ float gu_gelu(float y) {
+    if constexpr (sizeof(TA) == 2) return gl_activate_bf16_grade(y, GL_ACT_GELU_TANH);
+    else return gl_activate<true>(y, GL_ACT_GELU_TANH);
 }
 
 template <typename TA>
+__device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u, float2 bias, float rate);
+
+template <typename TA>
 __device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u) {
-    const float2 f = gu_factors(rs + g.bias[2 * c], is + g.bias[2 * c + 1], u, g.rate[c]);
+    gu_finish<TA>(g, t, c, rs, is, u, *(const float2*)(g.bias + 2 * c), g.rate[c]);
+}
+
+template <typename TA>
+__device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u, float2 bias, float rate) {
+    const float2 f = gu_factors<sizeof(TA) == 2>(rs + bias.x, is + bias.y, u, rate);
     if (!g.step) {
         g.ab[(size_t)t * g.C + c] = f;
         return;
@@ -66,7 +96,7 @@ __device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, 
     const float s = fmaf(f.x, *S, f.y);
     *S = s;
     gl_store((TA*)g.out + (size_t)t * g.C + c,
-             s * gl_activate<true>(gl_load((const TA*)g.y + (size_t)t * g.y_ld + g.y_off + c), GL_ACT_GELU_TANH));
+             s * gu_gelu<TA>(gl_load((const TA*)g.y + (size_t)t * g.y_ld + g.y_off + c)));
 }
 
 #define GG_BM 64
@@ -220,8 +250,10 @@ unit_gates_tc_kernel(UnitGatesArgs g) {
         const int n = n0 + j * 8 + 2 * t;
         if (n >= N) continue;
         const int c = n / 2, cc = blockIdx.z * size + c;
-        if (r_lo < g.T) gu_finish<__nv_bfloat16>(g, r_lo, cc, acc[j][0], acc[j][1], gl_load(U + (size_t)r_lo * g.C + c));
-        if (r_hi < g.T) gu_finish<__nv_bfloat16>(g, r_hi, cc, acc[j][2], acc[j][3], gl_load(U + (size_t)r_hi * g.C + c));
+        const float2 bias = *(const float2*)(g.bias + 2 * cc);
+        const float rate = g.rate[cc];
+        if (r_lo < g.T) gu_finish<__nv_bfloat16>(g, r_lo, cc, acc[j][0], acc[j][1], gl_load(U + (size_t)r_lo * g.C + c), bias, rate);
+        if (r_hi < g.T) gu_finish<__nv_bfloat16>(g, r_hi, cc, acc[j][2], acc[j][3], gl_load(U + (size_t)r_hi * g.C + c), bias, rate);
     }
 }
 
@@ -243,14 +275,14 @@ GL_API int gl_unit_gates(const UnitGatesArgs* args, int act_dtype, int w_dtype, 
 }
 
 // ---------------------------------------------------------------------------
-// The recurrence of a prompt.  A block owns 16 channels of one sequence and walks its run in pieces of 256 tokens: 32
-// segments of 8 consecutive tokens, a thread a (segment, channel).  A segment is the map S -> P S + Q (P the product
+// The recurrence of a prompt.  A block owns 16 channels of one sequence and walks its run in pieces of 128 tokens: 32
+// segments of 4 consecutive tokens, a thread a (segment, channel).  A segment is the map S -> P S + Q (P the product
 // of its decays, Q its result from zero); a warp a channel puts the 32 maps together in order, and every thread then
-// walks its 8 tokens from its segment's start.  The next piece's factors travel while this one is put together.
+// walks its 4 tokens from its segment's start.  The next piece's factors travel while this one is put together.
 // ---------------------------------------------------------------------------
 #define US_CH 16
 #define US_SEG 32
-#define US_LEN 8
+#define US_LEN 4
 
 struct UnitScanArgs {
     const float2* ab;         // [T, C]
@@ -264,7 +296,7 @@ struct UnitScanArgs {
 };
 
 template <typename TA>
-__global__ void __launch_bounds__(US_CH * US_SEG)
+__global__ void __launch_bounds__(US_CH * US_SEG, 2)
 unit_scan_kernel(UnitScanArgs a) {
     __shared__ float sP[US_CH][US_SEG + 1], sQ[US_CH][US_SEG + 1];
     gl_grid_launch_dependents();
@@ -318,7 +350,7 @@ unit_scan_kernel(UnitScanArgs a) {
         for (int k = 0; k < US_LEN; ++k) {
             const int t = s0 + seg * US_LEN + k;
             S = fmaf(f[k].x, S, f[k].y);
-            if (live && t < qlen) gl_store(out + (size_t)t * a.C, S * gl_activate<true>(yv[k], GL_ACT_GELU_TANH));
+            if (live && t < qlen) gl_store(out + (size_t)t * a.C, S * gu_gelu<TA>(yv[k]));
         }
         __syncthreads();
 #pragma unroll

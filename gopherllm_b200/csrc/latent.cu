@@ -37,14 +37,10 @@ struct LatentPrepareArgs {
     void* c_out;              // [T, kv_rank] cache type or null: c once more, a row a token
 };
 
+// token t by the whole block (up to 256 threads); smem: a row of the down projections, 32-bit
 template <typename TA, typename TC>
-__global__ void __launch_bounds__(256)
-latent_prepare_kernel(LatentPrepareArgs a) {
-    extern __shared__ float smem[];
+__device__ __forceinline__ void latent_prepare_token(const LatentPrepareArgs& a, int t, float* smem) {
     __shared__ float red[2][8];
-    gl_grid_launch_dependents();
-    gl_grid_wait();
-    const int t = blockIdx.x;
     const int n = a.q_rank + a.kv_rank + a.rot;
     const TA* row = (const TA*)a.proj + (size_t)t * a.ld;
     float* v = smem;
@@ -94,6 +90,15 @@ latent_prepare_kernel(LatentPrepareArgs a) {
     } else {
         for (int i = threadIdx.x; i < a.rot; i += blockDim.x) gl_store(kr + a.kv_rank + i, kp[i]);
     }
+}
+
+template <typename TA, typename TC>
+__global__ void __launch_bounds__(256)
+latent_prepare_kernel(LatentPrepareArgs a) {
+    extern __shared__ float smem[];
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    latent_prepare_token<TA, TC>(a, blockIdx.x, smem);
 }
 
 GL_API int gl_latent_prepare(const LatentPrepareArgs* args, int act_dtype, int cache_dtype, cudaStream_t stream) {
@@ -264,13 +269,9 @@ __device__ __forceinline__ void ht_mma(float (&d)[4], const unsigned (&a)[4], un
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-__global__ void __launch_bounds__(128)
-head_linear_tc_kernel(HeadLinearArgs g) {
+__device__ __forceinline__ void head_linear_tc_tile(const HeadLinearArgs& g, int h) {
     __shared__ __align__(16) unsigned char sA[64 * HT_ROW];
     __shared__ __align__(16) unsigned char sW[64 * HT_ROW];
-    gl_grid_launch_dependents();
-    gl_grid_wait();
-    const int h = blockIdx.z;
     const __nv_bfloat16* X = (const __nv_bfloat16*)g.x + (size_t)h * g.x_head + g.x_off;
     const __nv_bfloat16* W = (const __nv_bfloat16*)g.w + (size_t)h * g.N * g.K;
     __nv_bfloat16* O = (__nv_bfloat16*)g.out + (size_t)h * g.o_head + g.o_off;
@@ -349,6 +350,47 @@ head_linear_tc_kernel(HeadLinearArgs g) {
     }
 }
 
+__global__ void __launch_bounds__(128)
+head_linear_tc_kernel(HeadLinearArgs g) {
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    head_linear_tc_tile(g, blockIdx.z);
+}
+
+// Both readers of the down projections in one grid where there is no query latent between them: the first H slices take
+// the queries' products, the slices behind them a token a block for its latent.
+__global__ void __launch_bounds__(128)
+latent_queries_kernel(LatentPrepareArgs a, HeadLinearArgs g) {
+    extern __shared__ float smem[];
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    if ((int)blockIdx.z < g.H) {
+        head_linear_tc_tile(g, blockIdx.z);
+        return;
+    }
+    const int t = ((int)(blockIdx.z - g.H) * gridDim.y + blockIdx.y) * gridDim.x + blockIdx.x;
+    if (t < a.T) latent_prepare_token<__nv_bfloat16, __nv_bfloat16>(a, t, smem);
+}
+
+static bool head_linear_takes_tc(const HeadLinearArgs& g) {
+    return g.K % 16 == 0 && g.N % 8 == 0 && g.x_row % 8 == 0 && g.x_head % 8 == 0 && g.x_off % 8 == 0 && g.o_row % 2 == 0 &&
+           g.o_head % 2 == 0 && g.o_off % 2 == 0 && !(((uintptr_t)g.x | (uintptr_t)g.w) & 15) && !((uintptr_t)g.out & 3);
+}
+
+// bfloat16 throughout; GL_ERR_SHAPE for sizes the tensor-core form does not take (the caller then launches the two alone)
+GL_API int gl_latent_queries(const LatentPrepareArgs* prepare, const HeadLinearArgs* queries, cudaStream_t stream) {
+    const LatentPrepareArgs& a = *prepare;
+    const HeadLinearArgs& g = *queries;
+    if (a.T <= 0) return GL_OK;
+    if (a.q_rank != 0 || a.kv_rank <= 0 || a.rot < 0 || a.rot % 2 || a.ld < a.kv_rank + a.rot || g.T != a.T || g.H <= 0 || g.N <= 0 ||
+        g.K <= 0 || g.tail < 0 || (g.cosv && g.tail % 2) || !head_linear_takes_tc(g)) return GL_ERR_SHAPE;
+    const size_t smem = (size_t)(a.kv_rank + a.rot) * sizeof(float);
+    const unsigned gx = (g.N + HL_BN - 1) / HL_BN, gy = (g.T + HL_BM - 1) / HL_BM;
+    const unsigned slices = (a.T + gx * gy - 1) / (gx * gy);
+    if (gy > 65535 || g.H + slices > 65535 || smem > 24 * 1024) return GL_ERR_SHAPE;
+    return gl_launch(latent_queries_kernel, dim3(gx, gy, g.H + slices), dim3(128), smem, stream, 1, a, g) == 0 ? GL_OK : GL_ERR_LAUNCH;
+}
+
 GL_API int gl_head_linear(const HeadLinearArgs* args, int act_dtype, int w_dtype, cudaStream_t stream) {
     const HeadLinearArgs& g = *args;
     if (g.T <= 0 || g.H <= 0) return GL_OK;
@@ -356,9 +398,7 @@ GL_API int gl_head_linear(const HeadLinearArgs* args, int act_dtype, int w_dtype
     const dim3 grid((g.N + HL_BN - 1) / HL_BN, (g.T + HL_BM - 1) / HL_BM, g.H);
     if (grid.y > 65535) return GL_ERR_SHAPE;
     int rc;
-    if (act_dtype == GL_BF16 && w_dtype == GL_BF16 && g.K % 16 == 0 && g.N % 8 == 0 && g.x_row % 8 == 0 && g.x_head % 8 == 0 &&
-        g.x_off % 8 == 0 && g.o_row % 2 == 0 && g.o_head % 2 == 0 && g.o_off % 2 == 0 &&
-        !(((uintptr_t)g.x | (uintptr_t)g.w) & 15) && !((uintptr_t)g.out & 3))
+    if (act_dtype == GL_BF16 && w_dtype == GL_BF16 && head_linear_takes_tc(g))
         return gl_launch(head_linear_tc_kernel, grid, dim3(128), 0, stream, 1, g) == 0 ? GL_OK : GL_ERR_LAUNCH;
     if (act_dtype == GL_F32 && w_dtype == GL_F32) rc = gl_launch(head_linear_kernel<float, float>, grid, dim3(256), 0, stream, 1, g);
     else if (act_dtype == GL_BF16 && w_dtype == GL_BF16)

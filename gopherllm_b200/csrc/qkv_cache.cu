@@ -485,11 +485,67 @@ qkv_rownorm_cache_kernel(QkvRowNormArgs a) {
     }
 }
 
+// The same for bfloat16 without any norm, temperature or table, neighbouring dims turned together, every size in whole
+// 16-byte pieces: a piece a thread, turned in registers (its four pairs are its own), no shared memory.
+__global__ void __launch_bounds__(256)
+qkv_pieces_cache_kernel(QkvRowNormArgs a) {
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    const int nq = a.nH * a.hd, nk = a.q_only ? 0 : a.nKV * a.hd, nv = a.q_only ? 0 : a.nKV * a.vd;
+    const int per = (nq + nk + nv) / 8;
+    const long long n = (long long)a.T * per;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const int t = (int)(i / per), col = (int)(i - (long long)t * per) * 8;
+        uint4 raw = *(const uint4*)((const __nv_bfloat16*)a.qkv + (size_t)t * a.ld + col);
+        const bool is_q = col < nq, is_k = !is_q && col < nq + nk;
+        const int at = is_q ? col : (is_k ? col - nq : col - nq - nk);          // column among queries, keys or values
+        const int size = is_q || is_k ? a.hd : a.vd;
+        const int head = at / size, d = at - head * size;
+        if (is_q || is_k) {
+            const bool turned = a.cosv && d < 2 * a.half;
+            if (turned || (is_q && a.q_scale != 1.0f)) {
+                __nv_bfloat162* p2 = (__nv_bfloat162*)&raw;
+                const float mul = is_q ? a.q_scale : 1.0f;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float2 f = __bfloat1622float2(p2[e]);
+                    float u = f.x, x = f.y;
+                    const int k = d / 2 + e;
+                    if (turned && k < a.half) {
+                        const float c = a.cosv[(size_t)t * a.half + k], s = a.sinv[(size_t)t * a.half + k];
+                        const float v = u * c - x * s;
+                        x = x * c + u * s;
+                        u = v;
+                    }
+                    p2[e] = __floats2bfloat162_rn(u * mul, x * mul);
+                }
+            }
+        }
+        if (is_q) {
+            *(uint4*)((__nv_bfloat16*)a.q_out + (size_t)t * nq + col) = raw;
+            continue;
+        }
+        if (!a.write_kv) continue;
+        const int pos = a.tok_pos[t];
+        const int slot = gl_checked(pos / GL_PAGE, a.max_pages, GL_BAD_POSITION);
+        const int page = gl_checked(a.pages[(size_t)a.tok_seq[t] * a.max_pages + slot], a.n_pages > 0 ? a.n_pages : 0x7fffffff, GL_BAD_PAGE);
+        __nv_bfloat16* dst = (__nv_bfloat16*)(is_k ? a.k_cache : a.v_cache);
+        *(uint4*)(dst + (((size_t)page * a.nKV + head) * GL_PAGE + (pos % GL_PAGE)) * size + d) = raw;
+    }
+}
+
 GL_API int gl_qkv_rownorm_cache(const QkvRowNormArgs* args, int act_dtype, int cache_dtype, cudaStream_t stream) {
     const QkvRowNormArgs& a = *args;
     if (a.T <= 0) return GL_OK;
     if (a.hd <= 0 || a.vd <= 0 || a.nH <= 0 || a.nKV <= 0 || 2 * a.half > a.hd) return GL_ERR_SHAPE;
     const size_t smem = ((size_t)(a.nH + a.nKV) * a.hd + (a.talk ? (size_t)a.nH * a.nH : 0)) * sizeof(float);
+    if (act_dtype == GL_BF16 && cache_dtype == GL_BF16 && !a.q_gamma && !a.k_gamma && !a.head_unit && !a.talk && !a.k_joined &&
+        a.temp_every <= 0.f && (a.interleaved || !a.cosv) && a.hd % 8 == 0 && a.vd % 8 == 0 && a.ld % 8 == 0 &&
+        !(((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15)) {
+        const long long n = (long long)a.T * ((a.nH + (a.q_only ? 0 : a.nKV)) * a.hd + (a.q_only ? 0 : a.nKV * a.vd)) / 8;
+        const long long want = (n + 255) / 256;
+        return gl_launch(qkv_pieces_cache_kernel, dim3((unsigned)(want > 32768 ? 32768 : want)), dim3(256), 0, stream, 1, a);
+    }
     if (smem > 200 * 1024) return GL_ERR_SMEM;
     // few tokens: more threads a token, so that a row's loads are in flight together; a table on the queries: a thread
     // a column of the wide rows

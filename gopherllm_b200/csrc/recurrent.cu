@@ -685,8 +685,92 @@ conv_silu_wide_kernel(ConvArgs a) {
     mc_store16((TA*)a.out + (size_t)t * a.C + c0, acc);
 }
 
+// The same for runs of tokens: a thread takes 16 bytes of channels of four consecutive tokens, so that the weights and
+// the rows the four windows share are fetched once.  (Four tokens that are not of one sequence go one by one.)
+template <typename TA, int TAPS>
+__global__ void __launch_bounds__(256)
+conv_silu_tokens_kernel(ConvArgs a) {
+    constexpr int VEC = 16 / (int)sizeof(TA), NT = 4, back = TAPS - 1;
+    gl_grid_launch_dependents();
+    gl_grid_wait();
+    const int CV = a.C / VEC;
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const int t0 = (int)(i / CV) * NT, c0 = (int)(i - (long long)(t0 / NT) * CV) * VEC;
+    if (t0 >= a.T) return;
+    __align__(16) float w[VEC * TAPS], bias[VEC];
+#pragma unroll
+    for (int q = 0; q < VEC * TAPS / 4; ++q)
+        reinterpret_cast<float4*>(w)[q] = reinterpret_cast<const float4*>(a.w + (size_t)c0 * TAPS)[q];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) bias[k] = a.bias ? a.bias[c0 + k] : 0.f;
+    const int n = min(NT, a.T - t0);
+    const int b_first = a.tok_seq[t0];
+    const bool together = n == NT && b_first == a.tok_seq[t0 + NT - 1];
+    const int idx0 = t0 - a.seq_qstart[b_first];
+    const TA* x = (const TA*)a.x + a.x_off + c0;
+    if (together && idx0 >= back) {
+        __align__(16) float v[TAPS][VEC];             // rows t - back .. t, in a ring
+#pragma unroll
+        for (int j = 0; j < back; ++j) mc_load16(x + (size_t)(t0 - back + j) * a.ld, v[j]);
+#pragma unroll
+        for (int s = 0; s < NT; ++s) {
+            mc_load16(x + (size_t)(t0 + s) * a.ld, v[(s + back) % TAPS]);
+            __align__(16) float acc[VEC];
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) acc[k] = bias[k];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w[k * TAPS + j], v[(s + j) % TAPS][k], acc[k]);
+            if (a.silu) {
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) acc[k] = rc_silu(acc[k]);
+            }
+            mc_store16((TA*)a.out + (size_t)(t0 + s) * a.C + c0, acc);
+        }
+        return;
+    }
+    for (int s = 0; s < n; ++s) {
+        const int t = t0 + s, b = a.tok_seq[t], idx = t - a.seq_qstart[b];
+        const float* tail = a.state + (size_t)a.seq_slot[b] * a.state_stride + a.tail_off;
+        __align__(16) float acc[VEC], v[VEC];
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) acc[k] = bias[k];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const int rel = idx - back + j;
+            if (rel >= 0) {
+                mc_load16(x + (size_t)(t - back + j) * a.ld, v);
+            } else {
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) v[k] = tail[(size_t)(c0 + k) * back + rel + back];
+            }
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w[k * TAPS + j], v[k], acc[k]);
+        }
+        if (a.silu) {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) acc[k] = rc_silu(acc[k]);
+        }
+        mc_store16((TA*)a.out + (size_t)t * a.C + c0, acc);
+    }
+}
+
+template <typename TA>
+static int launch_conv_silu_tokens(const ConvArgs& a, cudaStream_t stream) {
+    const long long n = (long long)((a.T + 3) / 4) * (a.C / (16 / (int)sizeof(TA)));
+    const dim3 grid((unsigned)((n + 255) / 256));
+    switch (a.taps) {
+        case 2: return gl_launch(conv_silu_tokens_kernel<TA, 2>, grid, dim3(256), 0, stream, 1, a);
+        case 3: return gl_launch(conv_silu_tokens_kernel<TA, 3>, grid, dim3(256), 0, stream, 1, a);
+        default: return gl_launch(conv_silu_tokens_kernel<TA, 4>, grid, dim3(256), 0, stream, 1, a);
+    }
+}
+
 template <typename TA>
 static int launch_conv_silu_wide(const ConvArgs& a, dim3 grid, cudaStream_t stream) {
+    // (enough tokens that a quarter of the threads still fills the SMs)
+    if (a.taps > 1 && (long long)a.T * (a.C / (16 / (int)sizeof(TA))) >= 4 * 148 * 512) return launch_conv_silu_tokens<TA>(a, stream);
     switch (a.taps) {
         case 1: return gl_launch(conv_silu_wide_kernel<TA, 1>, grid, dim3(256), 0, stream, 1, a);
         case 2: return gl_launch(conv_silu_wide_kernel<TA, 2>, grid, dim3(256), 0, stream, 1, a);

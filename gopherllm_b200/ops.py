@@ -1585,10 +1585,28 @@ class _PairsArgs(Structure):
 
 
 USE_PAIRS_TC = True
-USE_ROWS_DECODE_TC = True      # one token a sequence, eight or more query heads on a key head: the heads as rows of a tensor-core product
+USE_ROWS_DECODE_TC = True      # one token a sequence: the query heads of a key head as rows of a tensor-core product
 
 
-ROWS_DECODE_MIN_ROWS = 1
+def _rows_decode_takes(q, k_cache, ctx, head_dim, value_dim, mix, softcap, slopes, values_in_keys) -> bool:
+    return (USE_ROWS_DECODE_TC and ctx.max_qlen == 1 and mix is None and softcap == 0.0 and slopes is None and not DEBUG_BOUNDS
+            and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and head_dim % 16 == 0 and value_dim % 16 == 0
+            and head_dim <= 256 and value_dim <= 256 and rows_decode_smem(head_dim, value_dim, values_in_keys) <= 227 * 1024)
+
+
+def _merges_projection(q, k_cache, ctx, num_heads, num_kv_heads, head_dim, value_dim, project, mix, softcap, slopes, value_heads,
+                       values_in_keys) -> bool:
+    _need(project, "project")
+    if project.shape[0] != num_heads or project.shape[2] != value_dim:
+        raise KernelError(f"attention_mixed: per-head matrices {tuple(project.shape)} do not fit {num_heads} results of {value_dim}")
+    return project.dtype == torch.bfloat16 and _rows_decode_takes(q, k_cache, ctx, head_dim, value_dim, mix, softcap, slopes, values_in_keys)
+
+
+class _MergeProjectArgs(Structure):
+    _fields_ = [("parts", c_void_p), ("ml", c_void_p), ("w", c_void_p), ("gate", c_void_p), ("sinks", c_void_p),
+                ("seq_qstart", c_void_p), ("out", c_void_p),
+                ("B", c_int), ("nH", c_int), ("N", c_int), ("R", c_int), ("splits", c_int), ("rows_per_block", c_int), ("g_ld", c_int),
+                ("g_off", c_int)]
 
 
 class _RowsDecodeArgs(Structure):
@@ -1617,7 +1635,8 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     mix: Optional[torch.Tensor] = None, window: int = 0, score_scale: float = 1.0,
                     softcap: float = 0.0, slopes: Optional[torch.Tensor] = None,
                     sinks: Optional[torch.Tensor] = None, value_heads: int = 0, values_in_keys: bool = False,
-                    chunk: int = 0) -> torch.Tensor:
+                    chunk: int = 0, project: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                    gate_off: int = 0) -> torch.Tensor:
     """Causal softmax attention of scaled queries [T, nH*hd] over the paged cache; with ``mix`` [nH, nH]
     head h applies sum_g mix[h, g] * (head g's softmax weights) to the values of its own key/value
     head.  A score is (q . k) * score_scale, then softcap * tanh(score / softcap) when softcap > 0, then
@@ -1628,7 +1647,10 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     with one of several value heads.  ``values_in_keys``: a position's values are the first ``value_dim`` numbers of its
     key row (``v_cache`` is the key cache).  ``chunk`` n > 0 (with window 0): a query sees the keys of its own chunk of
     n positions alone, chunks counted from a sequence's start.
-    Returns [T, nH*vd] in q's type.  Prompts in bfloat16 with key and value sizes that are
+    ``project`` [nH, N, vd]: a product per head behind the result, out[t, h] = project[h] result[t, h], times
+    sigmoid(gate[t, gate_off + h]) with ``gate``; one token a sequence takes it in the kernel that puts the context's ranges
+    together.
+    Returns [T, nH*vd] (with ``project`` [T, nH*N]) in q's type.  Prompts in bfloat16 with key and value sizes that are
     multiples of 16 compute the (query head, value head) pairs on the tensor cores (a library per pair
     of sizes); everything else runs the 32-bit kernels."""
     _need(q, "q")
@@ -1642,6 +1664,11 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         _need(sinks, "sinks", torch.float32, (num_heads,))
     if chunk < 0 or (chunk > 0 and window > 0):
         raise KernelError("attention_mixed: keys are limited by a window or by chunks, not by both")
+    if project is not None and not _merges_projection(q, k_cache, ctx, num_heads, num_kv_heads, head_dim, value_dim, project, mix, softcap,
+                                                      slopes, value_heads, values_in_keys):
+        y = attention_mixed(q, k_cache, v_cache, ctx, pages, num_heads, num_kv_heads, head_dim, value_dim, mix, window, score_scale,
+                            softcap, slopes, sinks, value_heads, values_in_keys, chunk)
+        return head_linear(y, project, value_dim, gate=gate, gate_off=gate_off)
     n_val = num_kv_heads if mix is not None else 1
     nvh = int(value_heads)
     # pages a token's keys can lie on
@@ -1680,11 +1707,8 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     group, share = num_heads // num_kv_heads, num_heads // (nvh or num_kv_heads)
     # query heads that share a value head, in equal runs of up to sixteen
     rows = max(n for n in range(1, 17) if share % n == 0)
-    if (USE_ROWS_DECODE_TC and ctx.max_qlen == 1 and mix is None and softcap == 0.0 and slopes is None and not DEBUG_BOUNDS
-            and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and head_dim % 16 == 0 and value_dim % 16 == 0
-            and head_dim <= 256 and value_dim <= 256 and rows >= ROWS_DECODE_MIN_ROWS
-            and rows_decode_smem(head_dim, value_dim, values_in_keys) <= 227 * 1024):
-        # one token a sequence and many query heads on a key head: runs of heads that share a value head are the rows
+    if _rows_decode_takes(q, k_cache, ctx, head_dim, value_dim, mix, softcap, slopes, values_in_keys):
+        # one token a sequence: runs of heads that share a value head are the rows
         # of a tensor-core product over the key head's pages; the ranges are put together by the mixing kernel
         smem = rows_decode_smem(head_dim, value_dim, values_in_keys)
         splits = rows_decode_splits(ctx.n_seqs, num_heads // rows, span, q.device, smem)
@@ -1699,6 +1723,14 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                             1 if values_in_keys else 0, score_scale, chunk)
         fn = _lib("attention_mixed_tc.cu", catalog.pair_dim_defines(head_dim, value_dim)).gl_attention_rows_decode_tc
         _check(_launch(fn, byref(r), _stream()), "attention_rows_decode_tc")
+        if project is not None:
+            N = project.shape[1]
+            out = empty((T, num_heads * N), q.dtype, q.device)
+            m = _MergeProjectArgs(parts.data_ptr(), ml.data_ptr(), project.data_ptr(), _addr(gate), _addr(sinks),
+                                  ctx.seq_qstart.data_ptr(), out.data_ptr(), ctx.n_seqs, num_heads, N, value_dim, splits, 0,
+                                  gate.shape[1] if gate is not None else 0, gate_off)
+            _check(_launch(_lib("attention_mixed.cu").gl_merge_project, byref(m), _stream()), "merge_project")
+            return out
         _check(_launch(_lib("attention_mixed.cu").gl_head_mix_split, byref(a), c_int(dtype_code(q.dtype)), _stream()), "head_mix_split")
         return out
     if mix is not None:
@@ -1803,6 +1835,17 @@ def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     Returns the normed query latent [T, q_rank] (``q_rank`` 0: there is none, None)."""
     _need(proj, "proj")
     T, ld = proj.shape
+    cq = empty((T, q_rank), proj.dtype, proj.device) if q_rank else None
+    a = _latent_prepare_args(proj, k_cache, v_cache, ctx, pages, q_rank, kv_rank, rot, q_gamma, kv_gamma, eps, cos, sin, interleaved,
+                             write_kv, c_rows, cq)
+    _check(_launch(_lib("latent.cu").gl_latent_prepare, byref(a), c_int(dtype_code(proj.dtype)),
+                   c_int(dtype_code(k_cache.dtype)), _stream()), "latent_prepare")
+    return cq
+
+
+def _latent_prepare_args(proj, k_cache, v_cache, ctx, pages, q_rank, kv_rank, rot, q_gamma, kv_gamma, eps, cos, sin, interleaved,
+                         write_kv, c_rows, cq) -> _LatentPrepareArgs:
+    T, ld = proj.shape
     if ld < q_rank + kv_rank + rot:
         raise KernelError("latent_prepare: the projection's rows are too short")
     if v_cache is not None and v_cache.data_ptr() == k_cache.data_ptr():
@@ -1815,16 +1858,29 @@ def latent_prepare(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     if cos is not None:
         _need(cos, "cos", torch.float32, (T, rot // 2))
         _need(sin, "sin", torch.float32, (T, rot // 2))
-    cq = empty((T, q_rank), proj.dtype, proj.device) if q_rank else None
-    a = _LatentPrepareArgs(proj.data_ptr(), _addr(cq), k_cache.data_ptr(), _addr(v_cache), _addr(cos), _addr(sin),
-                           _addr(q_gamma), kv_gamma.data_ptr(), ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(),
-                           pages.data_ptr(), T, ld, q_rank, kv_rank, rot, pages.shape[-1], k_cache.shape[0],
-                           1 if interleaved else 0, 1 if write_kv else 0, eps, _addr(c_rows))
     if c_rows is not None:
         _need(c_rows, "c_rows", k_cache.dtype, (T, kv_rank))
-    _check(_launch(_lib("latent.cu").gl_latent_prepare, byref(a), c_int(dtype_code(proj.dtype)),
-                   c_int(dtype_code(k_cache.dtype)), _stream()), "latent_prepare")
-    return cq
+    return _LatentPrepareArgs(proj.data_ptr(), _addr(cq), k_cache.data_ptr(), _addr(v_cache), _addr(cos), _addr(sin),
+                           _addr(q_gamma), kv_gamma.data_ptr(), ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(),
+                           pages.data_ptr(), T, ld, q_rank, kv_rank, rot, pages.shape[-1], k_cache.shape[0],
+                              1 if interleaved else 0, 1 if write_kv else 0, eps, _addr(c_rows))
+
+
+def latent_queries(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, ctx, pages: torch.Tensor, kv_rank: int,
+                   rot: int, kv_gamma: torch.Tensor, eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                   interleaved: bool, w: torch.Tensor, x_head: int, x_off: int, write_kv: bool = True) -> torch.Tensor:
+    """latent_prepare without a query latent, and head_linear of the queries in the same rows (columns x_off.., a tail of
+    ``rot`` columns turned): both read the down projections, so where the sizes allow they are one grid."""
+    H, N, K = w.shape
+    if proj.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and K % 16 == 0 and N % 8 == 0 \
+            and proj.shape[1] % 8 == 0 and x_off % 8 == 0 and x_head % 8 == 0 and (N + rot) % 2 == 0 and kv_rank + rot <= 6144:
+        a = _latent_prepare_args(proj, k_cache, v_cache, ctx, pages, 0, kv_rank, rot, None, kv_gamma, eps, cos, sin, interleaved,
+                                 write_kv, None, None)
+        out, g = _head_linear_args(proj, w, x_head, rot, cos, sin, interleaved, None, 0, x_off)
+        _check(_launch(_lib("latent.cu").gl_latent_queries, byref(a), byref(g), _stream()), "latent_queries")
+        return out
+    latent_prepare(proj, k_cache, v_cache, ctx, pages, 0, kv_rank, rot, None, kv_gamma, eps, cos, sin, interleaved, write_kv)
+    return head_linear(proj, w, x_head, tail=rot, cos=cos, sin=sin, interleaved=interleaved, x_off=x_off)
 
 
 def latent_rows(k_cache: torch.Tensor, ctx, pages: torch.Tensor, kv_rank: int) -> torch.Tensor:
@@ -1854,6 +1910,13 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, x_head: int, tail: int = 0, co
     at column x_off + h * x_head) and w [H, N, K].  ``tail`` > 0: the columns x[t, h, K:K + tail] are copied behind the result, turned by
     the token's angles when cos/sin [T, tail / 2] are given; out is [T, H * (N + tail)].  ``gate`` [T, ld]: the result
     of head h is multiplied by sigmoid(gate[t, gate_off + h])."""
+    out, a = _head_linear_args(x, w, x_head, tail, cos, sin, interleaved, gate, gate_off, x_off)
+    _check(_launch(_lib("latent.cu").gl_head_linear, byref(a), c_int(dtype_code(x.dtype)), c_int(dtype_code(w.dtype)),
+                   _stream()), "head_linear")
+    return out
+
+
+def _head_linear_args(x, w, x_head, tail, cos, sin, interleaved, gate, gate_off, x_off):
     _need(x, "x")
     _need(w, "w")
     T = x.shape[0]
@@ -1872,9 +1935,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, x_head: int, tail: int = 0, co
     out = empty((T, H * (N + tail)), x.dtype, x.device)
     a = _HeadLinearArgs(x.data_ptr(), w.data_ptr(), out.data_ptr(), _addr(gate), _addr(cos), _addr(sin), T, H, N, K,
                         x.shape[1], x_head, x_off, H * (N + tail), N + tail, 0, g_row, gate_off, tail, 1 if interleaved else 0)
-    _check(_launch(_lib("latent.cu").gl_head_linear, byref(a), c_int(dtype_code(x.dtype)), c_int(dtype_code(w.dtype)),
-                   _stream()), "head_linear")
-    return out
+    return out, a
 
 
 # ---------------------------------------------------------------------------

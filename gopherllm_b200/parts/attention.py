@@ -493,15 +493,18 @@ class LatentAttention(Mixer):
         tables = self.position.tables(ctx)
         cos, sin = tables if tables is not None else (None, None)
         pages = ctx.pages[cache.group]
-        cq = ops.latent_prepare(proj, cache.k, cache.v, ctx, pages, self.q_rank, self.kv_rank, self.rot, self.q_gamma,
-                                self.kv_gamma, self.eps, cos, sin, s.position.interleaved, write_kv=cache.writes)
-        q = ops.linear(cq, self.w_uq, None, out_dtype=ctx.act_dtype) if self.q_rank else proj
-        wide = ops.head_linear(q, self.w_uk_t, s.head_dim + self.rot, tail=self.rot, cos=cos, sin=sin,
-                               interleaved=s.position.interleaved, x_off=self.q_off)
-        mixed = ops.attention_mixed(wide, cache.k, cache.v, ctx, pages, H, 1, self.kv_rank + self.rot, self.kv_rank,
-                                    window=s.window, score_scale=self.score_scale, sinks=self.sinks, values_in_keys=True)
-        o = ops.head_linear(mixed, self.w_uv, self.kv_rank, gate=proj if self.gate else None,
-                            gate_off=self.gate_off)
+        if self.q_rank:
+            cq = ops.latent_prepare(proj, cache.k, cache.v, ctx, pages, self.q_rank, self.kv_rank, self.rot, self.q_gamma,
+                                    self.kv_gamma, self.eps, cos, sin, s.position.interleaved, write_kv=cache.writes)
+            q = ops.linear(cq, self.w_uq, None, out_dtype=ctx.act_dtype)
+            wide = ops.head_linear(q, self.w_uk_t, s.head_dim + self.rot, tail=self.rot, cos=cos, sin=sin,
+                                   interleaved=s.position.interleaved)
+        else:
+            wide = ops.latent_queries(proj, cache.k, cache.v, ctx, pages, self.kv_rank, self.rot, self.kv_gamma, self.eps, cos, sin,
+                                      s.position.interleaved, self.w_uk_t, s.head_dim + self.rot, self.q_off, write_kv=cache.writes)
+        o = ops.attention_mixed(wide, cache.k, cache.v, ctx, pages, H, 1, self.kv_rank + self.rot, self.kv_rank, window=s.window,
+                                score_scale=self.score_scale, sinks=self.sinks, values_in_keys=True, project=self.w_uv,
+                                gate=proj if self.gate else None, gate_off=self.gate_off)
         return o, self.w_out, None
 
     def forward(self, xn, ctx, cache, add: Sequence[torch.Tensor], out=None) -> torch.Tensor:

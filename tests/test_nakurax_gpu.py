@@ -564,3 +564,231 @@ def test_replay_of_a_trace(tmp_path):
     check(np.fromfile(tmp_path / "4.f32", dtype="<f4").reshape(1, -1), ra[69:70], "float32", "step 4")
     assert not m.engine.cache.live_slots()
     m.close()
+
+
+def _paged(qlens, ctxs, heads, dim, vdim, g):
+    """A cache's pages in scattered order filled with random keys and values: (k, v, pages, context, per-sequence lists)."""
+    lens = [q + c for q, c in zip(qlens, ctxs)]
+    per = max(-(-n // 64) for n in lens) + 1
+    n_pages = len(lens) * per + 3
+    order = torch.randperm(n_pages, generator=g)[:len(lens) * per].reshape(len(lens), per)
+    k = torch.randn(n_pages, heads, 64, dim, generator=g).to(torch.bfloat16)
+    v = torch.randn(n_pages, heads, 64, vdim, generator=g).to(torch.bfloat16)
+    ctx = _Ctx(qlens, list(range(len(qlens))))
+    i = lambda x: torch.tensor(x, dtype=torch.int32).to(DEV)
+    ctx.seq_ctx, ctx.max_len, ctx.total_len = i(ctxs), max(lens), sum(lens)
+    ctx.seq_base = i([sum(lens[:j]) for j in range(len(lens))])
+    ctx.tok_pos = i([c + j for c, q in zip(ctxs, qlens) for j in range(q)])
+    keys = [torch.cat([k[p].transpose(0, 1) for p in order[b]], 0)[:n].double() for b, n in enumerate(lens)]      # [n, heads, dim]
+    vals = [torch.cat([v[p].transpose(0, 1) for p in order[b]], 0)[:n].double() for b, n in enumerate(lens)]
+    return k.to(DEV), v.to(DEV), order.to(torch.int32).contiguous().to(DEV), ctx, keys, vals
+
+
+def _attend(q, keys, vals, qlens, ctxs, scale, first_key, sinks=None):
+    """64-bit attention of q [T, H, D] on per-sequence keys [n, G, D] and values [n, G, V]."""
+    out, at = [], 0
+    for b, n in enumerate(qlens):
+        H, G = q.shape[1], keys[b].shape[1]
+        for j in range(n):
+            p = ctxs[b] + j
+            lo = first_key(p)
+            kk = keys[b][lo:p + 1].repeat_interleave(H // G, 1)
+            s = torch.einsum("hd,nhd->hn", q[at + j].double(), kk) * scale
+            vv = vals[b][lo:p + 1].repeat_interleave(H // vals[b].shape[1], 1)
+            e = torch.exp(s - s.max(-1, keepdim=True).values)
+            den = e.sum(-1, keepdim=True)
+            if sinks is not None:
+                den = den + torch.exp(sinks.double()[:, None] - s.max(-1, keepdim=True).values)
+            out.append(torch.einsum("hn,nhv->hv", e / den, vv))
+        at += n
+    return torch.stack(out).reshape(at, -1)
+
+
+@pytest.mark.parametrize("tiles", [1, 2])
+@pytest.mark.parametrize("chunk", [0, 1, 24, 64, 100, 300])
+def test_prompt_kernel_with_chunks_and_a_factor(chunk, tiles):
+    """The tcgen05 prompt kernel: scattered pages, shared key heads, runs that start inside chunks, both block forms."""
+    from gopherllm_b200 import ops
+    from gopherllm_b200.csrc import catalog
+    H, G, D = 4, 2, 32
+    qlens, ctxs = [300, 2, 65], [0, 129, 63]
+    g = torch.Generator().manual_seed(chunk)
+    k, v, pages, ctx, keys, vals = _paged(qlens, ctxs, G, D, D, g)
+    q = torch.randn(sum(qlens), H * D, generator=g).to(torch.bfloat16)
+    lib = ops._lib("attention_prefill_tc.cu", catalog.head_dim_defines(D))
+    try:
+        lib.gl_attention_prefill_tc_tiles(tiles)
+        got = ops.attention_prefill_tc_chunked(q.to(DEV), k, v, ctx, pages, H, G, D, chunk=chunk, score_scale=0.37).cpu().double()
+    finally:
+        lib.gl_attention_prefill_tc_tiles(0)
+    ops.check_wait_failures()
+    want = _attend(q.view(-1, H, D), keys, vals, qlens, ctxs, 0.37, lambda p: p - p % chunk if chunk else 0)
+    assert (got - want).abs().max() < 3e-2 and (got - want).abs().mean() < 3e-3
+
+
+@pytest.mark.parametrize("dim,vdim", [(32, 32), (64, 64), (16, 32), (48, 16)])
+def test_attention_on_rows(dim, vdim):
+    """Keys and values as rows of one matrix, queries inside wider rows: both kernels (equal and unequal sizes)."""
+    from gopherllm_b200 import ops
+    H = 3
+    for qlens, ctxs in (([200, 17, 64], [0, 0, 0]), ([40, 2, 130], [70, 190, 1])):
+        g = torch.Generator().manual_seed(dim + vdim)
+        lens = [a + b for a, b in zip(qlens, ctxs)]
+        ctx = _Ctx(qlens, [0, 1, 2])
+        i = lambda x: torch.tensor(x, dtype=torch.int32).to(DEV)
+        ctx.seq_ctx, ctx.max_len, ctx.total_len = i(ctxs), max(lens), sum(lens)
+        ctx.seq_base = i([sum(lens[:j]) for j in range(3)])
+        kv = torch.randn(sum(lens), H * (dim + vdim), generator=g).to(torch.bfloat16)
+        proj = torch.randn(sum(qlens), 24 + H * dim + 8, generator=g).to(torch.bfloat16)
+        got = ops.attention_rows(proj.to(DEV), 24, kv.to(DEV), ctx, torch.zeros((3, 4), dtype=torch.int32, device=DEV), H, dim, vdim, 0.2)
+        ops.check_wait_failures()
+        base = [sum(lens[:j]) for j in range(3)]
+        keys = [kv[b:b + n, :H * dim].view(n, H, dim).double() for b, n in zip(base, lens)]
+        vals = [kv[b:b + n, H * dim:].view(n, H, vdim).double() for b, n in zip(base, lens)]
+        want = _attend(proj[:, 24:24 + H * dim].reshape(-1, H, dim), keys, vals, qlens, ctxs, 0.2, lambda p: 0)
+        got = got.cpu().double()
+        assert (got - want).abs().max() < 3e-2 and (got - want).abs().mean() < 3e-3
+
+
+@pytest.mark.parametrize("heads,groups,dim,vdim", [(4, 4, 16, 32), (6, 2, 32, 16), (5, 1, 64, 64), (12, 3, 48, 48), (40, 2, 32, 32)])
+def test_one_token_attention_of_any_group(heads, groups, dim, vdim):
+    """The kernel whose rows are query heads, from one head a key head to twenty: windows, chunks, sinks, contexts cut
+    into ranges, some of them empty."""
+    from gopherllm_b200 import ops
+    ctxs = [0, 1, 63, 64, 200, 390]
+    g = torch.Generator().manual_seed(heads)
+    k, v, pages, ctx, keys, vals = _paged([1] * len(ctxs), ctxs, groups, dim, vdim, g)
+    q = torch.randn(len(ctxs), heads * dim, generator=g).to(torch.bfloat16)
+    sinks = torch.randn(heads, generator=g)
+    for kw, lo in (({}, lambda p: 0), (dict(chunk=50), lambda p: p - p % 50), (dict(window=70), lambda p: max(0, p - 69))):
+        for s in (None, sinks):
+            got = ops.attention_mixed(q.to(DEV), k, v, ctx, pages, heads, groups, dim, vdim, score_scale=0.3,
+                                      sinks=None if s is None else s.to(DEV), **kw).cpu().double()
+            want = _attend(q.view(-1, heads, dim), keys, vals, [1] * len(ctxs), ctxs, 0.3, lo, s)
+            assert (got - want).abs().max() < 3e-2, (kw, s is not None, float((got - want).abs().max()))
+
+
+@pytest.mark.parametrize("batch", [1, 7, 20])
+@pytest.mark.parametrize("heads,rank,out", [(4, 32, 24), (12, 48, 64), (32, 256, 40)])
+def test_one_token_attention_with_a_product_behind_it(heads, rank, out, batch):
+    """Values inside the key rows, ranges put together and a matrix per head behind them, gated or not, with and without
+    a sink, against the separate kernels' mathematics in 64-bit."""
+    from gopherllm_b200 import ops
+    g = torch.Generator().manual_seed(rank)
+    ctxs = [int(x) for x in torch.randint(0, 500, (batch,), generator=g)]
+    k, _, pages, ctx, keys, _ = _paged([1] * batch, ctxs, 1, rank, rank, g)
+    q = torch.randn(batch, heads * rank, generator=g).to(torch.bfloat16)
+    w = (torch.randn(heads, out, rank, generator=g) / rank ** 0.5).to(torch.bfloat16)
+    gate = torch.randn(batch, heads + 9, generator=g).to(torch.bfloat16)
+    sinks = torch.randn(heads, generator=g)
+    for s in (None, sinks):
+        for gt in (None, gate):
+            got = ops.attention_mixed(q.to(DEV), k, k, ctx, pages, heads, 1, rank, rank, score_scale=0.2, values_in_keys=True,
+                                      sinks=None if s is None else s.to(DEV), project=w.to(DEV), gate=None if gt is None else gt.to(DEV),
+                                      gate_off=5).cpu().double()
+            y = _attend(q.view(-1, heads, rank), keys, keys, [1] * batch, ctxs, 0.2, lambda p: 0, s).view(batch, heads, rank)
+            want = torch.einsum("hnr,bhr->bhn", w.double(), y)
+            if gt is not None:
+                want = want * torch.sigmoid(gt[:, 5:5 + heads].double())[:, :, None]
+            assert (got - want.reshape(batch, -1)).abs().max() < 3e-2
+
+
+def test_prompts_on_latents_and_on_keys_built_from_them():
+    """Both forms of a prompt's latent attention, in pieces that go on from cached latents: each against the plain
+    implementation, with key and value sizes equal and unequal."""
+    from gopherllm_b200.parts import attention
+    for name, cfg in (("latent", nm.only(nm.ALPHA, 0)), ("latent_twentyfour_heads", nm.only(nm.BETA, 1)), ("WIDE_latent", nm.only(WIDE, 0))):
+        folder = folder_for(name, cfg, 11)
+        toks = tokens_for(cfg, 200, 8)
+        ref = plain_logits(folder, toks)
+        m = load(folder, "bfloat16")
+        for built in (True, False):
+            attention.LATENT_BUILDS_KEYS = built
+            try:
+                for cuts in ([200], [90, 110], [33, 64, 103]):
+                    s = m.open_sequence()
+                    check(feed(m, s, toks, cuts), ref, "bfloat16", f"{name}, keys built {built}, cuts {cuts}")
+                    m.close_sequence(s)
+                a, b = m.open_sequence(), m.open_sequence()
+                m.step([(a, toks[:50])])
+                out = m.step([(a, toks[50:120]), (b, toks[:150])], [list(range(70)), list(range(150))]).cpu().numpy()
+                check(out[:70], ref[50:120], "bfloat16", f"{name}, keys built {built}, a piece in a batch")
+                check(out[70:], ref[:150], "bfloat16", f"{name}, keys built {built}, a prompt in a batch")
+                m.close_sequence(a)
+                m.close_sequence(b)
+            finally:
+                attention.LATENT_BUILDS_KEYS = True
+        m.engine.check_device()
+        m.close()
+
+
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 5])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_convolution_of_many_tokens(taps, dtype):
+    """Without an activation and with silu: sequences whose ends cut the groups of four tokens everywhere, some of one
+    token, going on from kept inputs, as many tokens as the form that shares its rows takes."""
+    from gopherllm_b200 import ops
+    g = torch.Generator().manual_seed(taps)
+    C = 1024
+    qlens = [1, 2, 601, 3, 5, 1, 700, 1203, 130]
+    T, B = sum(qlens), len(qlens)
+    ctx = _Ctx(qlens, list(range(B)))
+    x = torch.randn(T, C + 16, generator=g).to(dtype)
+    w, bias = torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
+    tail0 = torch.randn(B, 3 + C * (taps - 1), generator=g)
+    for silu in (False, True):
+        state = tail0.clone().to(DEV)
+        got = ops.conv_silu(x.to(DEV), w.to(DEV), bias.to(DEV), state, 3, ctx, x_off=8, silu=silu).cpu().double()
+        at = 0
+        for b, n in enumerate(qlens):
+            before = tail0[b, 3:].view(C, taps - 1).double().T                       # oldest first
+            rows = torch.cat([before, x[at:at + n, 8:8 + C].double()], 0)
+            want = bias.double() + sum(rows[j:j + n] * w[:, j].double() for j in range(taps))
+            if silu:
+                want = want * torch.sigmoid(want)
+            tol = 1e-4 if dtype == torch.float32 else 1e-2
+            assert ((got[at:at + n] - want).abs() <= tol * (1.0 + want.abs())).all(), (b, silu)
+            kept = state[b, 3:].view(C, taps - 1).cpu().double().T
+            assert torch.equal(kept, rows[n:]) and torch.equal(state[b, :3].cpu(), tail0[b, :3])
+            at += n
+
+
+@pytest.mark.parametrize("half", [0, 4, 6, 16])
+def test_neighbouring_dims_turned_piece_by_piece(half):
+    """Queries turned, scaled and left, keys and values to scattered cache rows, in 16-byte pieces: bfloat16 against
+    64-bit on the same inputs."""
+    from gopherllm_b200 import ops
+    H, G, D, V = 6, 2, 32, 40
+    qlens, ctxs = [70, 1, 9], [5, 64, 127]
+    g = torch.Generator().manual_seed(half)
+    _, _, pages, ctx, _, _ = _paged(qlens, ctxs, G, D, V, g)
+    T = sum(qlens)
+    per = int(pages.shape[1])
+    k = torch.full((per * 3 + 3, G, 64, D), 7.0, dtype=torch.bfloat16, device=DEV)
+    v = torch.full((per * 3 + 3, G, 64, V), 7.0, dtype=torch.bfloat16, device=DEV)
+    qkv = torch.randn(T, (H + G) * D + G * V + 8, generator=g).to(torch.bfloat16)
+    angle = torch.randn(T, half, generator=g, dtype=torch.float64)
+    cos, sin = torch.cos(angle).float(), torch.sin(angle).float()
+    for scale in (1.0, 0.3):
+        q = ops.qkv_rownorm_to_cache(qkv.to(DEV), k, v, ctx, pages, H, G, D, V, scale, cos.to(DEV) if half else None,
+                                     sin.to(DEV) if half else None, True, None, None, 0.0).cpu().double().view(T, H, D)
+
+        def turned(x):
+            y = x.double().clone()
+            if half:
+                a, b = x[..., 0:2 * half:2].double(), x[..., 1:2 * half:2].double()
+                c, s = cos.double()[:, None], sin.double()[:, None]
+                y[..., 0:2 * half:2], y[..., 1:2 * half:2] = a * c - b * s, b * c + a * s
+            return y
+        assert (q - scale * turned(qkv[:, :H * D].view(T, H, D))).abs().max() < 2e-2
+        keys, vals = turned(qkv[:, H * D:(H + G) * D].view(T, G, D)), qkv[:, (H + G) * D:(H + G) * D + G * V].view(T, G, V)
+        at, pg = 0, pages.cpu()
+        for b, n in enumerate(qlens):
+            for j in range(n):
+                p = ctxs[b] + j
+                page, r = int(pg[b, p // 64]), p % 64
+                assert (k[page, :, r].cpu().double() - keys[at + j]).abs().max() < 2e-2
+                assert torch.equal(v[page, :, r].cpu(), vals[at + j])
+            at += n
+        written = sum(qlens)
+        assert int((k[..., 0] != 7.0).sum()) <= written * G and int((v.float() != 7.0).any(-1).sum()) <= written * G
