@@ -444,7 +444,7 @@ __device__ __forceinline__ void am_range_factors(const float* ml, int splits, co
 // weighted latent: few tokens, so a block takes up to AP_TOKENS tokens of a head and a run of output rows; the merged
 // latents stay in shared memory, a warp an output row at a time (a lane 16 bytes of it), and the row is fetched before the
 // kernel waits for the one that leaves the ranges.
-#define AP_TOKENS 8
+#define AP_TOKENS 4
 #define AP_THREADS 256
 struct MergeProjectArgs {
     const float* parts;       // [B, nH, splits, R]
@@ -472,14 +472,24 @@ merge_project_kernel(MergeProjectArgs a) {
     gl_grid_wait();
     if (warp < tokens) am_range_factors(a.ml + ((size_t)(b0 + warp) * a.nH + h) * a.splits * 2, a.splits, a.sinks, h, coef + warp * 64);
     __syncthreads();
-    for (int i = threadIdx.x; i < tokens * a.R; i += AP_THREADS) {
+    for (int i = threadIdx.x * 4; i < tokens * a.R; i += AP_THREADS * 4) {
         const int t = i / a.R, d = i - t * a.R;
         const float* src = a.parts + ((size_t)(b0 + t) * a.nH + h) * a.splits * a.R + d;
         const float* c = coef + t * 64;
-        float v = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < a.splits; ++s) v = fmaf(c[s], src[(size_t)s * a.R], v);
-        y[i] = v;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s0 = 0; s0 < a.splits; s0 += 8) {       // eight ranges asked for before the first is used
+            float4 p[8];
+#pragma unroll
+            for (int s = 0; s < 8; ++s)
+                p[s] = s0 + s < a.splits ? __ldcg((const float4*)(src + (size_t)(s0 + s) * a.R)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int s = 0; s < 8; ++s) {
+                const float f = s0 + s < a.splits ? c[s0 + s] : 0.f;
+                v.x = fmaf(f, p[s].x, v.x); v.y = fmaf(f, p[s].y, v.y);
+                v.z = fmaf(f, p[s].z, v.z); v.w = fmaf(f, p[s].w, v.w);
+            }
+        }
+        *(float4*)(y + i) = v;
     }
     __syncthreads();
     for (int n = n0 + warp; n < n_end; n += AP_THREADS / 32) {

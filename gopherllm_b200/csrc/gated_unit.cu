@@ -78,16 +78,8 @@ __device__ __forceinline__ float gu_gelu(float y) {
 }
 
 template <typename TA>
-__device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u, float2 bias, float rate);
-
-template <typename TA>
 __device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u) {
-    gu_finish<TA>(g, t, c, rs, is, u, *(const float2*)(g.bias + 2 * c), g.rate[c]);
-}
-
-template <typename TA>
-__device__ __forceinline__ void gu_finish(const UnitGatesArgs& g, int t, int c, float rs, float is, float u, float2 bias, float rate) {
-    const float2 f = gu_factors<sizeof(TA) == 2>(rs + bias.x, is + bias.y, u, rate);
+    const float2 f = gu_factors<sizeof(TA) == 2>(rs + g.bias[2 * c], is + g.bias[2 * c + 1], u, g.rate[c]);
     if (!g.step) {
         g.ab[(size_t)t * g.C + c] = f;
         return;
@@ -244,16 +236,46 @@ unit_gates_tc_kernel(UnitGatesArgs g) {
         __syncthreads();
     }
     asm volatile("cp.async.wait_group 0;");
-    const int r_lo = m0 + warp * 16 + grp, r_hi = r_lo + 8;
+    // everything the results are made with is asked for before the first is stored: behind a store no load may move up
+    const int r_lo = m0 + warp * 16 + grp, c0 = n0 / 2 + t;       // this thread's channels: c0, c0 + 4, ..
+    float2 bias[8];
+    float rate[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-        const int n = n0 + j * 8 + 2 * t;
-        if (n >= N) continue;
-        const int c = n / 2, cc = blockIdx.z * size + c;
-        const float2 bias = *(const float2*)(g.bias + 2 * cc);
-        const float rate = g.rate[cc];
-        if (r_lo < g.T) gu_finish<__nv_bfloat16>(g, r_lo, cc, acc[j][0], acc[j][1], gl_load(U + (size_t)r_lo * g.C + c), bias, rate);
-        if (r_hi < g.T) gu_finish<__nv_bfloat16>(g, r_hi, cc, acc[j][2], acc[j][3], gl_load(U + (size_t)r_hi * g.C + c), bias, rate);
+        const bool ok = c0 + 4 * j < size;
+        const int cc = blockIdx.z * size + (ok ? c0 + 4 * j : 0);
+        bias[j] = *(const float2*)(g.bias + 2 * cc);
+        rate[j] = g.rate[cc];
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int r = r_lo + 8 * half;
+        if (r >= g.T) continue;
+        float u[8], s[8], y[8];
+        float* S = g.step ? g.state + (size_t)g.seq_slot[g.tok_seq[r]] * g.state_stride + blockIdx.z * size : nullptr;
+        const __nv_bfloat16* Y = (const __nv_bfloat16*)g.y + (size_t)r * g.y_ld + g.y_off + blockIdx.z * size;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int c = c0 + 4 * j;
+            const bool ok = c < size;
+            u[j] = ok ? gl_load(U + (size_t)r * g.C + c) : 0.f;
+            s[j] = ok && g.step ? S[c] : 0.f;
+            y[j] = ok && g.step ? gl_load(Y + c) : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int c = c0 + 4 * j;
+            const float2 f = gu_factors<true>(acc[j][2 * half] + bias[j].x, acc[j][2 * half + 1] + bias[j].y, u[j], rate[j]);
+            if (c >= size) continue;
+            const size_t at = (size_t)r * g.C + blockIdx.z * size + c;
+            if (!g.step) {
+                g.ab[at] = f;
+            } else {
+                const float v = fmaf(f.x, s[j], f.y);
+                S[c] = v;
+                ((__nv_bfloat16*)g.out)[at] = __float2bfloat16_rn(v * gu_gelu<__nv_bfloat16>(y[j]));
+            }
+        }
     }
 }
 

@@ -1621,12 +1621,15 @@ def rows_decode_smem(head_dim: int, value_dim: int, values_in_keys: bool) -> int
     return max(stages, 16 * (2 * head_dim + 16) + (4 * 16 * value_dim + 128) * 4)
 
 
+ROWS_DECODE_FILL = 1.0      # waves of blocks (32 query heads on a latent of 256, 32 / 64 x 1,000 positions: 44 / 52 us with one, 55 / 63 with two)
+
+
 def rows_decode_splits(batch: int, runs: int, span_pages: int, device, smem: int) -> int:
     """Ranges of pages a sequence's context is cut into for the kernel whose rows are query heads: enough blocks
-    (runs of heads x sequences x ranges) to fill the blocks an SM holds of it twice over, no range shorter than a page."""
+    (runs of heads x sequences x ranges) to fill the blocks the SMs hold of it once, no range shorter than a page."""
     pages = max(1, int(span_pages))
     per_sm = max(1, min(4, (227 * 1024) // max(1, smem)))
-    want = max(1, (2 * per_sm * sm_count(device)) // max(1, batch * runs))
+    want = max(1, int(ROWS_DECODE_FILL * per_sm * sm_count(device)) // max(1, batch * runs))
     return max(1, min(pages, want, 64))
 
 
@@ -1712,8 +1715,8 @@ def attention_mixed(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         # of a tensor-core product over the key head's pages; the ranges are put together by the mixing kernel
         smem = rows_decode_smem(head_dim, value_dim, values_in_keys)
         splits = rows_decode_splits(ctx.n_seqs, num_heads // rows, span, q.device, smem)
-        a.splits = splits
         a.pages_per_split = -(-span // splits)
+        splits = a.splits = -(-span // a.pages_per_split)          # (no range that never has a page)
         parts = empty((ctx.n_seqs, num_heads, 1, splits, value_dim), torch.float32, q.device)
         ml = empty((ctx.n_seqs, num_heads, splits, 2), torch.float32, q.device)
         a.parts, a.ml = parts.data_ptr(), ml.data_ptr()
