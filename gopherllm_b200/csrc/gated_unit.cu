@@ -279,6 +279,102 @@ unit_gates_tc_kernel(UnitGatesArgs g) {
     }
 }
 
+// The same for prompts, whose tiles are limited by what they fetch: a block takes 128 tokens x 64 channels (128 rows of
+// both gates), each of its 8 warps 32 tokens x 32 channels.
+#define GW_TILE (128 * GT_ROW)
+
+__global__ void __launch_bounds__(256, 2)
+unit_gates_wide_kernel(UnitGatesArgs g) {
+    extern __shared__ __align__(16) unsigned char smem[];     // [2] token tiles, [2] weight tiles
+    gl_grid_launch_dependents();
+    const int size = g.C / g.blocks, N = 2 * size;
+    const __nv_bfloat16* U = (const __nv_bfloat16*)g.u + (size_t)blockIdx.z * size;
+    const __nv_bfloat16* W = (const __nv_bfloat16*)g.w + (size_t)blockIdx.z * N * size;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, grp = lane >> 2, t = lane & 3;
+    const int wm = (warp & 3) * 32, wn = (warp >> 2) * 64;    // this warp's part of the tile
+    const int m0 = blockIdx.y * 128, n0 = blockIdx.x * 128;
+    const unsigned base = (unsigned)__cvta_generic_to_shared(smem);
+    auto fetch = [&](int k0, int st, bool weights) {
+        const unsigned dst = base + (weights ? 2 + st : st) * GW_TILE;
+        for (int i = tid; i < 128 * 8; i += 256) {
+            const int r = i >> 3, c = i & 7;
+            const bool ok = k0 + c * 8 < size && (weights ? n0 + r < N : m0 + r < g.T);
+            const __nv_bfloat16* src = weights ? W + (size_t)(n0 + r) * size + k0 + c * 8 : U + (size_t)(m0 + r) * g.C + k0 + c * 8;
+            gt_cp16(dst + r * GT_ROW + c * 16, ok ? (const void*)src : g.w, ok ? 16 : 0);
+        }
+    };
+    fetch(0, 0, true);                                // (weights: they come while the kernel before drains)
+    gl_grid_wait();
+    fetch(0, 0, false);
+    asm volatile("cp.async.commit_group;");
+    float acc[2][8][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
+    const int steps = (size + 63) / 64;
+    for (int s = 0; s < steps; ++s) {
+        const int st = s & 1;
+        if (s + 1 < steps) {
+            fetch((s + 1) * 64, st ^ 1, true);
+            fetch((s + 1) * 64, st ^ 1, false);
+        }
+        asm volatile("cp.async.commit_group;");
+        asm volatile("cp.async.wait_group 1;");
+        __syncthreads();
+        const int kn = (min(64, size - s * 64) + 15) / 16;        // (what a part has no columns for is zero)
+        const unsigned sa = base + st * GW_TILE, sw = base + (2 + st) * GW_TILE;
+#pragma unroll 1
+        for (int kk = 0; kk < kn; ++kk) {
+            unsigned af[2][4];
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                gt_ldm4(sa + (wm + i * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * GT_ROW + (kk * 2 + (lane >> 4)) * 16,
+                        af[i][0], af[i][1], af[i][2], af[i][3]);
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                unsigned b0, b1, b2, b3;
+                gt_ldm4(sw + (wn + j * 8 + ((lane >> 4) & 1) * 8 + (lane & 7)) * GT_ROW + (kk * 2 + ((lane >> 3) & 1)) * 16, b0, b1, b2, b3);
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    gt_mma(acc[i][j], af[i], b0, b1);
+                    gt_mma(acc[i][j + 1], af[i], b2, b3);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    asm volatile("cp.async.wait_group 0;");
+    const int c0 = (n0 + wn) / 2 + t;                  // this thread's channels: c0, c0 + 4, ..
+    float2 bias[8];
+    float rate[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        const bool ok = c0 + 4 * j < size;
+        const int cc = blockIdx.z * size + (ok ? c0 + 4 * j : 0);
+        bias[j] = *(const float2*)(g.bias + 2 * cc);
+        rate[j] = g.rate[cc];
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int r = m0 + wm + i * 16 + grp + 8 * half;
+            if (r >= g.T) continue;
+            float u[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) u[j] = c0 + 4 * j < size ? gl_load(U + (size_t)r * g.C + c0 + 4 * j) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float2 f = gu_factors<true>(acc[i][j][2 * half] + bias[j].x, acc[i][j][2 * half + 1] + bias[j].y, u[j], rate[j]);
+                if (c0 + 4 * j < size) g.ab[(size_t)r * g.C + blockIdx.z * size + c0 + 4 * j] = f;
+            }
+        }
+    }
+}
+
 GL_API int gl_unit_gates(const UnitGatesArgs* args, int act_dtype, int w_dtype, cudaStream_t stream) {
     const UnitGatesArgs& g = *args;
     if (g.T <= 0) return GL_OK;
@@ -287,7 +383,19 @@ GL_API int gl_unit_gates(const UnitGatesArgs* args, int act_dtype, int w_dtype, 
     const int size = g.C / g.blocks;
     const dim3 grid((2 * size + GG_BN - 1) / GG_BN, (g.T + GG_BM - 1) / GG_BM, g.blocks);
     if (grid.y > 65535) return GL_ERR_SHAPE;
-    if (act_dtype == GL_BF16 && w_dtype == GL_BF16 && size % 8 == 0 && !(((uintptr_t)g.u | (uintptr_t)g.w) & 15))
+    const bool pieces = act_dtype == GL_BF16 && w_dtype == GL_BF16 && size % 8 == 0 && !(((uintptr_t)g.u | (uintptr_t)g.w) & 15);
+    if (pieces && !g.step && g.T > 64 && size > 32) {
+        static bool allowed = false;
+        if (!allowed) {
+            if (cudaFuncSetAttribute(unit_gates_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 4 * GW_TILE) != cudaSuccess) {
+                cudaGetLastError();
+                return GL_ERR_SMEM;
+            }
+            allowed = true;
+        }
+        return gl_launch(unit_gates_wide_kernel, dim3((2 * size + 127) / 128, (g.T + 127) / 128, g.blocks), dim3(256), 4 * GW_TILE, stream, 1, g);
+    }
+    if (pieces)
         return gl_launch(unit_gates_tc_kernel, grid, dim3(128), 0, stream, 1, g);
     if (act_dtype == GL_F32 && w_dtype == GL_F32) return gl_launch(unit_gates_kernel<float, float>, grid, dim3(256), 0, stream, 1, g);
     if (act_dtype == GL_BF16 && w_dtype == GL_BF16)
