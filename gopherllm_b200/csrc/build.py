@@ -27,7 +27,7 @@ _ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 _BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-shared",
                "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
 # sources with hundreds of kernel instances: the device code is split and compiled on all cores
-_SOURCE_FLAGS: Dict[str, Tuple[str, ...]] = {"recurrent.cu": ("-split-compile", "0")}
+_SOURCE_FLAGS: Dict[str, Tuple[str, ...]] = {"recurrent.cu": ("-split-compile", "0"), "attention_mixed.cu": ("-split-compile", "0")}
 _lock = threading.Lock()
 _loaded: Dict[str, ctypes.CDLL] = {}
 
