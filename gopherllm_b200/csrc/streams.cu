@@ -43,7 +43,7 @@ __device__ __forceinline__ StVec<VEC> st_load(const float* p) {
 
 // NS: streams the registers hold (S of them in use)
 template <typename TO, int NS, int VEC>
-__global__ void __launch_bounds__(ST_MAX_THREADS)
+__global__ void __launch_bounds__(ST_MAX_THREADS, NS <= 4 ? 2 : 1)
 streams_kernel(StreamArgs a) {
     extern __shared__ __align__(16) float row[];          // [W]: u
     __shared__ float ws[ST_MAX_STREAMS * (ST_MAX_STREAMS + 2)];      // mix, out, in
