@@ -3,8 +3,8 @@ through a latent without positions, or by a chunked softmax attention beside a g
 layers may run several times.
 
 config.json lists the layers one by one: ``layers[i].type`` is ``latent_attention`` or ``parallel``, ``layers[i].mixer``
-the mixer's sizes and constants, ``layers[i].mlp`` a dense feed-forward or null.  ``loop``: layers start .. stop-1 run
-``times`` times in a row with the same weights, each run on a cache entry of its own.  The scaled embedding fills
+the mixer's sizes and constants, ``layers[i].mlp`` a dense feed-forward or null.  ``loop``: the range start .. stop-1 is
+passed ``times`` times before what follows it, every pass on cache entries of its own.  The scaled embedding fills
 ``streams`` equal streams; a sublayer reads a weighted sum of them and joins them all at once (see parts/block.py,
 StreamsBlock), in front of it an RMS norm with a weight; the final norm reads the streams' sum, the head has weights
 of its own.

@@ -1,8 +1,8 @@
 // A real-gated linear recurrent unit: a recurrence with a diagonal decay that the input itself sets.
 //
 // u [T, C] is split into ``blocks`` equal parts of channels; with a square matrix per part and gate,
-//     r = sigmoid(R u + r_bias),  i = sigmoid(I u + i_bias),  log a = rate_c r   (rate_c <= 0: a learned number),
-//     S_t = a S_(t-1) + sqrt(1 - a^2) i u,       out = S * gelu(y)   (tanh form; y [T, C] another branch).
+//     r = sigmoid(R u + r_bias),  i = sigmoid(I u + i_bias),  a = e^(rate_c r)   (rate_c <= 0: a learned number),
+//     S <- a S + i u sqrt(1 - a^2),       out = S * gelu(y)   (tanh form; y [T, C] another branch).
 // Everything behind the two products' 32-bit sums is 32-bit; S lives in 32-bit rows per sequence, zero at its start.
 //
 //   gl_unit_gates   both gates' products and what follows from them.  The two matrices' rows alternate (r of channel

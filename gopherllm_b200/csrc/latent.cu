@@ -108,7 +108,8 @@ GL_API int gl_latent_prepare(const LatentPrepareArgs* args, int act_dtype, int c
     const size_t smem = (size_t)(a.q_rank + a.kv_rank + a.rot) * sizeof(float);
     if (smem > 48 * 1024) return GL_ERR_SMEM;
     if (act_dtype != cache_dtype) return GL_ERR_DTYPE;
-    const dim3 g((unsigned)a.T), b(256);
+    const int n = a.q_rank + a.kv_rank + a.rot;
+    const dim3 g((unsigned)a.T), b(n <= 256 ? 64 : (n <= 512 ? 128 : 256));      // (about four numbers a thread)
     int rc;
     if (act_dtype == GL_F32) rc = gl_launch(latent_prepare_kernel<float, float>, g, b, smem, stream, 1, a);
     else if (act_dtype == GL_BF16) rc = gl_launch(latent_prepare_kernel<__nv_bfloat16, __nv_bfloat16>, g, b, smem, stream, 1, a);

@@ -1,13 +1,13 @@
 // Several residual streams instead of one (hyper-connections).
 //
-// A token's residual is S rows of W numbers, 32-bit.  A sublayer reads one weighted sum of them,
-//     u = sum_s in[s] x_s,
-// and what it returns, y, joins all of them at once, each stream becoming a weighted sum of the old ones:
-//     x_t <- sum_s mix[s, t] x_s + out[t] y          (mix is indexed [from, to]).
+// A token's residual is a matrix X of S rows of W numbers, 32-bit.  With vectors i, o of S numbers and a matrix M [S, S] a
+// sublayer is
+//     u = X^T i,      y = sublayer(norm(u)),      X <- M^T X + o y^T:
+// row s of M says where the old stream s goes, o how much of y every stream takes.
 // Between two sublayers stands one kernel that does both and the norm of the next sublayer's input: it takes y (or
 // two branches of a sublayer with a factor each, y = f a + f2 b), updates the streams in place and leaves
 // rms(u) * gamma of the new streams in the activation type.  Without y it only reads (before the first layer; behind
-// the last one, with in = 1, for selected rows); without ``in`` it only updates.
+// the last one, with i all ones, for selected rows); without ``in_share`` it only updates.
 // A block a token; the row u stays in shared memory between the sum of its squares and its use.
 #include "common.cuh"
 
@@ -18,9 +18,9 @@ struct StreamArgs {
     float* x;                 // [T, S, W]
     const float* a;           // [T, W] or null: what the sublayer returned
     const float* b;           // [T, W] or null: its second branch
-    const float* mix;         // [S, S] (from, to)
-    const float* out_share;   // [S]
-    const float* in_share;    // [S] or null: the next sublayer's weights (null: nothing is read)
+    const float* mix;         // [S, S]: M
+    const float* out_share;   // [S]: o
+    const float* in_share;    // [S] or null: the next sublayer's i (null: nothing is read)
     const float* gamma;       // [W] or null: no norm, u itself
     void* h;                  // [R, W]
     const int* rows;          // [R] or null: rows of x that are read (without an update)

@@ -260,9 +260,9 @@ class PostNormBlock(AssembledBlock):
 
 class StreamsBlock(AssembledBlock):
     """Hyper-connections: the residual is n streams x_1 .. x_n (option ``streams``) in one tensor [T, n, hidden].  A
-    sublayer reads a weighted sum of them and what it returns joins all of them at once,
-        u = sum_s in[s] x_s;  y = sublayer(norm(u));  x_t <- sum_s mix[s, t] x_s + out[t] y   (mix is [from, to]),
-    with weights of its own for the mixer ("hc1") and the feed-forward ("hc2"); a layer without a feed-forward
+    sublayer reads one combination of a token's streams X [n, hidden] and returns into all of them,
+        y = sublayer(norm(X^T i)),   X <- M^T X + o y^T,
+    with i ("in"), M ("mix", row s: where stream s goes) and o ("out") of its own for the mixer ("hc1") and the feed-forward ("hc2"); a layer without a feed-forward
     (``spec.ffn`` None, no norm2) is the first half alone.  One kernel joins a sublayer's result, reads the streams for
     the next sublayer and norms what it read, across layers too: a run finds its input in the step's context and leaves
     the next run's there (see Block).  A mixer that offers ``branches`` is summed inside that kernel."""
@@ -307,7 +307,8 @@ class StreamsBlock(AssembledBlock):
 
 
 class StreamWeights(Part):
-    """How a sublayer reads n streams ("in" [n]) and how its result joins them ("mix" [n, n], from and to; "out" [n])."""
+    """How a sublayer reads n streams ("in" [n]), where they go behind it ("mix" [n, n], a row a stream) and how much of its
+    result each takes ("out" [n])."""
     capturable = True
     launches_only = True
 

@@ -488,13 +488,14 @@ class StateSpaceDual(Mixer):
 
 
 class GatedLinearUnit(Mixer):
-    """Griffin's recurrent block with a real-gated linear recurrent unit.  Two branches of ``width`` channels,
-        y = gelu(W_y h + b_y) (tanh form),  u = conv(W_x h + b_x),
-    the convolution causal and per channel (``conv`` taps, the last the current token's, zeros before the start, bias, no
-    activation).  u falls into ``blocks`` equal parts with a square matrix per part and gate:
-        r = sigmoid(R u + b_r),  i = sigmoid(I u + b_i),  log a = -``decay`` r softplus(lam),  a = e^(log a),
-        S <- a S + sqrt(1 - a^2) i u  from S = 0;  output W_o (S y).
-    The state row holds S [width] and the convolution's last taps - 1 inputs; gates, decays and the state are 32-bit.
+    """A recurrence with a diagonal decay that its input sets (the real-gated unit of the Griffin models), multiplied by a
+    second branch.  Over ``width`` channels
+        g = gelu(W_y h + b_y) (tanh form),   u = filter(W_x h + b_x),
+    the filter per channel over the ``conv`` latest tokens, bias included; both of the unit's gates are block-diagonal products
+    of u (``blocks`` square matrices each) through a sigmoid, r and i;
+        a = e^(-``decay`` r softplus(lam)),   s <- a s + i u sqrt(1 - a^2)  (s = 0 at the start),
+    and the mixer returns W_o (s g).
+    The state row holds s [width] and the filter's latest conv - 1 inputs; gates, decays and the state are 32-bit.
     Options: ``width``, ``blocks``, ``conv``, ``decay``."""
     capturable = True
     launches_only = True

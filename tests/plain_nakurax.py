@@ -146,8 +146,8 @@ MIXERS = {"latent_attention": latent_attention, "parallel": parallel_mixer}
 
 
 def hyper_connected(X, w, pre, sublayer):
-    """X [streams, T, W]: the sublayer reads a weighted sum of the streams; every stream becomes a weighted sum of the
-    old ones (mix [from, to]) plus a share of what the sublayer returned."""
+    """X [streams, T, W]: the sublayer reads sum_s in_s X_s; stream t then holds sum_s mix_st X_s plus out_t times what the
+    sublayer returned."""
     u = sum(w[pre + "in"][s] * X[s] for s in range(X.shape[0]))
     y = sublayer(u)
     return torch.stack([sum(w[pre + "mix"][s, t] * X[s] for s in range(X.shape[0])) + w[pre + "out"][t] * y
